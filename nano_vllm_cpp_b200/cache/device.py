@@ -15,7 +15,7 @@ from typing import Optional
 
 import torch
 
-from ..parts.base import KVCacheSpec, StateCacheSpec, CompositeCacheSpec
+from ..parts.base import KVCacheSpec, StateCacheSpec, CompositeCacheSpec, SharedCacheSpec
 
 
 @dataclass
@@ -41,7 +41,7 @@ def _group_key(spec: KVCacheSpec):
 
 
 def _leaves(spec):
-    """The page and state specs inside a cache spec, composites opened, in order."""
+    """The page and state specs inside a cache spec, composites opened, in order (what is shared takes no memory)."""
     if isinstance(spec, CompositeCacheSpec):
         for p in spec.parts:
             yield from _leaves(p)
@@ -132,6 +132,11 @@ class DeviceCache:
             at, n = next(places)
             st = self.state_buffers[s.dtype][:, at:at + n].view(self.max_slots, *s.shape)
             return CacheView("state", -1, None, None, st, True, self.page_size)
+        if isinstance(s, SharedCacheSpec):        # an earlier call's entry, or one part of it, to read only
+            lent = self.views[s.call]
+            if s.part is not None and lent.parts is not None:
+                lent = lent.parts[s.part]
+            return lent.read_only()
         if isinstance(s, CompositeCacheSpec):
             return CacheView("multi", -1, None, None, None, True, self.page_size, [self._view(p, places) for p in s.parts])
         return CacheView("none")

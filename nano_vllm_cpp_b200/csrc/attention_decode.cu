@@ -70,6 +70,7 @@ struct DecArgs {
   float softcap;          // > 0: a scaled score s becomes softcap * tanh(s / softcap) (lane-per-chunk kernel only)
   int has_sink;           // the softmax's denominator also holds exp(sink): a key with that score and no value
   float sink;             // (the lane-per-chunk kernel and the merges add it; the tensor-core form does not know it)
+  HeadGate gate;          // multiplies a head's output where its final value is written (here or in the merge)
 };
 
 // Called by every thread of a block once the block has written its split's partial results for the query heads
@@ -102,7 +103,7 @@ __device__ __forceinline__ void merge_when_last(const DecArgs& a, int r, int t, 
       o = fmaf(__ldcg(a.part_o + (pi + s) * D + d), sc, o);
     }
     if (a.has_sink) ll += __expf(a.sink - mm);
-    st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, o * (ll > 0.f ? 1.f / ll : 0.f));
+    st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, o * ((ll > 0.f ? 1.f / ll : 0.f) * head_gate_of(a.gate, t, h)));
   }
 }
 
@@ -311,7 +312,7 @@ __global__ void __launch_bounds__((WARPS + 1) * 32) attention_decode_kernel(DecA
     const int h = kvh * G + g0 + g;
     if (a.splits == 1) {
       if (a.has_sink) ll += __expf(a.sink - mm);
-      st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, ll > 0.f ? o / ll : 0.f);
+      st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, ll > 0.f ? o / ll * head_gate_of(a.gate, t, h) : 0.f);
     } else {
       const size_t pi = ((size_t)r * a.Hq + h) * a.splits + split;
       a.part_o[pi * D + d] = o;
@@ -609,7 +610,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
     }
     const int h = kvh * G + g0 + gg;
     if (a.splits == 1) {
-      st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, ll > 0.f ? ov / ll : 0.f);
+      st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, ll > 0.f ? ov / ll * head_gate_of(a.gate, t, h) : 0.f);
     } else {
       const size_t pi = ((size_t)r * a.Hq + h) * a.splits + split;
       a.part_o[pi * D + d] = ov;
@@ -625,7 +626,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
 // Combines the splits of one (row, head) in split order.
 __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               const int* __restrict__ rows, void* __restrict__ out, int out_dt,
-                                              int Hq, int D, int splits, int has_sink, float sink) {
+                                              int Hq, int D, int splits, int has_sink, float sink, HeadGate gate) {
   const int r = blockIdx.x, h = blockIdx.y;
   const int t = rows ? rows[r] : r;
   const size_t pi = ((size_t)r * Hq + h) * splits;
@@ -636,7 +637,7 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, 
   float ll = 0.f;
   for (int s = 0; s < splits; ++s) ll = fmaf(part_ml[(pi + s) * 2 + 1], __expf(part_ml[(pi + s) * 2] - mm), ll);
   if (has_sink) ll += __expf(sink - mm);
-  const float inv = ll > 0.f ? 1.f / ll : 0.f;
+  const float inv = (ll > 0.f ? 1.f / ll : 0.f) * head_gate_of(gate, t, h);
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float o = 0.f;
     for (int s = 0; s < splits; ++s) o = fmaf(part_o[(pi + s) * D + d], __expf(part_ml[(pi + s) * 2] - mm), o);
@@ -743,7 +744,10 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
                                const int* rows, int R, float scale, int window, void* out, int out_dt, int Hq,
                                int Hkv, int D, int page, int num_pages, int splits, float* scratch, int* err,
                                int* split_count, int split_count_len, int has_sink, float sink_score,
-                               int float_weights, float softcap, cudaStream_t stream) {
+                               int float_weights, float softcap, const float* gate, long long gate_ld,
+                               cudaStream_t stream) {
+  // gate: head h's output of batch row t is multiplied by sigmoid(gate[t * gate_ld + h]) (nullptr: it is not); the
+  // gates must have been written before the kernel that precedes this one on the stream.
   // softcap > 0: scaled scores are capped, s -> softcap * tanh(s / softcap); like a sink it keeps the tensor-core form out.
   // has_sink: a further key with the score sink_score and no value in every softmax; it keeps the tensor-core form
   // out.  float_weights: the weights keep all their bits in their product with the values (the lane-per-chunk
@@ -766,6 +770,7 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
   a.err = err;
   a.has_sink = has_sink; a.sink = sink_score;
   a.softcap = softcap > 0.f ? softcap : 0.f;
+  a.gate = HeadGate{gate, gate_ld};
   // `split_count`: zeros (R * Hq of them are enough), kept zero from launch to launch by the kernel: the splits are
   // then added up by the block that finishes last instead of by a second kernel.  For a few rows only: with many,
   // the last blocks' sums lengthen the kernel's tail by more than the second kernel's launch costs (measured per
@@ -825,7 +830,7 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
   if (splits > 1 && !a.split_count) {
     dim3 grid(R, Hq);
     NV_RETURN_IF(launch_dep(attention_decode_merge_kernel, grid, dim3(128), 0, stream, (const float*)a.part_o,
-                            (const float*)a.part_ml, rows, out, out_dt, Hq, D, splits, has_sink, sink_score));
+                            (const float*)a.part_ml, rows, out, out_dt, Hq, D, splits, has_sink, sink_score, a.gate));
   }
   NV_RETURN_LAST();
 }
@@ -883,7 +888,7 @@ NV_API int nv_attention_decode_noalloc(const void* qkv, int q_dt, int q_stride, 
   }
   return nv_attention_decode(qkv, q_dt, q_stride, kc, vc, cache_dt, block_table, max_blocks, row_entry, positions,
                              rows, R, scale, window, out, out_dt, Hq, Hkv, D, page, num_pages, splits,
-                             g_noalloc_ptr[dev], g_noalloc_err_ptr[dev], nullptr, 0, 0, 0.f, 0, 0.f, stream);
+                             g_noalloc_ptr[dev], g_noalloc_err_ptr[dev], nullptr, 0, 0, 0.f, 0, 0.f, nullptr, 0, stream);
 }
 
 NV_API int nv_attention_decode_noalloc_status(void) {

@@ -38,6 +38,7 @@ struct PfArgs {
                             // (scale_log2 is then log2(e) alone)
   int has_sink;             // the softmax's denominator also holds exp(sink): a key with that score and no value
   float sink_log2;          // the sink's score times log2(e)
+  HeadGate gate;            // multiplies a head's output as it is written
   int terms;                // the weights enter P V as one bfloat16 term (rounded) or three (all 24 bits of the float)
 };
 
@@ -326,7 +327,8 @@ __global__ void __launch_bounds__(BM * 2, DP <= 128 ? 2 : 1) attention_prefill_k
     l_lo += exp2f(a.sink_log2 - (m_lo == -INFINITY ? 0.f : m_lo * a.scale_log2));
     l_hi += exp2f(a.sink_log2 - (m_hi == -INFINITY ? 0.f : m_hi * a.scale_log2));
   }
-  const float inv_lo = l_lo > 0.f ? 1.f / l_lo : 0.f, inv_hi = l_hi > 0.f ? 1.f / l_hi : 0.f;
+  const float inv_lo = l_lo > 0.f && live_lo ? head_gate_of(a.gate, row0 + r_lo, h) / l_lo : 0.f;
+  const float inv_hi = l_hi > 0.f && live_hi ? head_gate_of(a.gate, row0 + r_hi, h) / l_hi : 0.f;
 #pragma unroll
   for (int i = 0; i < DP / 8; ++i) {
     const int d = i * 8 + 2 * tq;
@@ -369,14 +371,14 @@ int launch_prefill(const PfArgs& a, int max_tiles64, int num_sms, cudaStream_t s
 // bfloat16 only; head_dim a multiple of 16 up to 256.  `max_tiles` >= sum over entries of
 // ceil(rows / nv_attention_prefill_tile_rows()), the smallest tile the launcher may choose; surplus CTAs leave at once.
 // Entries with fewer than `min_rows` rows are skipped (their rows of `out` stay untouched): in a mixed step the
-// single rows go to the decode kernel.
+// single rows go to the decode kernel.  gate: head h's output of row t is multiplied by sigmoid(gate[t * gate_ld + h]).
 NV_API int nv_attention_prefill_tile_rows() { return 64; }
 
 NV_API int nv_attention_prefill(const void* qkv, int q_stride, const void* kc, const void* vc,
                                 const int* block_table, int max_blocks, const int* cu_rows, const int* entry_pos0,
                                 int S, int max_tiles, float scale, int window, void* out, int Hq, int Hkv, int D,
                                 int page, int min_rows, int has_sink, float sink_score, int terms,
-                                float softcap, cudaStream_t stream) {
+                                float softcap, const float* gate, long long gate_ld, cudaStream_t stream) {
   if (D <= 0 || D > 256 || D % 16 || Hkv <= 0 || Hq % Hkv || (terms != 1 && terms != 3)) return NV_ERR_UNSUPPORTED;
   if (q_stride % 8 || ((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15)) return NV_ERR_UNSUPPORTED;
   if (S == 0 || max_tiles == 0) return NV_OK;
@@ -389,6 +391,7 @@ NV_API int nv_attention_prefill(const void* qkv, int q_stride, const void* kc, c
   a.S = S; a.q_stride = q_stride; a.max_blocks = max_blocks; a.window = window; a.Hq = Hq; a.Hkv = Hkv; a.D = D;
   a.page = page;
   a.min_rows = min_rows;
+  a.gate = HeadGate{gate, gate_ld};
   a.has_sink = has_sink; a.sink_log2 = sink_score * 1.4426950408889634f; a.terms = terms;
   static int num_sms = 0;
   if (!num_sms) {

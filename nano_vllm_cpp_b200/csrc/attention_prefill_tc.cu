@@ -52,6 +52,7 @@ struct PtArgs {
                             // (scale_log2 is then log2(e) alone)
   int has_sink;             // the softmax's denominator also holds exp(sink): a key with that score and no value
   float sink_log2;          // the sink's score times log2(e)
+  HeadGate gate;            // multiplies a head's output as it is written
   int S, max_blocks, window, Hq, Hkv, page;
   int min_rows;             // entries with fewer rows are left to another kernel
   int first_wave;           // CTAs that start alone on a multiprocessor (their number), before the second ones join them
@@ -343,7 +344,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       mbar_wait(&pv_done, (n_blocks - 1) & 1, a.err, 0x7208);
       tc_fence_after();
       if (a.has_sink) l += exp2f(a.sink_log2 - (m == -INFINITY ? 0.f : m * a.scale_log2));   // relative to the sums' reference
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = l > 0.f && live ? head_gate_of(a.gate, row0 + r, h) / l : 0.f;
 #pragma unroll
       for (int c = 0; c < D / 32; ++c) {
         float o[32];
@@ -408,9 +409,10 @@ NV_API int nv_attention_prefill_tc(const void* qkv, int q_stride, int T, const v
                                    const int* block_table, int max_blocks, const int* cu_rows, const int* entry_pos0,
                                    int S, int max_tiles, float scale, int window, void* out, int Hq, int Hkv, int D,
                                    int page, int min_rows, int weight_terms, int* err, int has_sink, float sink_score,
-                                   float softcap, cudaStream_t stream) {
+                                   float softcap, const float* gate, long long gate_ld, cudaStream_t stream) {
   // has_sink: a further key with the score sink_score and no value in every softmax.  softcap > 0: a scaled score s
-  // becomes softcap * tanh(s / softcap) before mask and softmax.
+  // becomes softcap * tanh(s / softcap) before mask and softmax.  gate: head h's output of row t is multiplied by
+  // sigmoid(gate[t * gate_ld + h]).
   if (!nv_attention_prefill_tc_usable(D, page) || Hkv <= 0 || Hq % Hkv) return NV_ERR_UNSUPPORTED;
   if (weight_terms != 1 && weight_terms != 3) return NV_ERR_UNSUPPORTED;
   if (q_stride % 8 || ((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15)) return NV_ERR_UNSUPPORTED;
@@ -420,6 +422,7 @@ NV_API int nv_attention_prefill_tc(const void* qkv, int q_stride, int T, const v
   a.scale_log2 = (softcap > 0.f ? 1.f : scale) * 1.4426950408889634f;
   a.softcap = softcap > 0.f ? softcap : 0.f;
   a.cap_in = softcap > 0.f ? scale / softcap : 0.f;
+  a.gate = HeadGate{gate, gate_ld};
   a.has_sink = has_sink ? 1 : 0;
   a.sink_log2 = sink_score * 1.4426950408889634f;
   a.S = S; a.max_blocks = max_blocks; a.window = window; a.Hq = Hq; a.Hkv = Hkv; a.page = page;

@@ -76,9 +76,16 @@ __device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f +
 // g = min(g, p0), u = clamp(u, -p0, p0), out = g sigmoid(p1 g) (u + 1).  7: the square of relu.
 #define NV_EPI_GLU_CLAMPED 6
 #define NV_EPI_RELU2 7
-#define NV_EPI_LAST NV_EPI_RELU2
+// 8: a third pairing of gate and up rows, gelu in its tanh form on the gate: out = gelu_tanh(g) u.
+#define NV_EPI_GEGLU_TANH 8
+#define NV_EPI_LAST NV_EPI_GEGLU_TANH
 // Which codes pair a gate row with an up row (two accumulators per output), and the pairings themselves.
-__host__ __device__ __forceinline__ int epi_pair(int code) { return (code == NV_EPI_SWIGLU || code == NV_EPI_GLU_CLAMPED) ? code : 0; }
+__host__ __device__ __forceinline__ int epi_pair(int code) {
+  return (code == NV_EPI_SWIGLU || code == NV_EPI_GLU_CLAMPED || code == NV_EPI_GEGLU_TANH) ? code : 0;
+}
+__device__ __forceinline__ float gelu_tanh_of(float z) {
+  return 0.5f * z * (1.f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
+}
 __host__ __device__ __forceinline__ int epi_unary(int code) { return (code >= 2 && !epi_pair(code)) ? code : 0; }
 __device__ __forceinline__ float pair_mul(int pair, float g, float u, float p0, float p1) {
   if (pair == NV_EPI_GLU_CLAMPED) {
@@ -86,6 +93,7 @@ __device__ __forceinline__ float pair_mul(int pair, float g, float u, float p0, 
     u = fminf(fmaxf(u, -p0), p0);
     return g / (1.0f + expf(-p1 * g)) * (u + 1.0f);
   }
+  if (pair == NV_EPI_GEGLU_TANH) return gelu_tanh_of(g) * u;
   return silu_mul(g, u);
 }
 __device__ __forceinline__ float epilogue_act(int act, float v, float p0 = 0.f, float p1 = 0.f) {
@@ -93,8 +101,18 @@ __device__ __forceinline__ float epilogue_act(int act, float v, float p0 = 0.f, 
   if (act == NV_EPI_RELU2) { v = fmaxf(v, 0.f); return v * v; }
   if (act == NV_EPI_XIELU) return v > 0.f ? fmaf(p0 * v, v, 0.5f * v) : fmaf(p1, expm1f(v) - v, 0.5f * v);
   if (act == NV_EPI_GELU_ERF) return 0.5f * v * (1.f + erff(v * 0.70710678118654752440f));
-  if (act == NV_EPI_GELU_TANH) return 0.5f * v * (1.f + tanhf(0.79788456080286535588f * (v + 0.044715f * v * v * v)));
+  if (act == NV_EPI_GELU_TANH) return gelu_tanh_of(v);
   return v / (1.f + expf(-v));
+}
+
+// What multiplies a query head's attention output before it is stored: sigmoid of `gate[t * ld + h]` (t the batch row, h
+// the query head), or one without a gate (gate == nullptr).
+struct HeadGate {
+  const float* gate;
+  long long ld;
+};
+__device__ __forceinline__ float head_gate_of(const HeadGate& g, long long t, int h) {
+  return g.gate ? 1.f / (1.f + expf(-g.gate[t * g.ld + h])) : 1.f;
 }
 
 // Programmatic dependent launch.  A kernel launched with the programmatic-serialization attribute may start

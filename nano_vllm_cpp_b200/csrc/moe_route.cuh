@@ -5,8 +5,8 @@
 
 #include "common.cuh"
 
-// How a row's router logits become choices and weights.  mode 0: p = softmax(logits), the K largest p are chosen
-// and weigh p (or p / their sum).  mode 1: s = sigmoid(logit) in float32; the K largest s + bias[e] are chosen
+// How a row's router logits become choices and weights.  mode 0: p = softmax(logits + bias) (bias may be nullptr), the
+// K largest p are chosen and weigh p (or p / their sum, which is the softmax over the chosen logits).  mode 1: s = sigmoid(logit) in float32; the K largest s + bias[e] are chosen
 // (bias may be nullptr) and weigh s, without the bias.  Either way the weights are multiplied by `scale`.
 struct RouteRule {
   int mode;
@@ -30,11 +30,12 @@ __device__ __forceinline__ void route_row(const float* __restrict__ r, int E, in
     }
   } else {
     float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, r[e]);
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, rule.bias ? r[e] + rule.bias[e] : r[e]);
     mx = warp_max(mx);
     double s = 0.0;
     for (int e = lane; e < E; e += 32) {
-      double v = exp((double)r[e] - (double)mx);
+      const float z = rule.bias ? r[e] + rule.bias[e] : r[e];
+      double v = exp((double)z - (double)mx);
       pr[e] = v;
       s += v;
     }

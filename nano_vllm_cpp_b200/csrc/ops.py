@@ -312,6 +312,7 @@ def add_rmsnorm(x, branch, w, eps: float, out, out32=None, *, mix=None, branch2=
 ADD_RMSNORM_MAX_MIX = 64
 
 
+EPILOGUE_PAIRS = {"geglu_tanh": 8}     # with ``swiglu``: another pairing of gate and up rows, gelu_tanh(g) u
 EPILOGUE_ACTS = {"gelu_erf": 2, "gelu_tanh": 3, "silu": 4, "relu2": 7}
 EPILOGUE_XIELU = 5          # given as the tuple ("xielu", p0, p1) with its two positive numbers
 EPILOGUE_GLU_CLAMPED = 6    # with ``swiglu``: the tuple ("glu_clamped", limit, slope) makes the pairing of gate and up rows
@@ -329,6 +330,8 @@ def _epilogue(swiglu: bool, act) -> int:
             return EPILOGUE_GLU_CLAMPED
         _need(len(act) == 3 and act[0] == "xielu", "a product's activation with numbers is ('xielu', p0, p1)")
         return EPILOGUE_XIELU
+    if swiglu and act in EPILOGUE_PAIRS:
+        return EPILOGUE_PAIRS[act]
     _need(not swiglu and act in EPILOGUE_ACTS, f"a product's activation is one of {sorted(EPILOGUE_ACTS)} and excludes swiglu")
     return EPILOGUE_ACTS[act]
 
@@ -399,13 +402,13 @@ def attention_decode_usable(k_cache, D: int) -> bool:
 
 def attention_decode(qkv, k_cache, v_cache, block_table, row_entry, positions, scale: float, window: int, out,
                      Hq: int, Hkv: int, D: int, max_context: int, rows=None, err=None, sink_score=None,
-                     float_weights: bool = False, softcap: float = 0.0) -> None:
+                     float_weights: bool = False, softcap: float = 0.0, gate=None) -> None:
     """One query row per request (``rows``: which batch rows; None = all) against its paged keys.  ``qkv``: rows
     whose first Hq * D elements are the query heads.  ``sink_score``: a further key with that score and no value
     in every softmax.  ``float_weights``: the weights keep all their bits in the product with the values (the
     tensor-core form takes them as three bfloat16 terms instead of one rounded one; the kernel that gives a lane a
     chunk of a key, which other head sizes and a sink go to, multiplies in float32).  ``softcap`` > 0: a scaled score s
-    becomes ``softcap * tanh(s / softcap)`` (the lane-per-chunk kernel)."""
+    becomes ``softcap * tanh(s / softcap)`` (the lane-per-chunk kernel).  ``gate``: see ``_head_gates``."""
     _cuda_contig(qkv, k_cache, v_cache, block_table, row_entry, positions, out, rows)
     _i32(block_table, row_entry, positions, rows)
     R = qkv.shape[0] if rows is None else rows.numel()
@@ -423,8 +426,18 @@ def attention_decode(qkv, k_cache, v_cache, block_table, row_entry, positions, s
                                  splits, _p(scratch), _p(err.t if err is not None else _global_err().t),
                                  _p(counts), (counts.numel() if counts is not None else 0),
                                  (0 if sink_score is None else 1), float(sink_score or 0.0),
-                                 (1 if float_weights else 0), float(softcap), _stream()),
-           "attention_decode")
+                                 (1 if float_weights else 0), float(softcap), *_head_gates(gate, qkv.shape[0], Hq),
+                                 _stream()), "attention_decode")
+
+
+def _head_gates(gate, T: int, Hq: int):
+    """``gate`` (float32 [T, Hq], rows ``stride(0)`` apart, or None): head h's attention output of row t is multiplied by
+    ``sigmoid(gate[t, h])`` where it is written.  What the attention launchers take for it."""
+    if gate is None:
+        return None, 0
+    _need(gate.is_cuda and gate.dtype == torch.float32 and gate.shape == (T, Hq) and gate.stride(1) == 1,
+          "attention: the gates are float32, one column per query head")
+    return _p(gate), gate.stride(0)
 
 
 _counts = {}
@@ -445,13 +458,15 @@ def attention_prefill_tile_rows() -> int:
 
 def attention_prefill(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, max_tiles: int, scale: float,
                       window: int, out, Hq: int, Hkv: int, D: int, err=None, min_rows: int = 1,
-                      kernel: str = "auto", sink_score=None, weight_terms: int = 1, softcap: float = 0.0) -> None:
+                      kernel: str = "auto", sink_score=None, weight_terms: int = 1, softcap: float = 0.0,
+                      gate=None) -> None:
     """bfloat16 rows of any mix of portions against their paged keys: the tcgen05 kernel for head sizes 64 and
     128 and pages of 16, 32 or 64 keys, else the mma.sync kernel (``kernel="mma"`` asks for that one).  Entries
     with fewer than ``min_rows`` rows are skipped and their rows of ``out`` left as they are.
     ``weight_terms`` = 3: the float32 weights enter the product with the values as three bfloat16 terms, all their
     bits (either kernel).  ``sink_score``: a further key with that score and no value in every softmax; ``softcap``
-    > 0: a scaled score s becomes ``softcap * tanh(s / softcap)`` before mask and softmax (either kernel)."""
+    > 0: a scaled score s becomes ``softcap * tanh(s / softcap)`` before mask and softmax (either kernel).  ``gate``: see
+    ``_head_gates``."""
     _cuda_contig(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, out)
     _i32(block_table, cu_rows, entry_pos0)
     _need(qkv.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
@@ -469,14 +484,15 @@ def attention_prefill(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, m
                                          window, _p(out), Hq, Hkv, D, page,
                                          min_rows, weight_terms, _p(err.t if err is not None else _global_err().t),
                                          (0 if sink_score is None else 1), float(sink_score or 0.0), float(softcap),
-                                         _stream()),
+                                         *_head_gates(gate, qkv.shape[0], Hq), _stream()),
                "attention_prefill_tc")
         return
     _check(L.nv_attention_prefill(_p(qkv), qkv.shape[1], _p(k_cache), _p(v_cache), _p(block_table),
                                   block_table.shape[1], _p(cu_rows), _p(entry_pos0), S,
                                   max_tiles, scale, window, _p(out), Hq, Hkv,
                                   D, page, min_rows, (0 if sink_score is None else 1), float(sink_score or 0.0),
-                                  weight_terms, float(softcap), _stream()), "attention_prefill")
+                                  weight_terms, float(softcap), *_head_gates(gate, qkv.shape[0], Hq), _stream()),
+           "attention_prefill")
 
 
 def attention_prefill_wide_usable(D: int, key_span: int, Dv: int) -> bool:
@@ -599,14 +615,15 @@ ROUTE_SCORES = {"softmax": 0, "sigmoid": 1}
 
 
 def _route_rule(rule, E: int):
-    """``rule`` = None (softmax, no bias, weights as they are) or (score kind, choice bias [E] float32 or None,
-    weight scale): what the routing kernels take as their last three arguments."""
+    """``rule`` = None (softmax, no bias, weights as they are) or (score kind, bias [E] float32 or None, weight scale):
+    what the routing kernels take as their last three arguments.  With sigmoid scores the bias steers the choice only;
+    with softmax scores it is added to the logits."""
     if rule is None:
         return 0, None, 1.0
     kind, bias, scale = rule
     _need(kind in ROUTE_SCORES, f"router: the score is one of {sorted(ROUTE_SCORES)}")
-    _need(bias is None or (kind == "sigmoid" and bias.is_cuda and bias.dtype == torch.float32 and bias.is_contiguous()
-                           and bias.numel() == E), "router: the choice bias is float32 [E], with sigmoid scores")
+    _need(bias is None or (bias.is_cuda and bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == E),
+          "router: the bias is float32 [E]")
     return ROUTE_SCORES[kind], bias, float(scale)
 
 
@@ -1047,7 +1064,7 @@ def qk_prepare_store(src, q0: int, k0: int, v0: int, positions, row_entry, block
                      inv_freq, rot_dim: int, interleaved: bool, amplitude: float, q_out, k_cache, v_cache,
                      Hq: int, Hkv: int, D: int, Dv: int, write_kv: bool, err: ErrorFlag, *, v_inv_freq=None,
                      v_rot_dim: int = 0, rot0: int = 0, k_norm_dim: int = 0, norm_always: bool = False,
-                     norm_after: bool = False) -> None:
+                     norm_after: bool = False, norm_whole: bool = False) -> None:
     """Per row: q and k heads RMS-normed over D (weights may be None), their first ``rot_dim`` elements turned in
     pairs by the row's position, q to ``q_out`` [T, Hq * D], k and v to the row's place in their pages.
     ``Hq`` may be 0 (``q_out`` None: only keys and values are written) and ``v_cache`` None (only keys).
@@ -1055,12 +1072,16 @@ def qk_prepare_store(src, q0: int, k0: int, v0: int, positions, row_entry, block
     ``(i, i + v_rot_dim / 2)`` by ``position * v_inv_freq[i]``, before they are stored.
     ``rot0``: the turned elements are ``rot0 .. rot0 + rot_dim - 1`` of a head.  ``k_norm_dim`` > 0: a key head's norm is
     taken over, and applied to, its first so many elements only.  ``norm_always``: heads are normed also where the
-    weight is None (the weight is then one).  ``norm_after``: the norm follows the turn instead of preceding it."""
+    weight is None (the weight is then one).  ``norm_after``: the norm follows the turn instead of preceding it.
+    ``norm_whole``: the norm is taken over all q heads at once, and over all k heads at once, instead of head by head
+    (the weights then have an entry per element of all heads)."""
     _cuda_contig(positions, row_entry, block_table, q_weight, k_weight, inv_freq, q_out, k_cache, v_cache, v_inv_freq)
     _i32(positions, row_entry, block_table)
     _f32(q_weight, k_weight, inv_freq, v_inv_freq)
     T = src.shape[0]
     page = k_cache.shape[2]
+    _need(not norm_whole or (not norm_after and k_norm_dim == 0 and (q_weight is None or q_weight.numel() == Hq * D)
+                             and (k_weight is None or k_weight.numel() == Hkv * D)), "qk_prepare_store: norm over all heads")
     QP = q_out.shape[1] // Hq if Hq else D
     KP, VP = k_cache.shape[3], (v_cache.shape[3] if v_cache is not None else Dv)   # a head's elements, padded with zeros
     _need(src.stride(-1) == 1 and (Hq == 0 or q_out.shape == (T, Hq * QP)) and QP >= D, "qk_prepare_store: shapes")
@@ -1078,20 +1099,22 @@ def qk_prepare_store(src, q0: int, k0: int, v0: int, positions, row_entry, block
                                      (dt(q_out) if q_out is not None else 0),
                                      _p(k_cache), _p(v_cache), dt(k_cache), Hq, Hkv, D, Dv, page,
                                      (1 if write_kv else 0), _p(err.t), T, QP, KP, VP, _p(v_inv_freq), v_rot_dim,
-                                     rot0, k_norm_dim, (1 if norm_always else 0) | (2 if norm_after else 0),
+                                     rot0, k_norm_dim, (1 if norm_always else 0) | (2 if norm_after else 0)
+                                     | (4 if norm_whole else 0),
                                      _stream()), "qk_prepare_store")
 
 
 def paged_attention_general(q, k_cache, v_cache, block_table, row_entry, positions, scale: float, window: int, out,
                             Hq: int, Hkv: int, D: int, Dv: int, sink_score=None, *, sinks=None, keep_first: int = 0,
-                            key_span: int = 1, value_heads: int | None = None, softcap: float = 0.0) -> None:
+                            key_span: int = 1, value_heads: int | None = None, softcap: float = 0.0,
+                            gate=None) -> None:
     """Causal softmax attention of every row over its request's paged keys; values may be wider or narrower than
     keys; ``sink_score``: a further key with that score and no value in every softmax (None: none), ``sinks``
     (float32 [Hq]): one such score per head; ``keep_first``: with a window, the sequence's first so many positions
     stay visible; ``key_span`` = Hkv: a query row holds Hkv * D elements per head and a score is the sum of its
     parts' products with all kv heads' keys (see ``mix_query_heads``); ``v_cache`` None: the values are read where
     the keys are; ``value_heads``: kv heads of the values where that is not ``Hkv``; ``softcap`` > 0: a scaled score
-    s becomes ``softcap * tanh(s / softcap)`` before mask and softmax."""
+    s becomes ``softcap * tanh(s / softcap)`` before mask and softmax; ``gate``: see ``_head_gates``."""
     if v_cache is None:
         v_cache = k_cache
     Hv = Hkv if value_heads is None else value_heads
@@ -1107,7 +1130,7 @@ def paged_attention_general(q, k_cache, v_cache, block_table, row_entry, positio
                                             block_table.shape[1], _p(row_entry), _p(positions), scale, window,
                                             keep_first, (0 if sink_score is None else 1), float(sink_score or 0.0),
                                             _p(sinks), _p(out), dt(out), T, Hq, Hkv, Hv, D, Dv, key_span,
-                                            k_cache.shape[2], float(softcap), _stream()),
+                                            k_cache.shape[2], float(softcap), *_head_gates(gate, T, Hq), _stream()),
            "paged_attention_general")
 
 
@@ -1133,6 +1156,78 @@ def rotate_heads(x, positions, inv_freq, rot_dim: int, sign: float, out, H: int,
           and x.data_ptr() != out.data_ptr(), "rotate_heads: shapes")
     _check(lib().nv_rotate_heads(_p(x), dt(x), _p(positions), _p(inv_freq), rot_dim, float(sign), _p(out), dt(out),
                                  T, H, D, _stream()), "rotate_heads")
+
+
+def causal_conv_add(h, w, batch, state, out) -> None:
+    """``out[t, c] = h[t, c] + sum_j w[j, c] * h[t - (taps - 1) + j, c]``: a causal convolution over time on every channel,
+    added to its input.  ``h`` float32 [T, H], ``w`` float32 [taps, H] (the last row the current token's), ``state``
+    [slots, taps - 1, H] float32: what came before the rows of this step (None with one tap), brought up to date here."""
+    _cuda_contig(h, w, out)
+    _f32(h, w)
+    T, H = h.shape
+    taps = w.shape[0]
+    _need(w.shape == (taps, H) and out.shape == (T, H) and out.data_ptr() != h.data_ptr(), "causal_conv_add: shapes")
+    _need(taps == 1 or (state is not None and state.shape[1:] == (taps - 1, H)), "causal_conv_add: state")
+    single = taps > 1 and batch.decode_only
+    _check(lib().nv_causal_conv_add(_p(h), _p(w), taps, _p(batch.row_entry), _p(batch.cu_rows), _p(batch.entry_slot),
+                                    _p(state) if taps > 1 else None, _slot_stride(state) if taps > 1 else 0, _p(out), dt(out),
+                                    T, H, 1 if single else 0, _stream()), "causal_conv_add",
+           nbytes=float(T) * H * (4 + out.element_size()))
+    if taps > 1 and not single:
+        conv_state_update(h, 0, H, taps, batch, state)
+
+
+def retention_usable(form: str, dk: int, dv: int) -> bool:
+    """``form``: ``step`` (entries of one row), ``chunks`` (entries of many rows on the tensor cores) or ``scan``."""
+    return bool(lib().nv_retention_usable({"step": 0, "chunks": 1, "scan": 2}[form], dk, dv))
+
+
+def retention_chunk_rows() -> int:
+    return 64
+
+
+def retention(proj, cols: dict, batch, S, powers, inv_freq, rot_dim: int, H: int, dk: int, dv: int, eps: float, out,
+              *, fast: bool = True) -> None:
+    """Linear attention with a fixed decay per head, from and to the entries' states ``S`` [slots, H, dk, dv]: per head
+    ``S = d S + k v^T``, ``o = S^T q`` with q and k turned by their positions (pairs ``(i, i + rot_dim / 2)``) and k times
+    ``dk^-1/2``; ``out = o / sqrt(mean(o^2) + eps) * silu(gate)``.  ``proj`` float32 [T, P] holds q, k, v and the gate at
+    ``cols``; ``powers`` float32 [H, 65]: the decays to the power 0 .. 64.  ``fast``: entries of one row in one launch,
+    the others in chunks on the tensor cores; else (or where those do not take the sizes) the scan."""
+    _cuda_contig(proj, powers, inv_freq, out)
+    _f32(proj, powers, inv_freq)
+    T = proj.shape[0]
+    rc = retention_chunk_rows()
+    _need(powers.shape == (H, rc + 1) and out.shape == (T, H * dv) and S.shape[1:] == (H, dk, dv), "retention: shapes")
+    _need(rot_dim % 2 == 0 and 0 <= rot_dim <= dk and inv_freq.numel() >= rot_dim // 2, "retention: rotation")
+    half = rot_dim // 2
+    dev = proj.device
+
+    def launch(what, name, *, table=None, rows=None, R=0, raw=None, chunks=None, max_chunks=0, min_rows=1, flops=0.0):
+        _check(lib().nv_retention(what, _p(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols["g"], _p(table),
+                                  _p(batch.positions), _p(inv_freq), half, _p(batch.row_entry), _p(batch.cu_rows),
+                                  _p(batch.entry_slot), batch.S, _p(rows), R, _p(S), _slot_stride(S), _p(powers),
+                                  float(dk) ** -0.5, float(eps), _p(out), dt(out), _p(raw), _p(chunks), max_chunks, T, H, dk,
+                                  dv, min_rows, _stream()), name, flops)
+
+    single = batch.n_single if fast and retention_usable("step", dk, dv) else 0
+    if single:
+        launch(0, "retention_step", rows=None if batch.decode_only else batch.single_rows, R=single)
+    if single == batch.S:
+        return
+    table = None
+    if half:
+        table = torch.empty((T, half, 2), dtype=torch.float32, device=dev)
+        _check(lib().nv_rotary_table(_p(batch.positions), _p(inv_freq), half, _p(table), T, _stream()), "rotary_table")
+    min_rows = 2 if single else 1
+    if fast and retention_usable("chunks", dk, dv):
+        # an upper bound of the entries' chunks that depends on the step's totals only (surplus blocks leave at once)
+        most = (T - single) // rc + (batch.S - single)
+        chunks = torch.empty((most, H, dk, dv), dtype=torch.int32, device=dev)
+        launch(1, "retention_chunks", table=table, chunks=chunks, max_chunks=most, min_rows=min_rows,
+               flops=4.0 * T * H * dk * dv)
+    else:
+        raw = torch.empty((T, H, dv), dtype=torch.float32, device=dev)
+        launch(2, "retention_scan", table=table, raw=raw, min_rows=min_rows)
 
 
 def cols_rmsnorm(src, col0: int, n: int, w, eps: float, out) -> None:
@@ -1186,7 +1281,8 @@ def stream_mix_norm(x, streams: int, *, branch=None, mix=None, carry=None, write
        ``sum_c carry[c, d] * x_c + write[d] * y`` (``carry`` [streams, streams] indexed [from, to], ``write``
        [streams]); with one copy and neither tensor ``x += y``;
     2. ``u = sum_d read[d] * x_d`` (``read`` None: the plain sum of the copies);
-    3. ``norm`` = (alpha [1], gain [H], shift [H]), all float32: ``tanh(alpha * u) * gain + shift``; None: u itself;
+    3. ``norm`` = (alpha [1], gain [H], shift [H]), all float32: ``tanh(alpha * u) * gain + shift``; ``norm`` =
+       ("rms", gain [H], eps): ``u / sqrt(mean(u^2) + eps) * gain``; None: u itself;
     4. the result goes to ``out`` (float32 or bfloat16) and / or ``out32``; with neither, only step 1 is done."""
     _need(x.dtype == torch.float32 and x.is_cuda and x.is_contiguous() and x.dim() == 2 and x.shape[1] % streams == 0,
           "stream_mix_norm: the copies are float32 [T, streams * H]")
@@ -1212,7 +1308,15 @@ def stream_mix_norm(x, streams: int, *, branch=None, mix=None, carry=None, write
               and write.dtype == torch.float32 and write.numel() == streams, "stream_mix_norm: carry / write shapes")
     _need(read is None or (read.dtype == torch.float32 and read.numel() == streams), "stream_mix_norm: read shape")
     alpha = gain = shift = None
-    if norm is not None:
+    kind, eps = 0, 0.0
+    if norm is not None and isinstance(norm[0], str):
+        _need(norm[0] == "rms", "stream_mix_norm: the norm with a name is 'rms'")
+        _, gain, eps = norm
+        kind = 2
+        _f32(gain)
+        _need(gain.numel() == H and gain.is_contiguous(), "stream_mix_norm: norm shapes")
+    elif norm is not None:
+        kind = 1
         alpha, gain, shift = norm
         _f32(alpha, gain, shift)
         _need(alpha.numel() == 1 and gain.numel() == H and shift.numel() == H, "stream_mix_norm: norm shapes")
@@ -1220,8 +1324,7 @@ def stream_mix_norm(x, streams: int, *, branch=None, mix=None, carry=None, write
         for t_ in (x, branch, rows, dense, out, out32, gain, shift):
             _need(t_ is None or t_.data_ptr() % 16 == 0, "stream_mix_norm: rows must start on 16-byte boundaries")
     _check(lib().nv_stream_mix_norm(_p(x), T, streams, H, _p(branch), _p(rows), _p(index), _p(weight), R, _p(dense),
-                                    _p(carry), _p(write), _p(read), (0 if norm is None else 1), _p(alpha), _p(gain),
-                                    _p(shift), _p(out), (dt(out) if out is not None else 0), _p(out32), _stream()),
+                                    _p(carry), _p(write), _p(read), kind, _p(alpha), _p(gain), _p(shift), float(eps), _p(out), (dt(out) if out is not None else 0), _p(out32), _stream()),
            "stream_mix_norm", nbytes=4.0 * T * H * (2 * streams + 2))
 
 

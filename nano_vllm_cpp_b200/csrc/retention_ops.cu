@@ -1,0 +1,917 @@
+// Retention (linear attention with one fixed decay per head) and the causal convolution over a mixer's input.
+//
+//   causal_conv_add        out = h + conv(h), a short convolution over time on every channel, its history kept per request
+//   rotary_table           cosine and sine of every row's angles, shared by the heads
+//   retention_step         entries of one row: rotation, state update, output, head norm and gate in one launch
+//   retention_scan         any sizes, row by row (the twin of the others; float32 runs)
+//   retention_chunk_*      entries of many rows on the tensor cores, 64 rows at a time
+//
+// Per head with the decay d, keys k (turned by their positions, times dk^-1/2) and values v:
+//   S_t = d S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t,   y_t = o_t / sqrt(mean(o_t^2) + eps) * silu(gate_t).
+// S lives in float32.  The chunked form writes the recurrence for the rows i = 0 .. n - 1 of a chunk that starts from S:
+//   o_i = d^(i+1) S^T q_i + sum_{j <= i} d^(i-j) (q_i . k_j) v_j,   S' = d^n S + sum_j d^(n-1-j) k_j v_j^T
+// in three launches: every chunk's own sum over j (all chunks at once), a pass over each entry's chunks that turns
+// these into the states the chunks start from, and every chunk's outputs (all chunks at once).  All operands of the
+// tensor-core products are float32 numbers split into two bfloat16 terms (hi, and what its rounding left), with the
+// three products hi hi, hi lo and lo hi, so that a product carries sixteen bits of each operand; sums are float32.
+#include "common.cuh"
+
+#include <algorithm>
+
+namespace {
+
+// ------------------------------------------------------------------ causal convolution
+struct ConvArgs {
+  const float* h;           // [T, H]
+  const float* w;           // [taps, H]: row j multiplies the input taps - 1 - j positions back
+  const int* row_entry;
+  const int* cu_rows;
+  const int* entry_slot;
+  float* state;             // per slot [taps - 1, H]: the inputs of the request's last taps - 1 positions
+  long long slot_stride;
+  void* out;
+  int out_dt, T, H, taps, rows, update;
+};
+
+template <int VEC>
+struct Vals { float v[VEC]; };
+template <int VEC>
+__device__ __forceinline__ Vals<VEC> ldv(const float* p) {
+  Vals<VEC> c;
+  if (VEC == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    c.v[0] = q.x; c.v[VEC > 1 ? 1 : 0] = q.y; c.v[VEC > 2 ? 2 : 0] = q.z; c.v[VEC > 3 ? 3 : 0] = q.w;
+  } else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) c.v[j] = p[j];
+  }
+  return c;
+}
+template <int VEC>
+__device__ __forceinline__ void stv(float* p, const Vals<VEC>& c) {
+  if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(c.v[0], c.v[VEC > 1 ? 1 : 0], c.v[VEC > 2 ? 2 : 0], c.v[VEC > 3 ? 3 : 0]);
+  else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) p[j] = c.v[j];
+  }
+}
+template <int VEC>
+__device__ __forceinline__ void st_out(void* out, int dt, size_t i, const Vals<VEC>& c) {
+  if (VEC == 4 && dt == NV_DT_BF16) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(c.v[0], c.v[VEC > 1 ? 1 : 0]);
+    const __nv_bfloat162 hi = __floats2bfloat162_rn(c.v[VEC > 2 ? 2 : 0], c.v[VEC > 3 ? 3 : 0]);
+    uint2 pk;
+    pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+    pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>((bf16*)out + i) = pk;
+  } else if (VEC == 4) {
+    stv<VEC>((float*)out + i, c);
+  } else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) st_dt(out, dt, i + j, c.v[j]);
+  }
+}
+
+// A thread owns VEC channels and `rows` consecutive rows of the batch; the inputs it still needs stay in registers from
+// row to row (TAPS > 0) and come from the request's state where they lie before the entry.  `update`: the state is
+// brought up to date here too, which is safe where every entry has one row (nobody else reads it).
+// The taps are added in ascending order of time, whatever the cut, so a row's result does not depend on it.
+template <int VEC, int TAPS>
+__global__ void __launch_bounds__(256) causal_conv_add_kernel(ConvArgs a) {
+  grid_dep_wait();
+  grid_dep_launch();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c * VEC >= a.H) return;
+  const size_t col = (size_t)c * VEC;
+  const int t0 = blockIdx.x * a.rows, t1 = min(a.T, t0 + a.rows);
+  constexpr int HN = TAPS > 1 ? TAPS - 1 : 1;
+  Vals<VEC> hist[HN], w[TAPS > 0 ? TAPS : 1];          // hist[d - 1]: the input d positions back
+  const int taps = TAPS > 0 ? TAPS : a.taps;
+  if (TAPS > 0) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = ldv<VEC>(a.w + (size_t)j * a.H + col);
+  }
+  for (int t = t0; t < t1; ++t) {
+    const int e = a.row_entry[t];
+    const int j = t - a.cu_rows[e];
+    float* st = a.state + (size_t)a.entry_slot[e] * a.slot_stride + col;
+    auto back = [&](int d) {
+      return j >= d ? ldv<VEC>(a.h + (size_t)(t - d) * a.H + col) : ldv<VEC>(st + (size_t)(taps - 1 + j - d) * a.H);
+    };
+    const Vals<VEC> cur = ldv<VEC>(a.h + (size_t)t * a.H + col);
+    Vals<VEC> acc;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc.v[i] = 0.f;
+    if (TAPS > 0) {
+      if (t == t0 || j == 0) {
+#pragma unroll
+        for (int d = 1; d < TAPS; ++d) hist[d - 1] = back(d);
+      }
+#pragma unroll
+      for (int d = TAPS - 1; d >= 1; --d)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) acc.v[i] = fmaf(w[TAPS - 1 - d].v[i], hist[d - 1].v[i], acc.v[i]);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) acc.v[i] = cur.v[i] + fmaf(w[TAPS > 0 ? TAPS - 1 : 0].v[i], cur.v[i], acc.v[i]);
+      st_out<VEC>(a.out, a.out_dt, (size_t)t * a.H + col, acc);
+#pragma unroll
+      for (int d = HN - 1; d >= 1; --d) hist[d] = hist[d - 1];
+      hist[0] = cur;
+      if (a.update && TAPS > 1) {
+#pragma unroll
+        for (int s = 0; s < TAPS - 1; ++s) stv<VEC>(st + (size_t)s * a.H, hist[TAPS - 2 - s]);
+      }
+    } else {
+      for (int d = taps - 1; d >= 1; --d) {
+        const Vals<VEC> x = back(d), wd = ldv<VEC>(a.w + (size_t)(taps - 1 - d) * a.H + col);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) acc.v[i] = fmaf(wd.v[i], x.v[i], acc.v[i]);
+      }
+      const Vals<VEC> wl = ldv<VEC>(a.w + (size_t)(taps - 1) * a.H + col);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) acc.v[i] = cur.v[i] + fmaf(wl.v[i], cur.v[i], acc.v[i]);
+      st_out<VEC>(a.out, a.out_dt, (size_t)t * a.H + col, acc);
+      if (a.update)
+        for (int s = 0; s < taps - 1; ++s)
+          stv<VEC>(st + (size_t)s * a.H, s + 1 < taps - 1 ? ldv<VEC>(st + (size_t)(s + 1) * a.H) : cur);
+    }
+  }
+}
+
+// ------------------------------------------------------------------ rotation
+__global__ void rotary_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq, int half,
+                                    float2* __restrict__ out, long long n) {
+  grid_dep_wait();
+  grid_dep_launch();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float ang = (float)positions[i / half] * inv_freq[i % half];
+  out[i] = make_float2(cosf(ang), sinf(ang));
+}
+
+struct RetArgs {
+  const float* proj;        // [T, ld]: q | k | v | gate at their columns, heads side by side
+  long long ld;
+  int q0, k0, v0, g0;
+  const float2* table;      // [T, half]: cosine and sine (the step kernel works them out itself)
+  const int* positions;
+  const float* inv_freq;
+  int half;                 // pairs (i, i + half) of the first 2 half elements of a q or k head are turned
+  const int* row_entry;
+  const int* cu_rows;
+  const int* entry_slot;
+  const int* rows;          // step: which batch rows (nullptr: all)
+  float* S;                 // [slots][H, dk, dv]
+  long long S_stride;
+  const float* powers;      // [H, RC + 1]: the decay to the power 0 .. RC
+  float k_scale, eps;
+  void* out;                // [T, H * dv]
+  float* raw;               // scan: [T, H, dv]
+  uint32_t* chunks;         // chunked form: per chunk and head dk * dv words (float32 sums, then the states' two terms)
+  int out_dt, H, dk, dv, num_entries, min_rows, slice, v2;
+};
+
+constexpr int RC = 64;                 // rows of a chunk
+constexpr int RT_THREADS = 256;
+
+__device__ __forceinline__ float silu_of(float x) { return x / (1.f + expf(-x)); }
+
+// ------------------------------------------------------------------ one row per entry
+// grid (rows, heads).  The head's matrix streams through registers once: a thread owns VEC neighbouring columns and every
+// RS-th row of it, and the threads' shares of the output are added in order through shared memory.
+template <int VEC>
+__global__ void __launch_bounds__(RT_THREADS) retention_step_kernel(RetArgs a) {
+  extern __shared__ float sm[];        // q [dk], k [dk], shares [RS][dv]
+  __shared__ float red[RT_THREADS / 32];
+  const int h = blockIdx.y, tid = threadIdx.x, dk = a.dk, dv = a.dv, half = a.half;
+  const int t = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
+  const int groups = dv / VEC, RS = RT_THREADS / groups;
+  float* q = sm;
+  float* k = q + dk;
+  float* share = k + dk;
+  float* Sg = a.S + (size_t)a.entry_slot[a.row_entry[t]] * a.S_stride + (size_t)h * dk * dv;
+  const float* p = a.proj + (size_t)t * a.ld;
+  const int cg = tid % groups, rs = tid / groups;
+  const bool owner = rs < RS;
+  constexpr int U = 8;                 // rows of the matrix in flight per thread
+  // The state's first rows are asked for before the projections of this step are there.
+  Vals<VEC> cur[U];
+  if (owner) {
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (rs + u * RS < dk) cur[u] = ldv<VEC>(Sg + (size_t)(rs + u * RS) * dv + cg * VEC);
+  }
+  grid_dep_wait();
+  grid_dep_launch();
+  const int items = half + (dk - 2 * half);
+  for (int i = tid; i < items; i += RT_THREADS) {
+    const float* pq = p + a.q0 + (size_t)h * dk;
+    const float* pk = p + a.k0 + (size_t)h * dk;
+    if (i < half) {
+      const float ang = (float)a.positions[t] * a.inv_freq[i];
+      const float cs = cosf(ang), sn = sinf(ang);
+      q[i] = pq[i] * cs - pq[i + half] * sn;
+      q[i + half] = pq[i + half] * cs + pq[i] * sn;
+      k[i] = (pk[i] * cs - pk[i + half] * sn) * a.k_scale;
+      k[i + half] = (pk[i + half] * cs + pk[i] * sn) * a.k_scale;
+    } else {
+      q[i + half] = pq[i + half];
+      k[i + half] = pk[i + half] * a.k_scale;
+    }
+  }
+  const float d = a.powers[(size_t)h * (RC + 1) + 1];
+  __syncthreads();
+  if (owner) {
+    Vals<VEC> v, o;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      v.v[i] = p[a.v0 + (size_t)h * dv + cg * VEC + i];
+      o.v[i] = 0.f;
+    }
+    for (int r0 = rs; r0 < dk; r0 += U * RS) {
+      if (r0 != rs) {
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+          if (r0 + u * RS < dk) cur[u] = ldv<VEC>(Sg + (size_t)(r0 + u * RS) * dv + cg * VEC);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int r = r0 + u * RS;
+        if (r < dk) {
+          const float kr = k[r], qr = q[r];
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) {
+            cur[u].v[i] = fmaf(d, cur[u].v[i], kr * v.v[i]);
+            o.v[i] = fmaf(cur[u].v[i], qr, o.v[i]);
+          }
+          stv<VEC>(Sg + (size_t)r * dv + cg * VEC, cur[u]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) share[(size_t)rs * dv + cg * VEC + i] = o.v[i];
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < dv; c += RT_THREADS) {
+    float o = 0.f;
+    for (int i = 0; i < RS; ++i) o += share[(size_t)i * dv + c];
+    share[c] = o;                      // (column c's shares are read by this thread alone)
+    ss = fmaf(o, o, ss);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < RT_THREADS / 32; ++i) sum += red[i];
+  const float r = rsqrtf(sum / (float)dv + a.eps);
+  for (int c = tid; c < dv; c += RT_THREADS)
+    st_dt(a.out, a.out_dt, ((size_t)t * a.H + h) * dv + c, share[c] * r * silu_of(p[a.g0 + (size_t)h * dv + c]));
+}
+
+// ------------------------------------------------------------------ any sizes, row by row
+// grid (entries, heads, slices of `slice` columns); the slice of the head's matrix lives in shared memory.
+__global__ void __launch_bounds__(RT_THREADS) retention_scan_kernel(RetArgs a) {
+  extern __shared__ float sm[];        // S [dk][slice], q [dk], k [dk], shares [RS][slice]
+  const int e = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, dk = a.dk, dv = a.dv, half = a.half, W = a.slice;
+  const int row0 = a.cu_rows[e], row1 = a.cu_rows[e + 1];
+  if (row1 - row0 < a.min_rows) return;
+  const int RS = RT_THREADS / W, c = tid % W, rs = tid / W, col = blockIdx.z * W + c;
+  float* S = sm;
+  float* q = S + (size_t)dk * W;
+  float* k = q + dk;
+  float* share = k + dk;
+  float* Sg = a.S + (size_t)a.entry_slot[e] * a.S_stride + (size_t)h * dk * dv;
+  for (int r = rs; r < dk; r += RS) S[r * W + c] = col < dv ? Sg[(size_t)r * dv + col] : 0.f;
+  const float d = a.powers[(size_t)h * (RC + 1) + 1];
+  const int items = half + (dk - 2 * half);
+  for (int t = row0; t < row1; ++t) {
+    const float* p = a.proj + (size_t)t * a.ld;
+    const float* pq = p + a.q0 + (size_t)h * dk;
+    const float* pk = p + a.k0 + (size_t)h * dk;
+    for (int i = tid; i < items; i += RT_THREADS) {
+      if (i < half) {
+        const float2 cs = a.table[(size_t)t * half + i];
+        q[i] = pq[i] * cs.x - pq[i + half] * cs.y;
+        q[i + half] = pq[i + half] * cs.x + pq[i] * cs.y;
+        k[i] = (pk[i] * cs.x - pk[i + half] * cs.y) * a.k_scale;
+        k[i + half] = (pk[i + half] * cs.x + pk[i] * cs.y) * a.k_scale;
+      } else {
+        q[i + half] = pq[i + half];
+        k[i + half] = pk[i + half] * a.k_scale;
+      }
+    }
+    __syncthreads();
+    const float v = col < dv ? p[a.v0 + (size_t)h * dv + col] : 0.f;
+    float o = 0.f;
+    for (int r = rs; r < dk; r += RS) {
+      const float s = fmaf(d, S[r * W + c], k[r] * v);
+      S[r * W + c] = s;
+      o = fmaf(s, q[r], o);
+    }
+    share[rs * W + c] = o;
+    __syncthreads();
+    if (rs == 0 && col < dv) {
+      float sum = 0.f;
+      for (int i = 0; i < RS; ++i) sum += share[i * W + c];
+      a.raw[((size_t)t * a.H + h) * dv + col] = sum;
+    }
+  }
+  if (col < dv)
+    for (int r = rs; r < dk; r += RS) Sg[(size_t)r * dv + col] = S[r * W + c];
+}
+
+// A row and head per warp: y = o / sqrt(mean(o^2) + eps) * silu(gate), for the rows of entries with min_rows or more.
+__global__ void __launch_bounds__(256) retention_finish_kernel(RetArgs a, int T) {
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= (long long)T * a.H) return;
+  const int t = (int)(item / a.H), h = (int)(item % a.H), dv = a.dv;
+  const int e = a.row_entry[t];
+  if (a.cu_rows[e + 1] - a.cu_rows[e] < a.min_rows) return;
+  const float* x = a.raw + (size_t)item * dv;
+  float ss = 0.f;
+  for (int i = lane; i < dv; i += 32) ss = fmaf(x[i], x[i], ss);
+  const float r = rsqrtf(warp_sum(ss) / (float)dv + a.eps);
+  for (int i = lane; i < dv; i += 32)
+    st_dt(a.out, a.out_dt, (size_t)item * dv + i, x[i] * r * silu_of(a.proj[(size_t)t * a.ld + a.g0 + (size_t)h * dv + i]));
+}
+
+// ------------------------------------------------------------------ the chunked form
+constexpr int CK_THREADS = 128;        // four warps
+constexpr int VLD = 64 + 8;            // row of a 64-column slab in shared memory (sixteen bytes of padding)
+
+__device__ __forceinline__ uint32_t s_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm4(const bf16* p, uint32_t* r) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s_u32(p)));
+}
+__device__ __forceinline__ void ldsm4_t(const bf16* p, uint32_t* r) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s_u32(p)));
+}
+__device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// Two floats as packed bfloat16 pairs: their roundings, and the roundings of what those left.
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __bfloat162float(h.x), y - __bfloat162float(h.y));
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ void split1(float x, bf16* hi, bf16* lo) {
+  const bf16 h = __float2bfloat16_rn(x);
+  *hi = h;
+  *lo = __float2bfloat16_rn(x - __bfloat162float(h));
+}
+// c += a b for operands in two terms each (the product of the two small terms is left out)
+__device__ __forceinline__ void mma_terms(float* c, const uint32_t* ah, const uint32_t* al, uint32_t bh0, uint32_t bh1,
+                                          uint32_t bl0, uint32_t bl1) {
+  mma16816(c, ah, bh0, bh1);
+  mma16816(c, ah, bl0, bl1);
+  mma16816(c, al, bh0, bh1);
+}
+
+// Which (entry, chunk of it) is chunk number `want` of the step?  Entries with fewer than min_rows rows have none.
+// Called by warp 0; info: entry (-1: none), first row in the batch, rows.
+__device__ __forceinline__ void find_chunk(const int* cu_rows, int S, int min_rows, int want, int* info) {
+  const int lane = threadIdx.x & 31;
+  int base = 0;
+  for (int b = 0; b < S; b += 32) {
+    const int e = b + lane;
+    const int n = e < S ? cu_rows[e + 1] - cu_rows[e] : 0;
+    const int mine = n >= min_rows ? (n + RC - 1) / RC : 0;
+    int inc = mine;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int up = __shfl_up_sync(0xffffffffu, inc, o);
+      if (lane >= o) inc += up;
+    }
+    const int total = __shfl_sync(0xffffffffu, inc, 31);
+    if (want < base + total) {
+      if (base + inc > want && base + inc - mine <= want) {
+        const int at = want - (base + inc - mine);
+        info[0] = e;
+        info[1] = cu_rows[e] + at * RC;
+        info[2] = min(RC, n - at * RC);
+      }
+      return;
+    }
+    base += total;
+  }
+  if (lane == 0) info[0] = -1;
+}
+
+// Rows row0 .. row0 + n - 1 of one q or k head, turned, times factor(row), as two bfloat16 terms in shared memory
+// [RC][LDS]; rows beyond n and elements beyond dk are zero.
+template <int DKP, typename F>
+__device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, int row0, int n, F factor, bf16* hi, bf16* lo) {
+  constexpr int LDS = DKP + 8;
+  const int half = a.half, dk = a.dk, tid = threadIdx.x;
+  if (a.v2) {                          // two neighbouring elements at a time (sizes and addresses are even)
+    const int h2 = half / 2, items = h2 + (dk - 2 * half) / 2;
+    for (int x = tid; x < RC * items; x += CK_THREADS) {
+      const int r = x / items, i = x - r * items;
+      const bool live = r < n;
+      const float f = live ? factor(r) : 0.f;
+      const float* p = src + (size_t)(row0 + (live ? r : 0)) * a.ld;
+      uint32_t wh, wl;
+      if (i < h2) {
+        const float2 u = *reinterpret_cast<const float2*>(p + 2 * i), w = *reinterpret_cast<const float2*>(p + 2 * i + half);
+        const float4 cs = *reinterpret_cast<const float4*>(a.table + (size_t)(row0 + (live ? r : 0)) * half + 2 * i);
+        split2(live ? (u.x * cs.x - w.x * cs.y) * f : 0.f, live ? (u.y * cs.z - w.y * cs.w) * f : 0.f, wh, wl);
+        *reinterpret_cast<uint32_t*>(hi + r * LDS + 2 * i) = wh;
+        *reinterpret_cast<uint32_t*>(lo + r * LDS + 2 * i) = wl;
+        split2(live ? (w.x * cs.x + u.x * cs.y) * f : 0.f, live ? (w.y * cs.z + u.y * cs.w) * f : 0.f, wh, wl);
+        *reinterpret_cast<uint32_t*>(hi + r * LDS + 2 * i + half) = wh;
+        *reinterpret_cast<uint32_t*>(lo + r * LDS + 2 * i + half) = wl;
+      } else {
+        const int d = 2 * half + 2 * (i - h2);
+        const float2 u = *reinterpret_cast<const float2*>(p + d);
+        split2(live ? u.x * f : 0.f, live ? u.y * f : 0.f, wh, wl);
+        *reinterpret_cast<uint32_t*>(hi + r * LDS + d) = wh;
+        *reinterpret_cast<uint32_t*>(lo + r * LDS + d) = wl;
+      }
+    }
+  } else {
+    const int items = half + (dk - 2 * half);
+    for (int x = tid; x < RC * items; x += CK_THREADS) {
+      const int r = x / items, i = x - r * items;
+      const bool live = r < n;
+      const float f = live ? factor(r) : 0.f;
+      const float* p = src + (size_t)(row0 + (live ? r : 0)) * a.ld;
+      if (i < half) {
+        const float2 cs = a.table[(size_t)(row0 + (live ? r : 0)) * half + i];
+        const float u = p[i], w = p[i + half];
+        split1(live ? (u * cs.x - w * cs.y) * f : 0.f, hi + r * LDS + i, lo + r * LDS + i);
+        split1(live ? (w * cs.x + u * cs.y) * f : 0.f, hi + r * LDS + i + half, lo + r * LDS + i + half);
+      } else {
+        split1(live ? p[i + half] * f : 0.f, hi + r * LDS + i + half, lo + r * LDS + i + half);
+      }
+    }
+  }
+  const int pad = DKP - dk;
+  for (int x = tid; x < RC * pad; x += CK_THREADS) {
+    const int i = (x / pad) * LDS + dk + x % pad;
+    hi[i] = lo[i] = __float2bfloat16_rn(0.f);
+  }
+}
+
+// Columns c0 .. c0 + 63 of the value head of the chunk's rows, as two terms [RC][VLD]; what does not exist is zero.
+__device__ __forceinline__ void load_values(const RetArgs& a, const float* src, int row0, int n, int c0, bf16* hi, bf16* lo) {
+  if (a.v2) {
+    for (int x = threadIdx.x; x < RC * 32; x += CK_THREADS) {
+      const int r = x / 32, c = 2 * (x % 32);
+      float2 v = make_float2(0.f, 0.f);
+      if (r < n && c0 + c < a.dv) v = *reinterpret_cast<const float2*>(src + (size_t)(row0 + r) * a.ld + c0 + c);
+      uint32_t wh, wl;
+      split2(v.x, v.y, wh, wl);
+      *reinterpret_cast<uint32_t*>(hi + r * VLD + c) = wh;
+      *reinterpret_cast<uint32_t*>(lo + r * VLD + c) = wl;
+    }
+  } else {
+    for (int x = threadIdx.x; x < RC * 64; x += CK_THREADS) {
+      const int r = x / 64, c = x % 64;
+      const float v = r < n && c0 + c < a.dv ? src[(size_t)(row0 + r) * a.ld + c0 + c] : 0.f;
+      split1(v, hi + r * VLD + c, lo + r * VLD + c);
+    }
+  }
+}
+
+// Every chunk's own sum: U = sum_j d^(n-1-j) k_j v_j^T, float32 [dk][dv].  grid (chunks, heads).
+template <int DKP>
+__global__ void __launch_bounds__(CK_THREADS) retention_chunk_sum_kernel(RetArgs a) {
+  constexpr int LDS = DKP + 8;
+  extern __shared__ __align__(16) uint8_t ck_smem[];
+  bf16* kh = (bf16*)ck_smem;
+  bf16* kl = kh + RC * LDS;
+  bf16* vh = kl + RC * LDS;
+  bf16* vl = vh + RC * VLD;
+  __shared__ int info[3];
+  __shared__ float pw[RC + 1];
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+  grid_dep_wait();
+  grid_dep_launch();
+  if (warp == 0) find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
+  for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
+  __syncthreads();
+  if (info[0] < 0) return;
+  const int row0 = info[1], n = info[2];
+  const float ks = a.k_scale;
+  load_turned<DKP>(a, a.proj + a.k0 + (size_t)h * a.dk, row0, n, [&](int r) { return pw[n - 1 - r] * ks; }, kh, kl);
+  float* U = reinterpret_cast<float*>(a.chunks) + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
+  const int g = lane / 4, tq = lane % 4;
+  const bool even = (a.dv & 1) == 0;
+  for (int c0 = 0; c0 < a.dv; c0 += 64) {
+    if (c0) __syncthreads();
+    load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < DKP / 64; ++m) {
+      const int d0 = (m * 4 + warp) * 16;            // this warp's sixteen rows of U
+      if (d0 >= a.dk) continue;
+      float c[8][4];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
+#pragma unroll
+      for (int kb = 0; kb < RC / 16; ++kb) {
+        if (kb * 16 >= n) continue;
+        uint32_t ah[4], al[4];
+        const int at = (kb * 16 + (lane % 8) + 8 * (lane / 16)) * LDS + d0 + 8 * ((lane / 8) % 2);
+        ldsm4_t(kh + at, ah);
+        ldsm4_t(kl + at, al);
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          uint32_t bh[4], bl[4];
+          const int bt = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + np * 16 + 8 * (lane / 16);
+          ldsm4_t(vh + bt, bh);
+          ldsm4_t(vl + bt, bl);
+          mma_terms(c[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+          mma_terms(c[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int col = c0 + i * 8 + 2 * tq;
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int d = d0 + g + 8 * half;
+          if (d >= a.dk || col >= a.dv) continue;
+          float* p = U + (size_t)d * a.dv + col;
+          if (even) *reinterpret_cast<float2*>(p) = make_float2(c[i][2 * half], c[i][2 * half + 1]);
+          else {
+            p[0] = c[i][2 * half];
+            if (col + 1 < a.dv) p[1] = c[i][2 * half + 1];
+          }
+        }
+      }
+    }
+  }
+}
+
+// Turns an entry's chunk sums into the states its chunks start from, each packed as its two bfloat16 terms in one word
+// (in place: the same thread reads and writes an element), and leaves the last state in the request's slot.
+// grid (entries, heads, elements / 256).
+__global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
+  __shared__ int first_s;
+  const int e = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  grid_dep_wait();
+  grid_dep_launch();
+  const int n = a.cu_rows[e + 1] - a.cu_rows[e];
+  if (n < a.min_rows) return;
+  if (tid < 32) {                      // chunks of the entries before this one
+    int sum = 0;
+    for (int i = tid; i < e; i += 32) {
+      const int m = a.cu_rows[i + 1] - a.cu_rows[i];
+      sum += m >= a.min_rows ? (m + RC - 1) / RC : 0;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if (tid == 0) first_s = sum;
+  }
+  __syncthreads();
+  const int i = blockIdx.z * 256 + tid, size = a.dk * a.dv;
+  if (i >= size) return;
+  const int count = (n + RC - 1) / RC;
+  const size_t step = (size_t)a.H * size;
+  uint32_t* p = a.chunks + ((size_t)first_s * a.H + h) * size + i;
+  float* Sg = a.S + (size_t)a.entry_slot[e] * a.S_stride + (size_t)h * size + i;
+  const float full = a.powers[(size_t)h * (RC + 1) + RC], last = a.powers[(size_t)h * (RC + 1) + n - (count - 1) * RC];
+  float S = *Sg;
+  constexpr int U = 8;                 // chunk sums in flight
+  for (int c0 = 0; c0 < count; c0 += U) {
+    float u[U];
+#pragma unroll
+    for (int j = 0; j < U; ++j) u[j] = c0 + j < count ? __uint_as_float(p[(size_t)(c0 + j) * step]) : 0.f;
+#pragma unroll
+    for (int j = 0; j < U; ++j)
+      if (c0 + j < count) {
+        const bf16 hi = __float2bfloat16_rn(S);
+        const __nv_bfloat162 pk = __halves2bfloat162(hi, __float2bfloat16_rn(S - __bfloat162float(hi)));
+        p[(size_t)(c0 + j) * step] = *reinterpret_cast<const uint32_t*>(&pk);
+        S = fmaf(c0 + j + 1 < count ? full : last, S, u[j]);
+      }
+  }
+  *Sg = S;
+}
+
+// Every chunk's outputs, its heads normed and gated.  grid (chunks, heads); a warp takes sixteen rows and all columns.
+// NS: slabs of 64 value columns.
+template <int DKP, int NS>
+__global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs a) {
+  constexpr int LDS = DKP + 8;
+  constexpr int KS = RC * LDS > DKP * VLD ? RC * LDS : DKP * VLD;      // the keys' place is the state's afterwards
+  extern __shared__ __align__(16) uint8_t ck_smem[];
+  bf16* qh = (bf16*)ck_smem;
+  bf16* ql = qh + RC * LDS;
+  bf16* kh = ql + RC * LDS;
+  bf16* kl = kh + KS;
+  bf16* vh = kl + KS;
+  bf16* vl = vh + RC * VLD;
+  __shared__ int info[3];
+  __shared__ float pw[RC + 1];
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+  grid_dep_wait();
+  grid_dep_launch();
+  if (warp == 0) find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
+  for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
+  __syncthreads();
+  if (info[0] < 0) return;
+  const int row0 = info[1], n = info[2];
+  const float ks = a.k_scale;
+  load_turned<DKP>(a, a.proj + a.q0 + (size_t)h * a.dk, row0, n, [](int) { return 1.f; }, qh, ql);
+  load_turned<DKP>(a, a.proj + a.k0 + (size_t)h * a.dk, row0, n, [&](int) { return ks; }, kh, kl);
+  __syncthreads();
+  const int g = lane / 4, tq = lane % 4;
+  const int r_lo = warp * 16 + g, r_hi = r_lo + 8;
+  const int q_at = (warp * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * LDS + 8 * (lane / 16);
+  const bool busy = warp * 16 < n;
+
+  // the weights d^(i-j) (q_i . k_j) of this warp's rows, two terms, as operands of the product with the values
+  uint32_t ph[4][4], pl[4][4];
+  {
+    float s[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+    if (busy) {
+#pragma unroll
+      for (int kk = 0; kk < DKP / 16; ++kk) {
+        uint32_t ah[4], al[4];
+        ldsm4(qh + q_at + kk * 16, ah);
+        ldsm4(ql + q_at + kk * 16, al);
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          if (np > warp) continue;                 // keys after this warp's last row
+          uint32_t bh[4], bl[4];
+          const int at = (np * 16 + (lane % 8) + 8 * (lane / 16)) * LDS + kk * 16 + 8 * ((lane / 8) % 2);
+          ldsm4(kh + at, bh);
+          ldsm4(kl + at, bl);
+          mma_terms(s[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+          mma_terms(s[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int j = i * 8 + 2 * tq + x;
+        s[i][x] = j <= r_lo ? s[i][x] * pw[r_lo - j] : 0.f;
+        s[i][2 + x] = j <= r_hi ? s[i][2 + x] * pw[r_hi - j] : 0.f;
+      }
+#pragma unroll
+    for (int kb = 0; kb < 4; ++kb) {
+      split2(s[2 * kb][0], s[2 * kb][1], ph[kb][0], pl[kb][0]);
+      split2(s[2 * kb][2], s[2 * kb][3], ph[kb][1], pl[kb][1]);
+      split2(s[2 * kb + 1][0], s[2 * kb + 1][1], ph[kb][2], pl[kb][2]);
+      split2(s[2 * kb + 1][2], s[2 * kb + 1][3], ph[kb][3], pl[kb][3]);
+    }
+  }
+  const uint32_t* St = a.chunks + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
+  const float f_lo = pw[r_lo + 1], f_hi = pw[r_hi + 1];
+  float o[NS][8][4];
+  float ss_lo = 0.f, ss_hi = 0.f;
+#pragma unroll
+  for (int sl = 0; sl < NS; ++sl) {
+    const int c0 = sl * 64;
+    __syncthreads();                               // the keys (or the last slab) have been read by everyone
+    load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
+    if (a.v2) {
+      for (int x = tid; x < DKP * 32; x += CK_THREADS) {
+        const int d = x / 32, c = 2 * (x % 32);
+        uint2 w = make_uint2(0, 0);
+        if (d < a.dk && c0 + c < a.dv) w = *reinterpret_cast<const uint2*>(St + (size_t)d * a.dv + c0 + c);
+        *reinterpret_cast<uint32_t*>(kh + d * VLD + c) = __byte_perm(w.x, w.y, 0x5410);
+        *reinterpret_cast<uint32_t*>(kl + d * VLD + c) = __byte_perm(w.x, w.y, 0x7632);
+      }
+    } else {
+      for (int x = tid; x < DKP * 64; x += CK_THREADS) {
+        const int d = x / 64, c = x % 64;
+        const uint32_t w = d < a.dk && c0 + c < a.dv ? St[(size_t)d * a.dv + c0 + c] : 0u;
+        const __nv_bfloat162 pk = *reinterpret_cast<const __nv_bfloat162*>(&w);
+        kh[d * VLD + c] = pk.x;
+        kl[d * VLD + c] = pk.y;
+      }
+    }
+    __syncthreads();
+    float (&oc)[8][4] = o[sl];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) oc[i][0] = oc[i][1] = oc[i][2] = oc[i][3] = 0.f;
+    if (!busy) continue;
+#pragma unroll
+    for (int kk = 0; kk < DKP / 16; ++kk) {
+      if (kk * 16 >= a.dk) continue;
+      uint32_t ah[4], al[4];
+      ldsm4(qh + q_at + kk * 16, ah);
+      ldsm4(ql + q_at + kk * 16, al);
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        uint32_t bh[4], bl[4];
+        const int at = (kk * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + np * 16 + 8 * (lane / 16);
+        ldsm4_t(kh + at, bh);
+        ldsm4_t(kl + at, bl);
+        mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+        mma_terms(oc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { oc[i][0] *= f_lo; oc[i][1] *= f_lo; oc[i][2] *= f_hi; oc[i][3] *= f_hi; }
+#pragma unroll
+    for (int kb = 0; kb < 4; ++kb) {
+      if (kb > warp) continue;
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        uint32_t bh[4], bl[4];
+        const int at = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + np * 16 + 8 * (lane / 16);
+        ldsm4_t(vh + at, bh);
+        ldsm4_t(vl + at, bl);
+        mma_terms(oc[2 * np], ph[kb], pl[kb], bh[0], bh[1], bl[0], bl[1]);
+        mma_terms(oc[2 * np + 1], ph[kb], pl[kb], bh[2], bh[3], bl[2], bl[3]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {                  // (columns beyond dv are zero)
+      ss_lo = fmaf(oc[i][0], oc[i][0], fmaf(oc[i][1], oc[i][1], ss_lo));
+      ss_hi = fmaf(oc[i][2], oc[i][2], fmaf(oc[i][3], oc[i][3], ss_hi));
+    }
+  }
+  ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 1);
+  ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
+  ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 1);
+  ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 2);
+  const float n_lo = rsqrtf(ss_lo / (float)a.dv + a.eps), n_hi = rsqrtf(ss_hi / (float)a.dv + a.eps);
+#pragma unroll
+  for (int sl = 0; sl < NS; ++sl)
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int col = sl * 64 + i * 8 + 2 * tq;
+      if (col >= a.dv) continue;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = half ? r_hi : r_lo;
+        if (r >= n) continue;
+        const float rn = half ? n_hi : n_lo;
+        const float* gp = a.proj + (size_t)(row0 + r) * a.ld + a.g0 + (size_t)h * a.dv + col;
+        const size_t at = ((size_t)(row0 + r) * a.H + h) * a.dv + col;
+        const float x = o[sl][i][2 * half] * rn, y = o[sl][i][2 * half + 1] * rn;
+        if (a.v2 && a.out_dt == NV_DT_BF16) {
+          const float2 gg = *reinterpret_cast<const float2*>(gp);
+          *reinterpret_cast<__nv_bfloat162*>((bf16*)a.out + at) = __floats2bfloat162_rn(x * silu_of(gg.x), y * silu_of(gg.y));
+        } else {
+          st_dt(a.out, a.out_dt, at, x * silu_of(gp[0]));
+          if (col + 1 < a.dv) st_dt(a.out, a.out_dt, at + 1, y * silu_of(gp[1]));
+        }
+      }
+    }
+}
+
+template <typename K>
+int allow(K kernel, size_t bytes) {
+  if (bytes > 227 * 1024) return NV_ERR_UNSUPPORTED;
+  if (bytes > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return NV_OK;
+}
+
+int step_vec(int dv) { return dv % 4 == 0 ? 4 : 1; }
+
+template <int DKP>
+size_t chunk_sum_smem() { return sizeof(bf16) * (2 * (size_t)RC * (DKP + 8) + 2 * (size_t)RC * VLD); }
+template <int DKP>
+size_t chunk_out_smem() {
+  const size_t ks = std::max((size_t)RC * (DKP + 8), (size_t)DKP * VLD);
+  return sizeof(bf16) * (2 * (size_t)RC * (DKP + 8) + 2 * ks + 2 * (size_t)RC * VLD);
+}
+
+template <int DKP, int NS>
+int launch_chunks(const RetArgs& a, int max_chunks, cudaStream_t s) {
+  int rc = allow(retention_chunk_sum_kernel<DKP>, chunk_sum_smem<DKP>());
+  if (rc) return rc;
+  rc = allow(retention_chunk_out_kernel<DKP, NS>, chunk_out_smem<DKP>());
+  if (rc) return rc;
+  const dim3 grid(max_chunks, a.H);
+  NV_RETURN_IF(launch_dep(retention_chunk_sum_kernel<DKP>, grid, dim3(CK_THREADS), chunk_sum_smem<DKP>(), s, a));
+  NV_RETURN_IF(launch_dep(retention_chunk_pass_kernel, dim3(a.num_entries, a.H, (a.dk * a.dv + 255) / 256), dim3(256), 0, s, a));
+  NV_RETURN_IF(launch_dep(retention_chunk_out_kernel<DKP, NS>, grid, dim3(CK_THREADS), chunk_out_smem<DKP>(), s, a));
+  NV_RETURN_LAST();
+}
+
+template <int DKP>
+int launch_chunks_ns(const RetArgs& a, int max_chunks, cudaStream_t s) {
+  if (a.dv <= 64) return launch_chunks<DKP, 1>(a, max_chunks, s);
+  if (a.dv <= 128) return launch_chunks<DKP, 2>(a, max_chunks, s);
+  return launch_chunks<DKP, 4>(a, max_chunks, s);
+}
+
+}  // namespace
+
+// out = h + conv(h).  h: [T, H] float32; w: [taps, H] float32; state: per slot [taps - 1, H] float32 (nullptr with one
+// tap).  `update` (allowed where every entry of the step has one row): the state is brought up to date as well.
+NV_API int nv_causal_conv_add(const float* h, const float* w, int taps, const int* row_entry, const int* cu_rows,
+                              const int* entry_slot, float* state, long long slot_stride, void* out, int out_dt, int T,
+                              int H, int update, cudaStream_t s) {
+  if (!dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
+  if (taps < 1 || H < 1 || (taps > 1 && !state)) return NV_ERR_BAD_SIZE;
+  if (T == 0) return NV_OK;
+  ConvArgs a = {h, w, row_entry, cu_rows, entry_slot, state, slot_stride, out, out_dt, T, H, taps, T > 512 ? 8 : 1, update};
+  const bool vec = H % 4 == 0 && slot_stride % 4 == 0 && !((uintptr_t)h & 15) && !((uintptr_t)w & 15) && !((uintptr_t)state & 15)
+                   && !((uintptr_t)out & 15);
+  const int chunks = vec ? H / 4 : H;
+  const int threads = chunks < 256 ? (chunks + 31) / 32 * 32 : 256;
+  const dim3 grid((T + a.rows - 1) / a.rows, (chunks + threads - 1) / threads);
+#define NV_CONV(VEC, TAPS) NV_RETURN_IF(launch_dep(causal_conv_add_kernel<VEC, TAPS>, grid, dim3(threads), 0, s, a))
+#define NV_CONV_TAPS(VEC)            \
+  switch (taps) {                    \
+    case 2: NV_CONV(VEC, 2); break;  \
+    case 3: NV_CONV(VEC, 3); break;  \
+    case 4: NV_CONV(VEC, 4); break;  \
+    default: NV_CONV(VEC, 0); break; \
+  }
+  if (vec) { NV_CONV_TAPS(4) } else { NV_CONV_TAPS(1) }
+#undef NV_CONV_TAPS
+#undef NV_CONV
+  NV_RETURN_LAST();
+}
+
+// out: [T, half] pairs (cosine, sine) of position * inv_freq.
+NV_API int nv_rotary_table(const int* positions, const float* inv_freq, int half, float* out, int T, cudaStream_t s) {
+  const long long n = (long long)T * half;
+  if (half < 0) return NV_ERR_BAD_SIZE;
+  if (n == 0) return NV_OK;
+  NV_RETURN_IF(launch_dep(rotary_table_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, positions, inv_freq, half,
+                          (float2*)out, n));
+  NV_RETURN_LAST();
+}
+
+NV_API int nv_retention_chunk_rows() { return RC; }
+
+// what 0: the form for entries of one row; 1: the chunked form; 2: the scan.
+NV_API int nv_retention_usable(int what, int dk, int dv) {
+  if (dk < 1 || dv < 1) return 0;
+  if (what == 0) {
+    const int groups = dv / step_vec(dv);
+    return groups <= RT_THREADS && sizeof(float) * (2 * (size_t)dk + (size_t)(RT_THREADS / groups) * dv) <= 200 * 1024;
+  }
+  if (what == 1) return dk <= 256 && dv <= 256;
+  return sizeof(float) * ((size_t)dk * 32 + 2 * (size_t)dk + RT_THREADS) <= 200 * 1024;
+}
+
+// One launch (what 0), or the launches of the chunked form (what 1: `chunks` holds max_chunks * H * dk * dv words) or of
+// the scan (what 2: `raw` [T, H, dv]).  Entries with fewer than `min_rows` rows are skipped by what 1 and 2; what 0 takes
+// the `R` batch rows in `rows` (nullptr: rows 0 .. R - 1), each an entry of its own.  Everything is float32 but `out`.
+NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k0, int v0, int g0, const float* table,
+                        const int* positions, const float* inv_freq, int half, const int* row_entry, const int* cu_rows,
+                        const int* entry_slot, int num_entries, const int* rows, int R, float* S, long long S_stride,
+                        const float* powers, float k_scale, float eps, void* out, int out_dt, float* raw, void* chunks,
+                        int max_chunks, int T, int H, int dk, int dv, int min_rows, cudaStream_t s) {
+  if (!dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
+  if (H < 1 || half < 0 || 2 * half > dk || num_entries < 0) return NV_ERR_BAD_SIZE;
+  if (!nv_retention_usable(what, dk, dv)) return NV_ERR_UNSUPPORTED;
+  if (T == 0 || num_entries == 0) return NV_OK;
+  RetArgs a = {};
+  a.proj = proj; a.ld = ld; a.q0 = q0; a.k0 = k0; a.v0 = v0; a.g0 = g0; a.table = (const float2*)table;
+  a.positions = positions; a.inv_freq = inv_freq; a.half = half; a.row_entry = row_entry; a.cu_rows = cu_rows;
+  a.entry_slot = entry_slot; a.rows = rows; a.S = S; a.S_stride = S_stride; a.powers = powers; a.k_scale = k_scale;
+  a.eps = eps; a.out = out; a.raw = raw; a.chunks = (uint32_t*)chunks; a.out_dt = out_dt; a.H = H; a.dk = dk; a.dv = dv;
+  a.num_entries = num_entries; a.min_rows = min_rows;
+  if (what == 0) {
+    if (R == 0) return NV_OK;
+    const bool vec = step_vec(dv) == 4 && S_stride % 4 == 0 && !((uintptr_t)S & 15);
+    const int groups = vec ? dv / 4 : dv;
+    if (groups > RT_THREADS) return NV_ERR_UNSUPPORTED;
+    const size_t smem = sizeof(float) * (2 * (size_t)dk + (size_t)(RT_THREADS / groups) * dv);
+    int rc = vec ? allow(retention_step_kernel<4>, smem) : allow(retention_step_kernel<1>, smem);
+    if (rc) return rc;
+    if (vec) NV_RETURN_IF(launch_dep(retention_step_kernel<4>, dim3(R, H), dim3(RT_THREADS), smem, s, a));
+    else NV_RETURN_IF(launch_dep(retention_step_kernel<1>, dim3(R, H), dim3(RT_THREADS), smem, s, a));
+    NV_RETURN_LAST();
+  }
+  if (half > 0 && !table) return NV_ERR_BAD_SIZE;
+  if (what == 1) {
+    if (!chunks || max_chunks < 1) return NV_ERR_BAD_SIZE;
+    a.v2 = (half % 2 == 0 && dk % 2 == 0 && dv % 2 == 0 && ld % 2 == 0 && q0 % 2 == 0 && k0 % 2 == 0 && v0 % 2 == 0 &&
+            g0 % 2 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)table & 15) && !((uintptr_t)chunks & 15) &&
+            !((uintptr_t)out & 15)) ? 1 : 0;
+    if (dk <= 64) return launch_chunks_ns<64>(a, max_chunks, s);
+    if (dk <= 128) return launch_chunks_ns<128>(a, max_chunks, s);
+    return launch_chunks_ns<256>(a, max_chunks, s);
+  }
+  if (!raw) return NV_ERR_BAD_SIZE;
+  a.slice = 32;
+  const size_t smem = sizeof(float) * ((size_t)dk * a.slice + 2 * (size_t)dk + RT_THREADS);
+  int rc = allow(retention_scan_kernel, smem);
+  if (rc) return rc;
+  retention_scan_kernel<<<dim3(num_entries, H, (dv + a.slice - 1) / a.slice), RT_THREADS, smem, s>>>(a);
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) return (int)e;
+  const long long items = (long long)T * H;
+  retention_finish_kernel<<<(unsigned)((items + 7) / 8), 256, 0, s>>>(a, T);
+  NV_RETURN_LAST();
+}

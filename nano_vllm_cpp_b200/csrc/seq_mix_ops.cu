@@ -491,7 +491,9 @@ struct QkArgs {
   int rot0;                 // the turned elements are rot0 .. rot0 + rot_dim - 1 of a head
   int k_norm_dim;           // key heads: the norm is taken over (and applied to) the first so many elements; 0: all D
   int norm_mode;            // bit 0: q and k heads are normed also without a weight (the weight is then one);
-                            // bit 1: after the turn instead of before it
+                            // bit 1: after the turn instead of before it; bit 2: over all q heads at once, and all k
+                            // heads at once, instead of head by head (before the turn; qw / kw then have an entry per
+                            // element of all heads)
   const float* v_inv_freq;  // values are turned too: the first v_rot_dim elements of every value head, in pairs
   int v_rot_dim;            // (i, i + v_rot_dim / 2), by position * v_inv_freq[i]; 0: values are stored as projected
 };
@@ -514,10 +516,33 @@ __global__ void __launch_bounds__(QK_THREADS) qk_prepare_store_kernel(QkArgs a) 
   }
   const size_t slot = (size_t)(pos % a.page);
   const int heads = a.Hq + (write_kv ? a.Hkv : 0);
+  const bool whole = (a.norm_mode & 4) != 0;
+  __shared__ float part[2][QK_THREADS / 32];
+  float whole_q = 0.f, whole_k = 0.f;
+  if (whole) {                       // 1 / rms of all q elements, and of all k elements, of the row
+#pragma unroll
+    for (int side = 0; side < 2; ++side) {
+      const int n = side == 0 ? a.Hq * D : (write_kv ? a.Hkv * D : 0);
+      const size_t src = (size_t)t * a.ld + (side == 0 ? a.q0 : a.k0);
+      float ss = 0.f;
+      for (int i = threadIdx.x; i < n; i += QK_THREADS) {
+        const float x = ld_dt(a.in, a.in_dt, src + i);
+        ss = fmaf(x, x, ss);
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) part[side][warp] = ss;
+    }
+    __syncthreads();
+    float sq = 0.f, sk = 0.f;
+    for (int i = 0; i < QK_THREADS / 32; ++i) { sq += part[0][i]; sk += part[1][i]; }
+    whole_q = rsqrtf(sq / (float)max(1, a.Hq * D) + a.eps);
+    whole_k = rsqrtf(sk / (float)max(1, a.Hkv * D) + a.eps);
+  }
   for (int h = warp; h < heads; h += QK_THREADS / 32) {
     const bool is_q = h < a.Hq;
     const size_t src = (size_t)t * a.ld + (is_q ? a.q0 + h * D : a.k0 + (h - a.Hq) * D);
     const float* w = is_q ? a.qw : a.kw;
+    if (whole && w) w += (is_q ? h : h - a.Hq) * D;
     const int nd = (!is_q && a.k_norm_dim > 0) ? a.k_norm_dim : D;     // what the norm covers
     const bool normed = w != nullptr || (a.norm_mode & 1);
     const bool after = (a.norm_mode & 2) != 0;
@@ -529,7 +554,7 @@ __global__ void __launch_bounds__(QK_THREADS) qk_prepare_store_kernel(QkArgs a) 
     }
     if (normed && !after) {
       ss = warp_sum(ss);
-      const float r = rsqrtf(ss / (float)nd + a.eps);
+      const float r = whole ? (is_q ? whole_q : whole_k) : rsqrtf(ss / (float)nd + a.eps);
       for (int i = lane; i < nd; i += 32) buf[i] = buf[i] * r * (w ? w[i] : 1.f);
     }
     __syncwarp();
@@ -594,7 +619,7 @@ __global__ void __launch_bounds__(ATTG_THREADS) paged_attention_general_kernel(
     const int* __restrict__ block_table, int max_blocks, const int* __restrict__ row_entry,
     const int* __restrict__ positions, float scale, int window, int keep_first, int has_sink, float sink_score,
     const float* __restrict__ sinks, void* __restrict__ out, int out_dt, int Hq, int Hkv, int Hv, int D, int Dv,
-    int KS, int page, float softcap) {
+    int KS, int page, float softcap, HeadGate gate) {
   extern __shared__ float qs[];      // KS * D
   __shared__ float p[ATTG_THREADS];
   __shared__ int pslot[ATTG_THREADS];
@@ -662,7 +687,7 @@ __global__ void __launch_bounds__(ATTG_THREADS) paged_attention_general_kernel(
     }
     __syncthreads();
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? head_gate_of(gate, t, h) / l : 0.f;
   const size_t ob = (size_t)t * Hq * Dv + (size_t)h * Dv;
 #pragma unroll
   for (int u = 0; u < ATTG_NV; ++u) {
@@ -1356,7 +1381,8 @@ NV_API int nv_qk_prepare_store(const void* in, int in_dt, long long ld, int q0, 
                                int norm_mode, cudaStream_t s) {
   if (!dt_ok(in_dt) || !dt_ok(q_dt) || !dt_ok(cache_dt)) return NV_ERR_BAD_DTYPE;
   if (rot_dim < 0 || rot0 < 0 || rot0 + rot_dim > D || rot_dim % 2 || D <= 0 || Dv <= 0) return NV_ERR_BAD_SIZE;
-  if (k_norm_dim < 0 || k_norm_dim > D || norm_mode < 0 || norm_mode > 3) return NV_ERR_BAD_SIZE;
+  if (k_norm_dim < 0 || k_norm_dim > D || norm_mode < 0 || norm_mode > 7) return NV_ERR_BAD_SIZE;
+  if ((norm_mode & 4) && ((norm_mode & 2) || k_norm_dim > 0)) return NV_ERR_UNSUPPORTED;
   if (v_rot_dim < 0 || v_rot_dim > Dv || v_rot_dim % 2 || (v_rot_dim && !v_inv_freq)) return NV_ERR_BAD_SIZE;
   if (QP < D || KP < D || VP < Dv) return NV_ERR_BAD_SIZE;
   if (T == 0) return NV_OK;
@@ -1375,7 +1401,7 @@ NV_API int nv_paged_attention_general(const void* q, int q_dt, const void* kc, c
                                       const int* positions, float scale, int window, int keep_first, int has_sink,
                                       float sink_score, const float* sinks, void* out, int out_dt, int T, int Hq,
                                       int Hkv, int Hv, int D, int Dv, int key_span, int page, float softcap,
-                                      cudaStream_t s) {
+                                      const float* gate, long long gate_ld, cudaStream_t s) {
   if (!dt_ok(q_dt) || !dt_ok(cache_dt) || !dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
   if (D <= 0 || Dv <= 0 || Dv > ATTG_NV * ATTG_THREADS || Hkv <= 0 || Hv <= 0 || Hq % Hv || keep_first < 0)
     return NV_ERR_UNSUPPORTED;
@@ -1386,7 +1412,7 @@ NV_API int nv_paged_attention_general(const void* q, int q_dt, const void* kc, c
   if (rc) return rc;
   paged_attention_general_kernel<<<dim3(T, Hq), ATTG_THREADS, smem, s>>>(
       q, q_dt, kc, vc, cache_dt, block_table, max_blocks, row_entry, positions, scale, window, keep_first, has_sink,
-      sink_score, sinks, out, out_dt, Hq, Hkv, Hv, D, Dv, key_span, page, softcap);
+      sink_score, sinks, out, out_dt, Hq, Hkv, Hv, D, Dv, key_span, page, softcap, HeadGate{gate, gate_ld});
   NV_RETURN_LAST();
 }
 

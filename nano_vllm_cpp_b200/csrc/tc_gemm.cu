@@ -144,6 +144,12 @@ __device__ __forceinline__ void chunk_act(float (&g)[W], float (&u)[W], float p0
   }
 }
 
+template <int W, int PAIR>
+__device__ __forceinline__ void chunk_pair(float (&g)[W], const float (&u)[W], float p0, float p1) {
+#pragma unroll
+  for (int j = 0; j < W; ++j) g[j] = pair_mul(PAIR, g[j], u[j], p0, p1);
+}
+
 template <int W>
 __device__ __forceinline__ void epilogue_chunk(const TcArgs& a, const Tile& t, int two, uint32_t taddr, int c0, int n,
                                                int n2, bool n_ok, bool n2_ok, float bias, float bias2) {
@@ -196,8 +202,9 @@ __device__ __forceinline__ void epilogue_chunk(const TcArgs& a, const Tile& t, i
     return;
   }
   if (a.swiglu) {
-#pragma unroll
-    for (int j = 0; j < W; ++j) g[j] = pair_mul(a.swiglu, g[j], u[j], a.act_p0, a.act_p1);
+    if (a.swiglu == NV_EPI_SWIGLU) chunk_pair<W, NV_EPI_SWIGLU>(g, u, a.act_p0, a.act_p1);
+    else if (a.swiglu == NV_EPI_GLU_CLAMPED) chunk_pair<W, NV_EPI_GLU_CLAMPED>(g, u, a.act_p0, a.act_p1);
+    else chunk_pair<W, NV_EPI_GEGLU_TANH>(g, u, a.act_p0, a.act_p1);
   }
 #pragma unroll
   for (int j = 0; j < W; ++j) {

@@ -50,10 +50,16 @@ class PagedAttention(Mixer):
     ``score_softcap * tanh(s / score_softcap)`` before mask and softmax.  ``round_weights``: a bfloat16 run of
     this path rounds the softmax weights (computed in float32) to bfloat16 for their product with the values, as it
     rounds every other operand of a product, instead of taking them in as three bfloat16 terms.
+
+    Three more, of the same path.  ``qk_norm_whole``: q's norm is taken over all its heads at once, k's over all of its
+    heads (weights of that size), instead of head by head.  ``output_gate``: head h's output is multiplied by
+    ``sigmoid(Wg h)_h``, one number per head and row (tensor ``g`` [heads, hidden]), where the attention kernel writes
+    it.  ``own_kv`` False: the layer has no k and v tensors; its call reads the pages of an earlier call (whose kv heads
+    and head sizes are the same) with its own queries, and writes none.
     """
 
     _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
-              "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias",
+              "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias", "g": "g_proj.weight",
               "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "head_mix": "head_mix", "sink": "sink"}
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, bias: bool,
@@ -62,7 +68,8 @@ class PagedAttention(Mixer):
                  names: dict | None = None, values_from_keys: bool = False, exact_weights: bool = False,
                  keep_first: int = 0, learned_sink: bool = False, head_mix: bool = False,
                  value_position: PartSpec | None = None, qk_norm_weight: bool = True,
-                 qk_norm_after_rotation: bool = False, score_softcap: float = 0.0, round_weights: bool = False):
+                 qk_norm_after_rotation: bool = False, score_softcap: float = 0.0, round_weights: bool = False,
+                 qk_norm_whole: bool = False, output_gate: bool = False, own_kv: bool = True):
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
         self.hidden, self.Hq, self.Hkv, self.D = hidden_size, num_heads, num_kv_heads, head_dim
@@ -96,11 +103,19 @@ class PagedAttention(Mixer):
             if self.values_from_keys or vp.pairing != "halves" or vp.amplitude != 1.0 or vp.rotary_dim > self.Dv:
                 raise ValueError("turned values: pairs (i, i + dims / 2) over at most the value head, no amplitude, and "
                                  "values of their own")
+        self.qk_norm_whole, self.output_gate, self.own_kv = bool(qk_norm_whole), bool(output_gate), bool(own_kv)
+        if self.qk_norm_whole and (self.qk_norm_eps is None or self.qk_norm_after):
+            raise ValueError("a norm over all heads comes with its eps and precedes the turn")
+        if not self.own_kv and (bias or self.values_from_keys):
+            raise ValueError("a layer without keys and values of its own has no biases of theirs")
         # the options that only the general kernels know, whatever the dtype
         self.extended = bool(self.keep_first or self.learned_sink or self.head_mix or self.value_position is not None)
         if self.extended and self.softcap > 0:
             raise ValueError("capped scores are not supported together with kept positions, learned sinks, mixed heads or turned values")
-        self.general = (self.extended or self.softcap > 0 or self.values_from_keys or bool(exact_weights) or self.Dv != self.D or self.qk_norm_eps is not None or self.sink_score is not None
+        if self.extended and (self.qk_norm_whole or self.output_gate or not self.own_kv):
+            raise ValueError("a norm over all heads, an output gate and borrowed keys are not supported together with kept "
+                             "positions, learned sinks, mixed heads or turned values")
+        self.general = (self.extended or self.output_gate or not self.own_kv or self.softcap > 0 or self.values_from_keys or bool(exact_weights) or self.Dv != self.D or self.qk_norm_eps is not None or self.sink_score is not None
                         or self.position.pairing != "halves" or self.position.amplitude != 1.0)
         if self.general:
             if self.extended:
@@ -120,14 +135,20 @@ class PagedAttention(Mixer):
              n["v"]: TensorSpec((vv, H)), n["o"]: TensorSpec((H, self.Hq * self.Dv))}
         if self.values_from_keys:
             del s[n["v"]]
+        if not self.own_kv:
+            del s[n["k"]], s[n["v"]]
+        if self.output_gate:
+            s[n["g"]] = TensorSpec((self.Hq, H))
         if self.bias:
             s.update({n["q_bias"]: TensorSpec((q,), kind="vector"), n["k_bias"]: TensorSpec((kv,), kind="vector"),
                       n["v_bias"]: TensorSpec((vv,), kind="vector")})
         if self.out_bias:
             s[n["o_bias"]] = TensorSpec((H,), kind="vector")
         if self.qk_norm_eps is not None and self.qk_norm_weight:
-            s[n["q_norm"]] = TensorSpec((self.D,), init="ones", kind="vector")
-            s[n["k_norm"]] = TensorSpec((self.D,), init="ones", kind="vector")
+            whole = self.qk_norm_whole
+            s[n["q_norm"]] = TensorSpec((q if whole else self.D,), init="ones", kind="vector")
+            if self.own_kv:
+                s[n["k_norm"]] = TensorSpec((kv if whole else self.D,), init="ones", kind="vector")
         if self.head_mix:
             s[n["head_mix"]] = TensorSpec((self.Hq, self.Hq), init="identity", kind="vector")
         if self.learned_sink:
@@ -140,7 +161,13 @@ class PagedAttention(Mixer):
         n = self.names
         self.position.load(fetch, ctx)
         # q, k and v rows are stacked so that one product makes all three (src/model.cpp:508-513)
-        self.qkv_weight = _cat([fetch(n["q"]), fetch(n["k"])] + ([] if self.values_from_keys else [fetch(n["v"])]))
+        rows = [fetch(n["q"])]
+        if self.own_kv:
+            rows += [fetch(n["k"])] + ([] if self.values_from_keys else [fetch(n["v"])])
+        self.gate_col = sum(t.shape[0] for t in rows)                    # the output gates' rows come last
+        if self.output_gate:
+            rows.append(fetch(n["g"]))
+        self.qkv_weight = _cat(rows)
         self.qkv_bias = None
         if self.bias:
             self.qkv_bias = _cat([fetch(n["q_bias"]), fetch(n["k_bias"]), fetch(n["v_bias"])])
@@ -163,7 +190,7 @@ class PagedAttention(Mixer):
                 self.o_weight = w.view(self.hidden, self.Hq * self.pad)
         self.q_norm = self.k_norm = None
         if self.qk_norm_eps is not None and self.qk_norm_weight:
-            self.q_norm, self.k_norm = fetch(n["q_norm"]), fetch(n["k_norm"])
+            self.q_norm, self.k_norm = fetch(n["q_norm"]), fetch(n["k_norm"]) if self.own_kv else None
 
     def cache_spec(self):
         if getattr(self, "pad", 0):
@@ -200,9 +227,11 @@ class PagedAttention(Mixer):
         # (values that are the keys are read where the keys are, as projected: the kernel norms and turns its own copy)
         ops.qk_prepare_store(proj, 0, Hq * D, Hq * D if self.values_from_keys else (Hq + Hkv) * D, batch.positions, batch.row_entry, bt, self.q_norm,
                              self.k_norm, self.qk_norm_eps or 0.0, pos.inv_freq(), pos.rotary_dim,
-                             pos.pairing == "interleaved", pos.amplitude, q, cache.k, cache.v, Hq, Hkv, D, Dv,
-                             cache.write, ctx.err, norm_always=self.qk_norm_eps is not None,
-                             norm_after=self.qk_norm_after)
+                             pos.pairing == "interleaved", pos.amplitude, q, cache.k, cache.v, Hq,
+                             Hkv if self.own_kv else 0, D, Dv, cache.write and self.own_kv, ctx.err,
+                             norm_always=self.qk_norm_eps is not None, norm_after=self.qk_norm_after,
+                             norm_whole=self.qk_norm_whole)
+        gate = proj[:, self.gate_col:self.gate_col + Hq] if self.output_gate else None
         att = torch.empty((T, Hq * (P or Dv)), dtype=ctx.act_dtype, device=h.device)
         if P:
             # Entries of one row go to the split-key decode kernel (with weights that keep their float32 bits), the
@@ -215,17 +244,18 @@ class PagedAttention(Mixer):
                                      att, Hq, Hkv, P, batch.max_context if batch.decode_only else batch.max_single_context,
                                      rows=None if batch.decode_only else batch.single_rows, err=ctx.err,
                                      sink_score=self.sink_score, float_weights=self.weight_terms == 3,
-                                     softcap=self.softcap)
+                                     softcap=self.softcap, gate=gate)
             if single < batch.S:
                 tiles = (batch.T - single) // ops.attention_prefill_tile_rows() + (batch.S - single)
                 ops.attention_prefill(q, cache.k, cache.v, bt, batch.cu_rows, batch.entry_pos0, tiles, self.scale,
                                       self.window, att, Hq, Hkv, P, err=ctx.err, min_rows=2 if single else 1,
                                       kernel="mma" if self.sink_score is not None and self.weight_terms == 3 else "auto",
-                                      sink_score=self.sink_score, weight_terms=self.weight_terms, softcap=self.softcap)
+                                      sink_score=self.sink_score, weight_terms=self.weight_terms, softcap=self.softcap,
+                                      gate=gate)
         else:
             ops.paged_attention_general(q, cache.k, cache.v, bt, batch.row_entry, batch.positions, self.scale,
                                         self.window, att, Hq, Hkv, D, Dv, sink_score=self.sink_score,
-                                        softcap=self.softcap)
+                                        softcap=self.softcap, gate=gate)
         return linear(ctx, att, self.o_weight, torch.float32, bias=self.o_bias)
 
     def _forward_extended(self, proj, bt, batch, cache):

@@ -14,6 +14,8 @@ part                 what it must provide
 ``Mixer``            ``cache_spec()``: what it keeps per request (pages of keys and values, a
                      fixed-size state, or nothing); ``forward(h, batch, cache)`` -> float32
                      ``[T, hidden]`` branch output
+``InputFilter``      between a norm and its mixer: ``forward(h32, batch, cache)`` -> rows for the mixer;
+                     ``cache_spec()`` as a mixer's
 ``FeedForward``      ``wants_f32_input``; ``forward(h, h32, batch)`` -> float32 ``[T, hidden]``
 ===================  =======================================================================
 
@@ -64,6 +66,14 @@ class StateCacheSpec:
     the step that runs the request's first token."""
     shape: tuple
     dtype: torch.dtype = torch.float32
+
+
+@dataclass(frozen=True)
+class SharedCacheSpec:
+    """What an earlier call of the model's order keeps, read and never written: the call's cache entry, or with ``part``
+    that part of it if the entry is a composite.  It takes no memory of its own."""
+    call: int
+    part: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -207,6 +217,17 @@ class Mixer(Part):
         return None
 
     def forward(self, h, batch, cache):
+        raise NotImplementedError
+
+
+class InputFilter(Part):
+    """Changes what a mixer reads, row by row, from the request's own earlier rows.  ``forward(h32, batch, cache)``: the
+    normed rows in float32 -> rows in the activation dtype; ``cache``: the filter's own view (None if it keeps nothing)."""
+
+    def cache_spec(self):
+        return None
+
+    def forward(self, h32, batch, cache):
         raise NotImplementedError
 
 

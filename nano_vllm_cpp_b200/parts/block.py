@@ -14,7 +14,7 @@ feed-forward, a post-norm block) declares its own slots and is registered like a
 """
 from __future__ import annotations
 
-from .base import PartSpec, StreamRows, BranchSum, NormedBranch, resolve_branch
+from .base import PartSpec, CompositeCacheSpec, SharedCacheSpec, StreamRows, BranchSum, NormedBranch, resolve_branch
 from .registry import register_part, build_part
 
 _DEFAULT_NAMES = {"norm1": "input_layernorm.", "mixer": "self_attn.", "norm2": "post_attention_layernorm.",
@@ -72,7 +72,30 @@ class Arrangement:
         return [(self.spec.prefix(slot), getattr(self, slot)) for slot in self.slots if getattr(self, slot) is not None]
 
     def cache_spec(self):
-        return getattr(self, self.cache_slot).cache_spec() if self.cache_slot else None
+        spec = getattr(self, self.cache_slot).cache_spec() if self.cache_slot else None
+        own = self._filter_spec()
+        return spec if own is None else CompositeCacheSpec((spec, own))
+
+    def borrowing_cache_spec(self, call: int):
+        """What the layer keeps where its mixer reads an earlier call's entry (``LayerCall.cache_of``): that entry, or,
+        if it has an input filter with a state, the mixer's part of that entry beside a state of its own."""
+        own = self._filter_spec()
+        return ("shared", call) if own is None else CompositeCacheSpec((SharedCacheSpec(call, 0), own))
+
+    def _filter_spec(self):
+        f = getattr(self, "input_filter", None)
+        return f.cache_spec() if f is not None else None
+
+    def mixer_input(self, norm, batch, cache):
+        """``norm(want_f32, want_rows)`` makes the mixer's rows; with an input filter they pass it.  Returns the rows and
+        the mixer's own cache view."""
+        f = getattr(self, "input_filter", None)
+        if f is None:
+            return norm(False, True)[0], cache
+        _, h32 = norm(True, False)
+        if f.cache_spec() is None:
+            return f.forward(h32, batch, None), cache
+        return f.forward(h32, batch, cache.parts[1]), cache.parts[0]
 
     def forward(self, x, pending, batch, cache):
         raise NotImplementedError
@@ -83,12 +106,16 @@ class PreNormBlock(Arrangement):
 
     The sum into the residual stream is fused with the next norm: a block hands its last branch
     output on as ``pending`` instead of adding it, and every norm adds what is pending first —
-    the reference's ``rms_norm_add`` convention (src/hip_ops.hip:395-417).
+    the reference's ``rms_norm_add`` convention (src/hip_ops.hip:395-417).  With an ``input_filter`` the mixer reads
+    ``filter(norm1(x))``.
     """
-    slots = {"norm1": "norm", "mixer": "mixer", "norm2": "norm", "feed_forward": "feed_forward"}
+    slots = {"norm1": "norm", "input_filter": "input_filter", "mixer": "mixer", "norm2": "norm",
+             "feed_forward": "feed_forward"}
+    optional = ("input_filter",)
 
     def forward(self, x, pending, batch, cache):
-        h, _ = self.norm1.forward(x, resolve_branch(self.norm1, pending))
+        h, cache = self.mixer_input(lambda f32, rows: self.norm1.forward(x, resolve_branch(self.norm1, pending), want_f32=f32),
+                                    batch, cache)
         pending = self.mixer.forward(h, batch, cache)
         h, h32 = self.norm2.forward(x, resolve_branch(self.norm2, pending), want_f32=self.feed_forward.wants_f32_input)
         pending = self.feed_forward.forward(h, h32, batch)

@@ -24,16 +24,21 @@ class DenseSwiGLU(FeedForward):
 
     ``clamp_limit`` > 0 makes the pairing of the two halves a clamped one instead, still in the first product's
     epilogue: ``g = min(gate(h), limit)``, ``u = clamp(up(h), -limit, limit)``, ``down(g sigmoid(slope g) (u + 1))``.
+    ``activation="gelu_tanh"``: ``down(gelu_tanh(gate(h)) * up(h))``, in the same epilogue.
     ``names`` renames the tensors (keys: gate, up, down)."""
 
     _NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
 
     def __init__(self, hidden_size: int, intermediate_size: int, clamp_limit: float = 0.0, slope: float = 1.702,
-                 names: dict | None = None):
+                 names: dict | None = None, activation: str = "silu"):
         self.hidden, self.inter = hidden_size, intermediate_size
         if clamp_limit < 0:
             raise ValueError("clamp_limit must not be negative")
-        self.pair = ("glu_clamped", float(clamp_limit), float(slope)) if clamp_limit > 0 else None
+        if activation not in ("silu", "gelu_tanh") or (activation != "silu" and clamp_limit > 0):
+            raise ValueError("the gate's activation is silu or gelu_tanh, and a clamped pairing has its own")
+        self.pair = "geglu_tanh" if activation == "gelu_tanh" else None
+        if clamp_limit > 0:
+            self.pair = ("glu_clamped", float(clamp_limit), float(slope))
         self.names = dict(self._NAMES, **(names or {}))
 
     def tensor_specs(self, available=None):
@@ -112,8 +117,10 @@ class SparseMoeSwiGLU(FeedForward):
     Other routers are options.  ``score="sigmoid"``: every expert's score is ``s = sigmoid(r)`` by itself, in
     float32; the ``top_k`` largest ``s + correction`` are chosen (``choice_bias``: a learned vector ``correction``
     [experts] that steers the choice only), and the weights are the chosen experts' ``s`` without it.  ``route_scale``
-    multiplies the weights.  ``shared_gate=False``: the shared expert has no gate and is added as it is.  ``names``
-    gives the tensors' names where they are not the usual ones (keys: router, correction, shared_gate, and the
+    multiplies the weights.  ``router_bias`` (softmax scores): a learned vector ``router_bias`` [experts] is added to the
+    logits before the softmax; with ``renormalize`` the weights are then the softmax over the chosen biased logits.
+    ``shared_gate=False``: the shared expert has no gate and is added as it is.  ``names``
+    gives the tensors' names where they are not the usual ones (keys: router, router_bias, correction, shared_gate, and the
     patterns expert_gate, expert_up, expert_down with ``{}`` for the expert's number, shared_gate_proj, shared_up,
     shared_down).
 
@@ -122,7 +129,7 @@ class SparseMoeSwiGLU(FeedForward):
     """
     wants_f32_input = True
 
-    _NAMES = {"router": "gate.weight", "correction": "correction", "shared_gate": "shared_expert_gate.weight",
+    _NAMES = {"router": "gate.weight", "router_bias": "gate.bias", "correction": "correction", "shared_gate": "shared_expert_gate.weight",
               "expert_gate": "experts.{}.gate_proj.weight", "expert_up": "experts.{}.up_proj.weight",
               "expert_down": "experts.{}.down_proj.weight", "shared_gate_proj": "shared_expert.gate_proj.weight",
               "shared_up": "shared_expert.up_proj.weight", "shared_down": "shared_expert.down_proj.weight"}
@@ -130,7 +137,7 @@ class SparseMoeSwiGLU(FeedForward):
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, intermediate_size: int,
                  shared_intermediate_size: int = 0, renormalize: bool = False, score: str = "softmax",
                  route_scale: float = 1.0, choice_bias: bool = False, shared_gate: bool = True,
-                 names: dict | None = None, expert_activation: str | None = None):
+                 names: dict | None = None, expert_activation: str | None = None, router_bias: bool = False):
         if not (1 <= top_k <= num_experts):
             raise ValueError("top_k must lie in 1..num_experts")
         if top_k > 32 or num_experts > 1536:
@@ -141,6 +148,9 @@ class SparseMoeSwiGLU(FeedForward):
             raise ValueError(f"score must be one of {sorted(ops.ROUTE_SCORES)}, found {score!r}")
         if choice_bias and score != "sigmoid":
             raise ValueError("a choice bias goes with sigmoid scores")
+        if router_bias and score != "softmax":
+            raise ValueError("a bias on the router's logits goes with softmax scores")
+        self.router_bias = bool(router_bias)
         self.score, self.route_scale, self.choice_bias = score, float(route_scale), bool(choice_bias)
         self.shared_gate = bool(shared_gate) and shared_intermediate_size > 0
         if expert_activation is not None and expert_activation not in ops.EPILOGUE_ACTS:
@@ -162,6 +172,8 @@ class SparseMoeSwiGLU(FeedForward):
         s = {n["router"]: TensorSpec((E, H))}
         if self.choice_bias:
             s[n["correction"]] = TensorSpec((E,), init="zeros", kind="vector")
+        if self.router_bias:
+            s[n["router_bias"]] = TensorSpec((E,), init="zeros", kind="vector")
         if self.gated and available is not None and available("experts.gate_up_proj"):  # stacked form, src/model.cpp:274-281
             s["experts.gate_up_proj"] = TensorSpec((E, 2 * I, H))
             s["experts.down_proj"] = TensorSpec((E, H, I))
@@ -185,6 +197,8 @@ class SparseMoeSwiGLU(FeedForward):
         H, I, E, SI, n = self.hidden, self.inter, self.E, self.shared_inter, self.names
         self.router = fetch(n["router"])
         bias = fetch(n["correction"]).float().contiguous() if self.choice_bias else None
+        if self.router_bias:
+            bias = fetch(n["router_bias"]).float().contiguous()
         if self.score != "softmax" or bias is not None or self.route_scale != 1.0:
             self.rule = (self.score, bias, self.route_scale)
         stacked = self.gated and fetch.has("experts.gate_up_proj")

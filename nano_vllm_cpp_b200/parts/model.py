@@ -121,11 +121,12 @@ class Model:
         return out
 
     def cache_specs(self) -> list:
-        """One entry per call: the cache spec of its mixer, or None, or ('shared', j)."""
+        """One entry per call: the cache spec of its layer, or None, or ('shared', j); a call that reads an earlier
+        call's entry and keeps a state of its own beside it has a composite with a ``SharedCacheSpec``."""
         out = []
         for c in self.calls:
             if c.cache_of is not None:
-                out.append(("shared", c.cache_of))
+                out.append(self.layers[c.layer].borrowing_cache_spec(c.cache_of))
             else:
                 out.append(self.layers[c.layer].cache_spec())
         return out

@@ -49,6 +49,13 @@ class RMSNorm(Norm):
                                 branch_weights=branch_weights, mix_scale=mix_scale)
         return out
 
+    def read_streams(self, x, streams: int, branch, carry, write, read, want_f32: bool = False, want_rows: bool = True):
+        """The same norm for a model that keeps several copies of its stream (``parts.streams``): ``x`` [T, streams * size]
+        is brought up to date in place with ``branch`` (a float32 matrix, a ``RowMix`` or None) through ``carry`` and
+        ``write``, then read with ``read`` (None: the plain sum of the copies) and normed, in one launch."""
+        return _read_streams(("rms", self.weight, self.eps), self.size, self.ctx, x, streams, branch, carry, write, read,
+                             want_f32, want_rows)
+
     def forward(self, x, branch, want_f32=False):
         out = torch.empty(x.shape, dtype=self.ctx.act_dtype, device=x.device)
         out32 = None
@@ -76,6 +83,25 @@ class RMSNorm(Norm):
         return out, out32
 
 
+def _read_streams(norm, size, ctx, x, streams, branch, carry, write, read, want_f32, want_rows):
+    """One launch of ``ops.stream_mix_norm`` with that norm; returns (rows in the activation dtype or None, float32 rows
+    or None)."""
+    T, dev = x.shape[0], x.device
+    out = torch.empty((T, size), dtype=ctx.act_dtype, device=dev) if want_rows or ctx.act_dtype == torch.float32 else None
+    out32 = None
+    if want_f32:
+        out32 = out if out is not None and out.dtype == torch.float32 else torch.empty((T, size), dtype=torch.float32, device=dev)
+    mix = None
+    if isinstance(branch, RowMix):
+        if branch.gate_logit is None and branch.index.shape[1] <= ops.STREAM_MAX_MIX:
+            mix, branch = branch.as_tuple(), None
+        else:
+            branch = branch.sum()
+    ops.stream_mix_norm(x, streams, branch=branch, mix=mix, carry=carry, write=write, read=read, norm=norm, out=out,
+                        out32=None if out32 is out else out32)
+    return out, out32
+
+
 class DynamicTanh(Norm):
     """``y = tanh(alpha * x) * gain + shift``: a norm without mean or variance, every element by itself.  ``alpha`` is
     one number, ``gain`` and ``shift`` are vectors over the width; all three are learned and held in float32, and the
@@ -100,27 +126,12 @@ class DynamicTanh(Norm):
         self.shift = fetch(self.shift_name).float().contiguous()
         self.alpha = fetch(self.alpha_name).float().reshape(1).contiguous()
 
-    def _outputs(self, T, device, want_f32):
-        out = torch.empty((T, self.size), dtype=self.ctx.act_dtype, device=device)
-        out32 = None
-        if want_f32:
-            out32 = out if out.dtype == torch.float32 else torch.empty((T, self.size), dtype=torch.float32, device=device)
-        return out, out32
-
-    def read_streams(self, x, streams: int, branch, carry, write, read, want_f32: bool = False):
+    def read_streams(self, x, streams: int, branch, carry, write, read, want_f32: bool = False, want_rows: bool = True):
         """``x`` [T, streams * size]: the copies, brought up to date in place with ``branch`` (a float32 matrix, a
         ``RowMix`` or None) through ``carry`` and ``write``, then read with ``read`` (None: their plain sum) and
         normed.  Returns (rows in the activation dtype, float32 copy or None)."""
-        out, out32 = self._outputs(x.shape[0], x.device, want_f32)
-        mix = None
-        if isinstance(branch, RowMix):
-            if branch.gate_logit is None and branch.index.shape[1] <= ops.STREAM_MAX_MIX:
-                mix, branch = branch.as_tuple(), None
-            else:
-                branch = branch.sum()
-        ops.stream_mix_norm(x, streams, branch=branch, mix=mix, carry=carry, write=write, read=read,
-                            norm=(self.alpha, self.gain, self.shift), out=out, out32=None if out32 is out else out32)
-        return out, out32
+        return _read_streams((self.alpha, self.gain, self.shift), self.size, self.ctx, x, streams, branch, carry, write,
+                             read, want_f32, want_rows)
 
     def forward(self, x, branch, want_f32=False):
         return self.read_streams(x, 1, branch, None, None, None, want_f32)

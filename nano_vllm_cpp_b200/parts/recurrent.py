@@ -6,9 +6,9 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .base import Mixer, StateCacheSpec, CompositeCacheSpec, TensorSpec
+from .base import Mixer, StateCacheSpec, CompositeCacheSpec, TensorSpec, PartSpec
 from .linear import linear
-from .registry import register_part
+from .registry import register_part, build_part
 
 
 def _stack(parts: list, dtype_like=None):
@@ -221,6 +221,68 @@ class GatedDeltaRule(Mixer):
         return linear(ctx, y, self.w_out, torch.float32)
 
 
+class Retention(Mixer):
+    """Linear attention with one fixed decay per head and no softmax or denominator.
+
+    ``q, k, v = Wq h, Wk h, Wv h`` (``heads`` heads of ``dim``, ``dim`` and ``vdim`` elements); q and k heads are turned by
+    their positions (``position``: a rotary encoding in the halves pairing), then k is multiplied by ``dim^-1/2``.  Per
+    head with the constant d = ``decay[h]``:
+
+        S = d S + k v^T;   o = S^T q
+
+    Every head's ``o`` is divided by its root mean square (``eps``, no weight), the heads side by side are multiplied by
+    ``silu(Wg h)``, and ``Wo`` projects back.  State per request: S, in float32.  ``names`` renames the tensors (keys: q,
+    k, v, g, o)."""
+
+    _NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
+
+    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, decay: list, eps: float,
+                 position: PartSpec | None = None, names: dict | None = None):
+        if min(heads, dim, vdim) < 1 or len(decay) != heads:
+            raise ValueError("retention: every size must be positive, and there is one decay per head")
+        if dim > 1400:
+            raise ValueError(f"retention keys of {dim} elements are not supported: the scan kernel takes up to 1400")
+        self.hidden, self.H, self.dk, self.dv, self.eps = hidden_size, heads, dim, vdim, float(eps)
+        self.decay = [float(d) for d in decay]
+        self.position = build_part("position", position if position is not None else PartSpec("none"))
+        pos = self.position
+        if pos.rotary_dim > dim or (pos.rotary_dim and (pos.pairing != "halves" or pos.amplitude != 1.0
+                                                        or pos.rotation_positions(None) is not None)):
+            raise ValueError("retention: pairs (i, i + dims / 2) inside a head, turned by the row's place in its sequence")
+        self.names = dict(self._NAMES, **(names or {}))
+
+    def tensor_specs(self, available=None):
+        W, H, dk, dv, n = self.hidden, self.H, self.dk, self.dv, self.names
+        s = {n["q"]: TensorSpec((H * dk, W)), n["k"]: TensorSpec((H * dk, W)), n["v"]: TensorSpec((H * dv, W)),
+             n["g"]: TensorSpec((H * dv, W)), n["o"]: TensorSpec((W, H * dv))}
+        s.update(self.position.tensor_specs(available))
+        return s
+
+    def load(self, fetch, ctx):
+        self.ctx = ctx
+        H, dk, dv, n = self.H, self.dk, self.dv, self.names
+        self.position.load(fetch, ctx)
+        self.w_in = _stack([fetch(n["q"]), fetch(n["k"]), fetch(n["v"]), fetch(n["g"])])     # one float32 product
+        self.cols = {"q": 0, "k": H * dk, "v": 2 * H * dk, "g": 2 * H * dk + H * dv}
+        self.w_out = fetch(n["o"])
+        # d^0 .. d^64 per head, worked out in float64
+        d = torch.tensor(self.decay, dtype=torch.float64)[:, None]
+        e = torch.arange(ops.retention_chunk_rows() + 1, dtype=torch.float64)[None, :]
+        self.powers = torch.pow(d, e).float().to(ctx.device).contiguous()
+
+    def cache_spec(self):
+        return StateCacheSpec((self.H, self.dk, self.dv))
+
+    def forward(self, h, batch, cache):
+        ctx = self.ctx
+        proj = linear(ctx, h, self.w_in, torch.float32)
+        y = torch.empty((h.shape[0], self.H * self.dv), dtype=ctx.act_dtype, device=h.device)
+        # float32 runs keep one kernel however the work is cut; bfloat16 runs take the step and chunk forms
+        ops.retention(proj, self.cols, batch, cache.state, self.powers, self.position.inv_freq(), self.position.rotary_dim,
+                      self.H, self.dk, self.dv, self.eps, y, fast=ctx.fast_kernels and ctx.act_dtype == torch.bfloat16)
+        return linear(ctx, y, self.w_out, torch.float32)
+
+
 def ops_scan_size_ok(dk: int, dv: int, parts: int = 1) -> bool:
     """What ``ops.scan_usable`` checks, without the library: a head's matrix and its helpers fit in 227 KB of
     shared memory and a value is at most 256 wide."""
@@ -232,3 +294,4 @@ def ops_scan_size_ok(dk: int, dv: int, parts: int = 1) -> bool:
 
 register_part("mixer", "matrix_lstm", MatrixLSTM)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
+register_part("mixer", "retention", Retention)

@@ -10,13 +10,15 @@ FEED_FORWARDS: dict = {}
 ARRANGEMENTS: dict = {}
 TOKEN_INPUTS: dict = {}
 CONNECTIONS: dict = {}
+INPUT_FILTERS: dict = {}
 
 _TABLES = {"norm": NORMS, "position": POSITION_ENCODINGS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS,
-           "arrangement": ARRANGEMENTS, "token_input": TOKEN_INPUTS, "connection": CONNECTIONS}
+           "arrangement": ARRANGEMENTS, "token_input": TOKEN_INPUTS, "connection": CONNECTIONS,
+           "input_filter": INPUT_FILTERS}
 
 
 def register_part(family: str, kind: str, cls) -> None:
-    """``family``: norm, position, mixer, feed_forward, token_input, connection or arrangement."""
+    """``family``: norm, position, mixer, feed_forward, token_input, connection, input_filter or arrangement."""
     _TABLES[family][kind] = cls
 
 

@@ -57,17 +57,18 @@ class StreamUpdate:
     link: StreamLink
 
 
-def read_streams(norm, x, streams: int, pending, read, want_f32: bool = False):
+def read_streams(norm, x, streams: int, pending, read, want_f32: bool = False, want_rows: bool = True):
     """Brings the copies ``x`` up to date with ``pending`` (a ``StreamUpdate`` or None), reads them with ``read``
     ([streams] float32, None: the plain sum) and norms the result.  A norm that has ``read_streams`` does all of it
-    in one kernel; any other norm gets what was read as a stream of its own."""
+    in one kernel; any other norm gets what was read as a stream of its own.  ``want_rows`` False: the rows in the
+    activation dtype are not needed (only the float32 ones)."""
     branch = carry = write = None
     if pending is not None:
         if not isinstance(pending, StreamUpdate):
             raise TypeError("the copies of a stream take a StreamUpdate")
         branch, carry, write = pending.branch, pending.link.carry, pending.link.write
     if hasattr(norm, "read_streams"):
-        return norm.read_streams(x, streams, branch, carry, write, read, want_f32)
+        return norm.read_streams(x, streams, branch, carry, write, read, want_f32, want_rows)
     mix = None
     if isinstance(branch, RowMix):
         if branch.gate_logit is None and branch.index.shape[1] <= ops.STREAM_MAX_MIX:
@@ -81,16 +82,16 @@ def read_streams(norm, x, streams: int, pending, read, want_f32: bool = False):
 
 class HyperConnectedBlock(Arrangement):
     """A pre-norm layer around ``streams`` copies of the residual stream (``LayerSpec.params["streams"]``): the mixer
-    behind ``norm1`` through ``link1``, then, if the layer has one, the feed-forward behind ``norm2`` through
+    behind ``norm1`` (and, if the layer has one, its ``input_filter``) through ``link1``, then, if the layer has one, the feed-forward behind ``norm2`` through
     ``link2``.  ``x`` is ``[T, streams * hidden]``; the layer's last output is handed on as a ``StreamUpdate``."""
-    slots = {"norm1": "norm", "mixer": "mixer", "link1": "connection", "norm2": "norm", "feed_forward": "feed_forward",
-             "link2": "connection"}
-    optional = ("norm2", "feed_forward", "link2")
+    slots = {"norm1": "norm", "input_filter": "input_filter", "mixer": "mixer", "link1": "connection", "norm2": "norm",
+             "feed_forward": "feed_forward", "link2": "connection"}
+    optional = ("input_filter", "norm2", "feed_forward", "link2")
 
     def __init__(self, spec):
         super().__init__(spec)
         self.streams = int(spec.params.get("streams", 1))
-        present = [getattr(self, s) is not None for s in self.optional]
+        present = [getattr(self, s) is not None for s in ("norm2", "feed_forward", "link2")]
         if any(present) != all(present):
             raise ValueError("a hyper-connected layer's feed-forward comes with its norm and its link")
         for link in (self.link1, self.link2):
@@ -98,7 +99,8 @@ class HyperConnectedBlock(Arrangement):
                 raise ValueError("a layer's links must have as many copies as the layer")
 
     def forward(self, x, pending, batch, cache):
-        h, _ = read_streams(self.norm1, x, self.streams, pending, self.link1.read)
+        h, cache = self.mixer_input(lambda f32, rows: read_streams(self.norm1, x, self.streams, pending, self.link1.read,
+                                                                   want_f32=f32, want_rows=rows), batch, cache)
         pending = StreamUpdate(self.mixer.forward(h, batch, cache), self.link1)
         if self.feed_forward is not None:
             h, h32 = read_streams(self.norm2, x, self.streams, pending, self.link2.read,
