@@ -170,9 +170,14 @@ def connected(X, W, p, g, eps, F):
 
 
 # ------------------------------------------------------------------------------ the whole model
-def forward(cfg, W, tokens, layer_sums=None, margins=None):
+def forward(cfg, W, tokens, layer_sums=None, margins=None, noise=None):
     """Logits [T, vocab] of a whole sequence.  ``layer_sums``: a list that receives the sum of the copies after every
-    layer; ``margins``: a list that receives every router's ``choice_margins``."""
+    layer; ``margins``: a list that receives every router's ``choice_margins``; ``noise`` = (generator, size): what every
+    sublayer reads and gives is multiplied by 1 + size * N(0, 1), element by element, as roundings would change it."""
+
+    def noisy(t):
+        return t if noise is None else t * (1.0 + noise[1] * torch.randn(t.shape, generator=noise[0], dtype=F64))
+
     n, eps = int(cfg.get("streams", 1)), float(cfg["norm"]["eps"])
     x = W["embed"][torch.tensor(tokens, dtype=torch.long)] * float(cfg["embedding"]["scale"])
     X = x[:, None, :].repeat(1, n, 1)
@@ -181,7 +186,7 @@ def forward(cfg, W, tokens, layer_sums=None, margins=None):
         p, m = f"l{i}.", L["mixer"]
 
         def mixer(h):
-            h = h + causal_convolution(h, W[p + "canon1"])
+            h = noisy(h + causal_convolution(h, W[p + "canon1"]))
             if L["type"].startswith("retention"):
                 return retention(h, W, p + "mix.", m, eps)
             j = m.get("kv_from")
@@ -189,12 +194,30 @@ def forward(cfg, W, tokens, layer_sums=None, margins=None):
                 kept[i] = keys_and_values(h, W, p + "mix.", m, eps)
             return attention(h, W, p + "mix.", m, eps, kept[i if j is None else int(j)])
 
-        X = connected(X, W, p + "hc1.", p + "norm1", eps, mixer)
+        X = connected(X, W, p + "hc1.", p + "norm1", eps, lambda h: noisy(mixer(h)))
         if L.get("mlp"):
-            X = connected(X, W, p + "hc2.", p + "norm2", eps, lambda h: feed_forward(h, W, p + "mlp.", L["mlp"], margins))
+            X = connected(X, W, p + "hc2.", p + "norm2", eps,
+                          lambda h: noisy(feed_forward(noisy(h), W, p + "mlp.", L["mlp"], margins)))
         if layer_sums is not None:
             layer_sums.append(X.sum(dim=1))
     return norm_one_plus(X.sum(dim=1), W["final.norm"], eps) @ W["head"].T
+
+
+def rounding_errors(cfg, W, tokens, size, draws=4, layer=None):
+    """Per row, the largest change of the logits (or of the stream's sum after layer ``layer``) that roundings of the
+    relative size ``size`` cause: some rows carry small differences of large terms (a retention head that is divided by
+    its root mean square) and move further than others."""
+    def run(noise):
+        sums = []
+        lg = forward(cfg, W, tokens, layer_sums=sums, noise=noise)
+        return sums if layer else [lg]
+
+    want = run(None)
+    worst = [torch.zeros(len(tokens), dtype=F64) for _ in want]
+    for d in range(draws):
+        for i, got in enumerate(run((torch.Generator().manual_seed(d), size))):
+            worst[i] = torch.maximum(worst[i], (got - want[i]).abs().max(dim=1).values)
+    return worst if layer else worst[0]
 
 
 def greedy_generate(cfg, W, prompt, n):
@@ -207,7 +230,7 @@ def greedy_generate(cfg, W, prompt, n):
 # ------------------------------------------------------------------------------ weights
 def tensor_table(cfg):
     """name -> (shape, kind) of every tensor the model has; kinds: embed, matrix, shift (around zero), gain (around one),
-    read / carry / write (the copies' small tensors), taps, bias."""
+    read / carry / write (the copies' small tensors), taps, router, bias."""
     Wd, V, n = int(cfg["width"]), int(cfg["vocab"]), int(cfg.get("streams", 1))
     out = {"embed": ((V, Wd), "embed"), "head": ((V, Wd), "matrix"), "final.norm": ((Wd,), "shift")}
 
@@ -241,7 +264,7 @@ def tensor_table(cfg):
             else:
                 E = int(f["router"]["experts"])
                 names, ff = [f"{y}e{e}." for e in range(E)], int(f["expert"]["ff"])
-                out[y + "router"], out[y + "router.b"] = ((E, Wd), "matrix"), ((E,), "bias")
+                out[y + "router"], out[y + "router.b"] = ((E, Wd), "router"), ((E,), "bias")
             for z in names:
                 out[z + "gate"], out[z + "up"], out[z + "down"] = ((ff, Wd), "matrix"), ((ff, Wd), "matrix"), ((Wd, ff), "matrix")
     return out
@@ -262,8 +285,10 @@ def make_weights(cfg, seed, scale=1.0):
             t = 1.0 + 0.2 * z
         elif kind == "shift":
             t = 0.2 * z
+        elif kind == "router":      # (choices that hang on the bias as much as on the row: few of them are close)
+            t = z * 0.5 / math.sqrt(shape[-1])
         elif kind == "bias":
-            t = 0.5 * z
+            t = 1.2 * z
         elif kind == "taps":
             t = 0.4 * z
         elif kind == "read":
