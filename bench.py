@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, one JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-    python bench.py --design bizodra|kifunex|sanesun|gekitar [--design-sizes s,m]     (another measurement, see ``design_bench``)
+    python bench.py --design bizodra|kifunex|sanesun|gekitar|sevelorn [--design-sizes s,m]     (another measurement, see ``design_bench``)
 
 Default run: the layer sizes of the Qwen1.5-MoE-A2.7B shape with random bfloat16 weights, a batch
 of 8 sequences each at a 2,048-token context; a step is one decode step of that batch.  ``value``
@@ -246,10 +246,10 @@ KIFUNEX_SIZES = {
 def kifunex_config(z):
     D = z["dim"]
     mixer = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5,
-             "mask": {"size": z["window"]},
+             "mask": {"size": z["window"]} if z["window"] else None,
              "rot": {"dims": D // 2, "base": 1e6, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
     mlp = {"kind": "moe", "expert": {"ff": z["ff"]}, "router": {"experts": z["experts"], "top": z["top"], "scale": 1.0},
-           "shared": {"ff": z["shared_ff"]}}
+           "shared": {"ff": z["shared_ff"]} if z["shared_ff"] else None}
     return {"architecture": "Kifunex", "vocab": z["vocab"], "width": z["width"], "streams": z["streams"],
             "norm": {"eps": 1e-6}, "logit_scale": 1.0, "logit_softcap": 30.0,
             "layers": [{"type": "attention", "mixer": mixer, "mlp": mlp} for _ in range(z["layers"])]}
@@ -315,10 +315,41 @@ def gekitar_config(z):
             "layers": layers}
 
 
-DESIGNS = {"bizodra": (DESIGN_SIZES, "bizodra", bizodra_config, "qwen2_dense", dense_qwen_config),
-           "kifunex": (KIFUNEX_SIZES, "kifunex", kifunex_config, "qwen2_moe", sparse_qwen_config),
-           "sanesun": (DESIGN_SIZES, "sanesun", sanesun_config, "bizodra", bizodra_config),
-           "gekitar": (KIFUNEX_SIZES, "gekitar", gekitar_config, "qwen2_moe", sparse_qwen_config)}
+# --design sevelorn: the same measurement for the Sevelorn decoder beside the two existing models that have its parts, at
+# equal size: the Kifunex decoder (several copies of the stream around attention and a mixture of SwiGLU experts; here
+# without a window and a shared expert, which Sevelorn has not) with the same width, depth, copies, heads, head size,
+# experts, expert width and vocabulary, and the Bizodra decoder (matrix memories beside attention) with the same width,
+# depth, heads, head size and vocabulary and a dense MLP of the width that a token uses in a mixture.  Sevelorn's layers go
+# retention, attention, retention, attention on the second layer's pages; the first feed-forward of four is dense.
+SEVELORN_SIZES = {
+    "s": dict(width=1024, layers=4, heads=8, kv_heads=2, dim=128, window=0, experts=16, top=4, ff=512, shared_ff=0,
+              streams=2, vocab=32000),
+    "m": dict(width=2048, layers=8, heads=16, kv_heads=4, dim=128, window=0, experts=32, top=4, ff=768, shared_ff=0,
+              streams=2, vocab=32000),
+}
+
+
+def sevelorn_config(z):
+    H, G, D = z["heads"], z["kv_heads"], z["dim"]
+    ret = {"heads": H, "dim": D, "vdim": D, "decay": [1.0 - 2.0 ** (-5 - 7 * h / max(1, H - 1)) for h in range(H)],
+           "rot": {"dims": D, "base": 1e4}}
+    attn = {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    dense = {"kind": "dense", "ff": z["top"] * z["ff"]}
+    kinds = lambda i: [("retention", ret, dense), ("attention", attn, moe), ("retention", ret, moe),
+                       ("attention", dict(attn, kv_from=i - 2), moe)][i % 4]
+    layers = [dict(zip(("type", "mixer", "mlp"), kinds(i))) for i in range(z["layers"])]
+    return {"architecture": "Sevelorn", "vocab": z["vocab"], "width": z["width"], "streams": z["streams"], "canon": {"taps": 4},
+            "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": layers}
+
+
+# sizes, the design, and the existing models it is measured beside
+DESIGNS = {"bizodra": (DESIGN_SIZES, [("bizodra", bizodra_config), ("qwen2_dense", dense_qwen_config)]),
+           "kifunex": (KIFUNEX_SIZES, [("kifunex", kifunex_config), ("qwen2_moe", sparse_qwen_config)]),
+           "sanesun": (DESIGN_SIZES, [("sanesun", sanesun_config), ("bizodra", bizodra_config)]),
+           "gekitar": (KIFUNEX_SIZES, [("gekitar", gekitar_config), ("qwen2_moe", sparse_qwen_config)]),
+           "sevelorn": (SEVELORN_SIZES, [("sevelorn", sevelorn_config), ("kifunex", kifunex_config),
+                                         ("bizodra", lambda z: bizodra_config(dict(z, ff=z["top"] * z["ff"])))])}
 
 
 def design_bench(args) -> int:
@@ -347,10 +378,11 @@ def design_bench(args) -> int:
             ts.append(a.elapsed_time(b))
         return sorted(ts)[len(ts) // 2]
 
-    sizes, design_name, design_cfg, beside_name, beside_cfg = DESIGNS[args.design]
+    sizes, models = DESIGNS[args.design]
     for size in args.design_sizes.split(","):
         z = sizes[size]
-        for model, cfg in ((design_name, design_cfg(z)), (beside_name, beside_cfg(z))):
+        for model, make in models:
+            cfg = make(z)
             work = tempfile.mkdtemp(prefix="bench_design_")
             with open(os.path.join(work, "config.json"), "w") as f:
                 json.dump(cfg, f)
@@ -387,7 +419,7 @@ def design_bench(args) -> int:
             with ops.KernelTimes() as kt:
                 prefill_many()
             row["prefill_together"]["kernels"] = [{"name": r["name"], "calls": r["calls"], "ms": round(r["ms"], 3)}
-                                                  for r in kt.summary()[:6]]
+                                                  for r in kt.summary()[:12]]
             runner.cuda_graphs = graphs
             # the prompt's kernels one by one (outside graphs, an event between any two)
             graphs, runner.cuda_graphs = runner.cuda_graphs, False
@@ -396,7 +428,7 @@ def design_bench(args) -> int:
             runner.close("kt")
             row["prefill_kernels"] = [{"name": r["name"], "calls": r["calls"], "ms": round(r["ms"], 3),
                                        **({"frac_bf16": round(r["flops"] / (r["ms"] * 1e-3) / (P["bf16_tflops"] * 1e12), 3)} if r["flops"] else {})}
-                                      for r in kt.summary()[:8]]
+                                      for r in kt.summary()[:12]]
             runner.cuda_graphs = graphs
             for B in batches:
                 rids = [f"d{B}_{i}" for i in range(B)]
@@ -429,7 +461,7 @@ def design_bench(args) -> int:
                             ops.delay(20000)
                             runner.step(entries, check=False)
                     row["decode_kernels"] = [{"name": r["name"], "calls": r["calls"] // 4, "ms": round(r["ms"] / 4, 4)}
-                                             for r in kt.summary()[:8]]
+                                             for r in kt.summary()[:12]]
                     runner.cuda_graphs = graphs
                 for rid in rids:
                     runner.close(rid)
@@ -437,7 +469,8 @@ def design_bench(args) -> int:
             rows.append(row)
             del runner
             torch.cuda.empty_cache()
-    print(json.dumps({"metric": "design_throughput", "design": design_name, "beside": beside_name, "dtype": "bf16",
+    print(json.dumps({"metric": "design_throughput", "design": models[0][0],
+                      "beside": ", ".join(name for name, _ in models[1:]), "dtype": "bf16",
                       "data": "synthetic", "peaks": {"source": peak_src, **P}, "steps": args.steps, "warmup": args.warmup,
                       "clocks": clocks.stop(), "rows": rows}))
     return 0

@@ -168,7 +168,8 @@ struct RetArgs {
   void* out;                // [T, H * dv]
   float* raw;               // scan: [T, H, dv]
   uint32_t* chunks;         // chunked form: per chunk and head dk * dv words (float32 sums, then the states' two terms)
-  int out_dt, H, dk, dv, num_entries, min_rows, slice, v2;
+  // v2: the chunked form reads two neighbouring elements at a time; planes: the states' terms lie row by row (see the pass)
+  int out_dt, H, dk, dv, num_entries, min_rows, slice, v2, planes;
 };
 
 constexpr int RC = 64;                 // rows of a chunk
@@ -343,6 +344,9 @@ constexpr int CK_THREADS = 128;        // four warps
 constexpr int VLD = 64 + 8;            // row of a 64-column slab in shared memory (sixteen bytes of padding)
 
 __device__ __forceinline__ uint32_t s_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s_u32(dst)), "l"(src) : "memory");
+}
 __device__ __forceinline__ void ldsm4(const bf16* p, uint32_t* r) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s_u32(p)));
@@ -413,29 +417,45 @@ template <int DKP, typename F>
 __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, int row0, int n, F factor, bf16* hi, bf16* lo) {
   constexpr int LDS = DKP + 8;
   const int half = a.half, dk = a.dk, tid = threadIdx.x;
-  if (a.v2) {                          // two neighbouring elements at a time (sizes and addresses are even)
-    const int h2 = half / 2, items = h2 + (dk - 2 * half) / 2;
-    for (int x = tid; x < RC * items; x += CK_THREADS) {
-      const int r = x / items, i = x - r * items;
-      const bool live = r < n;
-      const float f = live ? factor(r) : 0.f;
-      const float* p = src + (size_t)(row0 + (live ? r : 0)) * a.ld;
-      uint32_t wh, wl;
-      if (i < h2) {
-        const float2 u = *reinterpret_cast<const float2*>(p + 2 * i), w = *reinterpret_cast<const float2*>(p + 2 * i + half);
-        const float4 cs = *reinterpret_cast<const float4*>(a.table + (size_t)(row0 + (live ? r : 0)) * half + 2 * i);
-        split2(live ? (u.x * cs.x - w.x * cs.y) * f : 0.f, live ? (u.y * cs.z - w.y * cs.w) * f : 0.f, wh, wl);
-        *reinterpret_cast<uint32_t*>(hi + r * LDS + 2 * i) = wh;
-        *reinterpret_cast<uint32_t*>(lo + r * LDS + 2 * i) = wl;
-        split2(live ? (w.x * cs.x + u.x * cs.y) * f : 0.f, live ? (w.y * cs.z + u.y * cs.w) * f : 0.f, wh, wl);
-        *reinterpret_cast<uint32_t*>(hi + r * LDS + 2 * i + half) = wh;
-        *reinterpret_cast<uint32_t*>(lo + r * LDS + 2 * i + half) = wl;
-      } else {
-        const int d = 2 * half + 2 * (i - h2);
-        const float2 u = *reinterpret_cast<const float2*>(p + d);
-        split2(live ? u.x * f : 0.f, live ? u.y * f : 0.f, wh, wl);
-        *reinterpret_cast<uint32_t*>(hi + r * LDS + d) = wh;
-        *reinterpret_cast<uint32_t*>(lo + r * LDS + d) = wl;
+  if (a.v2) {
+    // Two neighbouring elements at a time (sizes and addresses are even): a warp takes every fourth row, its lanes the
+    // row's elements side by side, and the loads of four rows are in flight before the first is used.
+    const int h2 = half / 2, items = h2 + (dk - 2 * half) / 2, lane = tid & 31, warp = tid >> 5;
+    constexpr int B = 4;
+    for (int i = lane; i < items; i += 32) {
+      const bool turned = i < h2;
+      const int d = turned ? 2 * i : 2 * half + 2 * (i - h2);
+      for (int r0 = warp; r0 < RC; r0 += 4 * B) {
+        float2 u[B], w[B];
+        float4 cs[B];
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+          const int r = r0 + 4 * b;
+          u[b] = w[b] = make_float2(0.f, 0.f);
+          cs[b] = make_float4(1.f, 0.f, 1.f, 0.f);
+          if (r < n) {
+            const float* p = src + (size_t)(row0 + r) * a.ld + d;
+            u[b] = *reinterpret_cast<const float2*>(p);
+            if (turned) {
+              w[b] = *reinterpret_cast<const float2*>(p + half);
+              cs[b] = *reinterpret_cast<const float4*>(a.table + (size_t)(row0 + r) * half + 2 * i);
+            }
+          }
+        }
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+          const int r = r0 + 4 * b;
+          const float f = r < n ? factor(r) : 0.f;
+          uint32_t wh, wl;
+          split2((u[b].x * cs[b].x - w[b].x * cs[b].y) * f, (u[b].y * cs[b].z - w[b].y * cs[b].w) * f, wh, wl);
+          *reinterpret_cast<uint32_t*>(hi + r * LDS + d) = wh;
+          *reinterpret_cast<uint32_t*>(lo + r * LDS + d) = wl;
+          if (turned) {
+            split2((w[b].x * cs[b].x + u[b].x * cs[b].y) * f, (w[b].y * cs[b].z + u[b].y * cs[b].w) * f, wh, wl);
+            *reinterpret_cast<uint32_t*>(hi + r * LDS + d + half) = wh;
+            *reinterpret_cast<uint32_t*>(lo + r * LDS + d + half) = wl;
+          }
+        }
       }
     }
   } else {
@@ -465,14 +485,26 @@ __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, 
 // Columns c0 .. c0 + 63 of the value head of the chunk's rows, as two terms [RC][VLD]; what does not exist is zero.
 __device__ __forceinline__ void load_values(const RetArgs& a, const float* src, int row0, int n, int c0, bf16* hi, bf16* lo) {
   if (a.v2) {
-    for (int x = threadIdx.x; x < RC * 32; x += CK_THREADS) {
-      const int r = x / 32, c = 2 * (x % 32);
-      float2 v = make_float2(0.f, 0.f);
-      if (r < n && c0 + c < a.dv) v = *reinterpret_cast<const float2*>(src + (size_t)(row0 + r) * a.ld + c0 + c);
-      uint32_t wh, wl;
-      split2(v.x, v.y, wh, wl);
-      *reinterpret_cast<uint32_t*>(hi + r * VLD + c) = wh;
-      *reinterpret_cast<uint32_t*>(lo + r * VLD + c) = wl;
+    constexpr int B = 8;
+    const int c = 2 * (threadIdx.x & 31);
+    const bool col = c0 + c < a.dv;
+#pragma unroll
+    for (int r0 = threadIdx.x >> 5; r0 < RC; r0 += 4 * B) {
+      float2 v[B];
+#pragma unroll
+      for (int b = 0; b < B; ++b) {
+        const int r = r0 + 4 * b;
+        v[b] = make_float2(0.f, 0.f);
+        if (r < n && col) v[b] = *reinterpret_cast<const float2*>(src + (size_t)(row0 + r) * a.ld + c0 + c);
+      }
+#pragma unroll
+      for (int b = 0; b < B; ++b) {
+        const int r = r0 + 4 * b;
+        uint32_t wh, wl;
+        split2(v[b].x, v[b].y, wh, wl);
+        *reinterpret_cast<uint32_t*>(hi + r * VLD + c) = wh;
+        *reinterpret_cast<uint32_t*>(lo + r * VLD + c) = wl;
+      }
     }
   } else {
     for (int x = threadIdx.x; x < RC * 64; x += CK_THREADS) {
@@ -554,8 +586,80 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_sum_kernel(RetArgs
   }
 }
 
-// Turns an entry's chunk sums into the states its chunks start from, each packed as its two bfloat16 terms in one word
-// (in place: the same thread reads and writes an element), and leaves the last state in the request's slot.
+// Chunks of the entries before entry e, worked out by warp 0.
+__device__ __forceinline__ void count_chunks_before(const int* cu_rows, int e, int min_rows, int* first) {
+  if (threadIdx.x < 32) {
+    int sum = 0;
+    for (int i = threadIdx.x; i < e; i += 32) {
+      const int m = cu_rows[i + 1] - cu_rows[i];
+      sum += m >= min_rows ? (m + RC - 1) / RC : 0;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if (threadIdx.x == 0) *first = sum;
+  }
+  __syncthreads();
+}
+
+// Turns an entry's chunk sums into the states its chunks start from, in place, and leaves the last state in the request's
+// slot.  Here every row of a state becomes the row's leading terms [dv bfloat16] and behind them its rest terms
+// [dv bfloat16], which the next kernel copies as they are.  A warp owns a row (its lanes four columns each, NJ times):
+// all of a row's sums are read before its terms are written over them.  grid (entries, heads, dk / 8).
+template <int NJ>
+__global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs a) {
+  __shared__ int first_s;
+  const int e = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
+  grid_dep_wait();
+  grid_dep_launch();
+  const int n = a.cu_rows[e + 1] - a.cu_rows[e];
+  if (n < a.min_rows) return;
+  count_chunks_before(a.cu_rows, e, a.min_rows, &first_s);
+  const int d = blockIdx.z * 8 + (threadIdx.x >> 5);
+  if (d >= a.dk) return;
+  const int count = (n + RC - 1) / RC, dv = a.dv;
+  const size_t size = (size_t)a.dk * dv, step = (size_t)a.H * size;
+  uint32_t* p = a.chunks + ((size_t)first_s * a.H + h) * size + (size_t)d * dv;
+  float* Sg = a.S + (size_t)a.entry_slot[e] * a.S_stride + (size_t)h * size + (size_t)d * dv;
+  const float full = a.powers[(size_t)h * (RC + 1) + RC], last = a.powers[(size_t)h * (RC + 1) + n - (count - 1) * RC];
+  Vals<4> S[NJ];
+#pragma unroll
+  for (int j = 0; j < NJ; ++j)
+    if (4 * (lane + 32 * j) < dv) S[j] = ldv<4>(Sg + 4 * (lane + 32 * j));
+  constexpr int U = 8 / NJ;            // chunk sums in flight
+  for (int c0 = 0; c0 < count; c0 += U) {
+    Vals<4> u[U][NJ];
+#pragma unroll
+    for (int i = 0; i < U; ++i)
+#pragma unroll
+      for (int j = 0; j < NJ; ++j)
+        if (c0 + i < count && 4 * (lane + 32 * j) < dv)
+          u[i][j] = ldv<4>(reinterpret_cast<const float*>(p) + (size_t)(c0 + i) * step + 4 * (lane + 32 * j));
+    __syncwarp();                      // the row's sums have been read by all lanes
+#pragma unroll
+    for (int i = 0; i < U; ++i)
+      if (c0 + i < count) {
+        const float f = c0 + i + 1 < count ? full : last;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const int c = 4 * (lane + 32 * j);
+          if (c >= dv) continue;
+          uint2 hi, lo;
+          split2(S[j].v[0], S[j].v[1], hi.x, lo.x);
+          split2(S[j].v[2], S[j].v[3], hi.y, lo.y);
+          bf16* row = reinterpret_cast<bf16*>(p + (size_t)(c0 + i) * step);
+          *reinterpret_cast<uint2*>(row + c) = hi;
+          *reinterpret_cast<uint2*>(row + dv + c) = lo;
+#pragma unroll
+          for (int x = 0; x < 4; ++x) S[j].v[x] = fmaf(f, S[j].v[x], u[i][j].v[x]);
+        }
+      }
+  }
+#pragma unroll
+  for (int j = 0; j < NJ; ++j)
+    if (4 * (lane + 32 * j) < dv) stv<4>(Sg + 4 * (lane + 32 * j), S[j]);
+}
+
+// The same for other sizes: an element's two terms are packed in one word (the same thread reads and writes an element).
 // grid (entries, heads, elements / 256).
 __global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
   __shared__ int first_s;
@@ -564,17 +668,7 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
   grid_dep_launch();
   const int n = a.cu_rows[e + 1] - a.cu_rows[e];
   if (n < a.min_rows) return;
-  if (tid < 32) {                      // chunks of the entries before this one
-    int sum = 0;
-    for (int i = tid; i < e; i += 32) {
-      const int m = a.cu_rows[i + 1] - a.cu_rows[i];
-      sum += m >= a.min_rows ? (m + RC - 1) / RC : 0;
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    if (tid == 0) first_s = sum;
-  }
-  __syncthreads();
+  count_chunks_before(a.cu_rows, e, a.min_rows, &first_s);
   const int i = blockIdx.z * 256 + tid, size = a.dk * a.dv;
   if (i >= size) return;
   const int count = (n + RC - 1) / RC;
@@ -680,15 +774,20 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
   for (int sl = 0; sl < NS; ++sl) {
     const int c0 = sl * 64;
     __syncthreads();                               // the keys (or the last slab) have been read by everyone
-    load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
-    if (a.v2) {
-      for (int x = tid; x < DKP * 32; x += CK_THREADS) {
-        const int d = x / 32, c = 2 * (x % 32);
-        uint2 w = make_uint2(0, 0);
-        if (d < a.dk && c0 + c < a.dv) w = *reinterpret_cast<const uint2*>(St + (size_t)d * a.dv + c0 + c);
-        *reinterpret_cast<uint32_t*>(kh + d * VLD + c) = __byte_perm(w.x, w.y, 0x5410);
-        *reinterpret_cast<uint32_t*>(kl + d * VLD + c) = __byte_perm(w.x, w.y, 0x7632);
+    if (a.planes) {                                // the state's terms as they are, sixteen bytes at a time
+#pragma unroll 4
+      for (int x = tid; x < DKP * 16; x += CK_THREADS) {
+        const int d = x >> 4, c = 8 * (x & 7), term = (x >> 3) & 1;
+        bf16* dst = (term ? kl : kh) + d * VLD + c;
+        if (d < a.dk && c0 + c < a.dv)
+          cp_async16(dst, reinterpret_cast<const bf16*>(St + (size_t)d * a.dv) + term * a.dv + c0 + c);
+        else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
       }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
+    if (a.planes) {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
     } else {
       for (int x = tid; x < DKP * 64; x += CK_THREADS) {
         const int d = x / 64, c = x % 64;
@@ -798,7 +897,10 @@ int launch_chunks(const RetArgs& a, int max_chunks, cudaStream_t s) {
   if (rc) return rc;
   const dim3 grid(max_chunks, a.H);
   NV_RETURN_IF(launch_dep(retention_chunk_sum_kernel<DKP>, grid, dim3(CK_THREADS), chunk_sum_smem<DKP>(), s, a));
-  NV_RETURN_IF(launch_dep(retention_chunk_pass_kernel, dim3(a.num_entries, a.H, (a.dk * a.dv + 255) / 256), dim3(256), 0, s, a));
+  const dim3 rows(a.num_entries, a.H, (a.dk + 7) / 8);
+  if (a.planes && a.dv <= 128) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<1>, rows, dim3(256), 0, s, a));
+  else if (a.planes) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<2>, rows, dim3(256), 0, s, a));
+  else NV_RETURN_IF(launch_dep(retention_chunk_pass_kernel, dim3(a.num_entries, a.H, (a.dk * a.dv + 255) / 256), dim3(256), 0, s, a));
   NV_RETURN_IF(launch_dep(retention_chunk_out_kernel<DKP, NS>, grid, dim3(CK_THREADS), chunk_out_smem<DKP>(), s, a));
   NV_RETURN_LAST();
 }
@@ -899,6 +1001,7 @@ NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k
     a.v2 = (half % 2 == 0 && dk % 2 == 0 && dv % 2 == 0 && ld % 2 == 0 && q0 % 2 == 0 && k0 % 2 == 0 && v0 % 2 == 0 &&
             g0 % 2 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)table & 15) && !((uintptr_t)chunks & 15) &&
             !((uintptr_t)out & 15)) ? 1 : 0;
+    a.planes = (dv % 8 == 0 && S_stride % 4 == 0 && !((uintptr_t)S & 15) && !((uintptr_t)chunks & 15)) ? 1 : 0;
     if (dk <= 64) return launch_chunks_ns<64>(a, max_chunks, s);
     if (dk <= 128) return launch_chunks_ns<128>(a, max_chunks, s);
     return launch_chunks_ns<256>(a, max_chunks, s);

@@ -223,7 +223,7 @@ __global__ void conv_state_update_kernel(const void* __restrict__ in, int in_dt,
   const int e = blockIdx.x;
   const int row0 = cu_rows[e], len = cu_rows[e + 1] - row0;
   float* st = state + (size_t)entry_slot[e] * slot_stride;
-  for (int c = threadIdx.x; c < C; c += blockDim.x)
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x)
     for (int s = 0; s < taps - 1; ++s) {
       const int jj = len - (taps - 1) + s;
       st[(size_t)s * C + c] = jj >= 0 ? ld_dt(in, in_dt, (size_t)(row0 + jj) * ld + col0 + c) : st[(size_t)(s + len) * C + c];
@@ -1317,7 +1317,7 @@ NV_API int nv_conv_state_update(const void* in, int in_dt, long long ld, int col
   if (!dt_ok(in_dt)) return NV_ERR_BAD_DTYPE;
   if (C <= 0 || taps < 1) return NV_ERR_BAD_SIZE;
   if (S == 0 || taps == 1) return NV_OK;
-  conv_state_update_kernel<<<S, SM_THREADS, 0, s>>>(in, in_dt, ld, col0, C, taps, cu_rows, entry_slot, state,
+  conv_state_update_kernel<<<dim3(S, (C + SM_THREADS - 1) / SM_THREADS), SM_THREADS, 0, s>>>(in, in_dt, ld, col0, C, taps, cu_rows, entry_slot, state,
                                                     slot_stride);
   NV_RETURN_LAST();
 }
