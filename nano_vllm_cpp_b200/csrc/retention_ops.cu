@@ -340,7 +340,7 @@ __global__ void __launch_bounds__(256) retention_finish_kernel(RetArgs a, int T)
 }
 
 // ------------------------------------------------------------------ the chunked form
-constexpr int CK_THREADS = 128;        // four warps
+constexpr int CK_THREADS = 256, CK_WARPS = CK_THREADS / 32;
 constexpr int VLD = 64 + 8;            // row of a 64-column slab in shared memory (sixteen bytes of padding)
 
 __device__ __forceinline__ uint32_t s_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -418,19 +418,19 @@ __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, 
   constexpr int LDS = DKP + 8;
   const int half = a.half, dk = a.dk, tid = threadIdx.x;
   if (a.v2) {
-    // Two neighbouring elements at a time (sizes and addresses are even): a warp takes every fourth row, its lanes the
+    // Two neighbouring elements at a time (sizes and addresses are even): a warp takes every eighth row, its lanes the
     // row's elements side by side, and the loads of four rows are in flight before the first is used.
     const int h2 = half / 2, items = h2 + (dk - 2 * half) / 2, lane = tid & 31, warp = tid >> 5;
     constexpr int B = 4;
     for (int i = lane; i < items; i += 32) {
       const bool turned = i < h2;
       const int d = turned ? 2 * i : 2 * half + 2 * (i - h2);
-      for (int r0 = warp; r0 < RC; r0 += 4 * B) {
+      for (int r0 = warp; r0 < RC; r0 += CK_WARPS * B) {
         float2 u[B], w[B];
         float4 cs[B];
 #pragma unroll
         for (int b = 0; b < B; ++b) {
-          const int r = r0 + 4 * b;
+          const int r = r0 + CK_WARPS * b;
           u[b] = w[b] = make_float2(0.f, 0.f);
           cs[b] = make_float4(1.f, 0.f, 1.f, 0.f);
           if (r < n) {
@@ -444,7 +444,7 @@ __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, 
         }
 #pragma unroll
         for (int b = 0; b < B; ++b) {
-          const int r = r0 + 4 * b;
+          const int r = r0 + CK_WARPS * b;
           const float f = r < n ? factor(r) : 0.f;
           uint32_t wh, wl;
           split2((u[b].x * cs[b].x - w[b].x * cs[b].y) * f, (u[b].y * cs[b].z - w[b].y * cs[b].w) * f, wh, wl);
@@ -489,17 +489,17 @@ __device__ __forceinline__ void load_values(const RetArgs& a, const float* src, 
     const int c = 2 * (threadIdx.x & 31);
     const bool col = c0 + c < a.dv;
 #pragma unroll
-    for (int r0 = threadIdx.x >> 5; r0 < RC; r0 += 4 * B) {
+    for (int r0 = threadIdx.x >> 5; r0 < RC; r0 += CK_WARPS * B) {
       float2 v[B];
 #pragma unroll
       for (int b = 0; b < B; ++b) {
-        const int r = r0 + 4 * b;
+        const int r = r0 + CK_WARPS * b;
         v[b] = make_float2(0.f, 0.f);
         if (r < n && col) v[b] = *reinterpret_cast<const float2*>(src + (size_t)(row0 + r) * a.ld + c0 + c);
       }
 #pragma unroll
       for (int b = 0; b < B; ++b) {
-        const int r = r0 + 4 * b;
+        const int r = r0 + CK_WARPS * b;
         uint32_t wh, wl;
         split2(v[b].x, v[b].y, wh, wl);
         *reinterpret_cast<uint32_t*>(hi + r * VLD + c) = wh;
@@ -517,7 +517,7 @@ __device__ __forceinline__ void load_values(const RetArgs& a, const float* src, 
 
 // Every chunk's own sum: U = sum_j d^(n-1-j) k_j v_j^T, float32 [dk][dv].  grid (chunks, heads).
 template <int DKP>
-__global__ void __launch_bounds__(CK_THREADS) retention_chunk_sum_kernel(RetArgs a) {
+__global__ void __launch_bounds__(CK_THREADS, DKP <= 128 ? 3 : 1) retention_chunk_sum_kernel(RetArgs a) {
   constexpr int LDS = DKP + 8;
   extern __shared__ __align__(16) uint8_t ck_smem[];
   bf16* kh = (bf16*)ck_smem;
@@ -543,13 +543,13 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_sum_kernel(RetArgs
     if (c0) __syncthreads();
     load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
     __syncthreads();
+    // an item of work is sixteen rows and 32 columns of U
+    for (int item = warp; item < DKP / 8; item += CK_WARPS) {
+      const int d0 = (item >> 1) * 16, n0 = (item & 1) * 32;
+      if (d0 >= a.dk || c0 + n0 >= a.dv) continue;
+      float c[4][4];
 #pragma unroll
-    for (int m = 0; m < DKP / 64; ++m) {
-      const int d0 = (m * 4 + warp) * 16;            // this warp's sixteen rows of U
-      if (d0 >= a.dk) continue;
-      float c[8][4];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
+      for (int i = 0; i < 4; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
 #pragma unroll
       for (int kb = 0; kb < RC / 16; ++kb) {
         if (kb * 16 >= n) continue;
@@ -558,9 +558,9 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_sum_kernel(RetArgs
         ldsm4_t(kh + at, ah);
         ldsm4_t(kl + at, al);
 #pragma unroll
-        for (int np = 0; np < 4; ++np) {
+        for (int np = 0; np < 2; ++np) {
           uint32_t bh[4], bl[4];
-          const int bt = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + np * 16 + 8 * (lane / 16);
+          const int bt = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + n0 + np * 16 + 8 * (lane / 16);
           ldsm4_t(vh + bt, bh);
           ldsm4_t(vl + bt, bl);
           mma_terms(c[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
@@ -568,8 +568,8 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_sum_kernel(RetArgs
         }
       }
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int col = c0 + i * 8 + 2 * tq;
+      for (int i = 0; i < 4; ++i) {
+        const int col = c0 + n0 + i * 8 + 2 * tq;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int d = d0 + g + 8 * half;
@@ -694,10 +694,13 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
   *Sg = S;
 }
 
-// Every chunk's outputs, its heads normed and gated.  grid (chunks, heads); a warp takes sixteen rows and all columns.
-// NS: slabs of 64 value columns.
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+
+// Every chunk's outputs, its heads normed and gated.  grid (chunks, heads).  Two warps share sixteen rows: each takes half
+// of the keys for the weights, which both then read from shared memory, and half of every slab's columns.  NS: slabs of
+// 64 value columns.
 template <int DKP, int NS>
-__global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs a) {
+__global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) retention_chunk_out_kernel(RetArgs a) {
   constexpr int LDS = DKP + 8;
   constexpr int KS = RC * LDS > DKP * VLD ? RC * LDS : DKP * VLD;      // the keys' place is the state's afterwards
   extern __shared__ __align__(16) uint8_t ck_smem[];
@@ -707,6 +710,9 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
   bf16* kl = kh + KS;
   bf16* vh = kl + KS;
   bf16* vl = vh + RC * VLD;
+  bf16* ph = vl + RC * VLD;            // the weights, two terms [RC][VLD]
+  bf16* pl = ph + RC * VLD;
+  __shared__ float squares[2][RC];
   __shared__ int info[3];
   __shared__ float pw[RC + 1];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
@@ -722,27 +728,27 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
   load_turned<DKP>(a, a.proj + a.k0 + (size_t)h * a.dk, row0, n, [&](int) { return ks; }, kh, kl);
   __syncthreads();
   const int g = lane / 4, tq = lane % 4;
-  const int r_lo = warp * 16 + g, r_hi = r_lo + 8;
-  const int q_at = (warp * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * LDS + 8 * (lane / 16);
-  const bool busy = warp * 16 < n;
+  const int rb = warp >> 1, side = warp & 1;         // rows 16 rb .. 16 rb + 15; which half of the keys and columns
+  const int r_lo = rb * 16 + g, r_hi = r_lo + 8;
+  const int q_at = (rb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * LDS + 8 * (lane / 16);
+  const bool busy = rb * 16 < n;
 
-  // the weights d^(i-j) (q_i . k_j) of this warp's rows, two terms, as operands of the product with the values
-  uint32_t ph[4][4], pl[4][4];
+  // the weights d^(i-j) (q_i . k_j) of these rows and this warp's 32 keys, as two terms
   {
-    float s[8][4];
+    float s[4][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-    if (busy) {
+    for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+    if (busy && 2 * side <= rb) {
 #pragma unroll
       for (int kk = 0; kk < DKP / 16; ++kk) {
         uint32_t ah[4], al[4];
         ldsm4(qh + q_at + kk * 16, ah);
         ldsm4(ql + q_at + kk * 16, al);
 #pragma unroll
-        for (int np = 0; np < 4; ++np) {
-          if (np > warp) continue;                 // keys after this warp's last row
+        for (int np = 0; np < 2; ++np) {
+          if (2 * side + np > rb) continue;        // keys after these rows
           uint32_t bh[4], bl[4];
-          const int at = (np * 16 + (lane % 8) + 8 * (lane / 16)) * LDS + kk * 16 + 8 * ((lane / 8) % 2);
+          const int at = ((2 * side + np) * 16 + (lane % 8) + 8 * (lane / 16)) * LDS + kk * 16 + 8 * ((lane / 8) % 2);
           ldsm4(kh + at, bh);
           ldsm4(kl + at, bl);
           mma_terms(s[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
@@ -751,24 +757,20 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
-#pragma unroll
-      for (int x = 0; x < 2; ++x) {
-        const int j = i * 8 + 2 * tq + x;
-        s[i][x] = j <= r_lo ? s[i][x] * pw[r_lo - j] : 0.f;
-        s[i][2 + x] = j <= r_hi ? s[i][2 + x] * pw[r_hi - j] : 0.f;
-      }
-#pragma unroll
-    for (int kb = 0; kb < 4; ++kb) {
-      split2(s[2 * kb][0], s[2 * kb][1], ph[kb][0], pl[kb][0]);
-      split2(s[2 * kb][2], s[2 * kb][3], ph[kb][1], pl[kb][1]);
-      split2(s[2 * kb + 1][0], s[2 * kb + 1][1], ph[kb][2], pl[kb][2]);
-      split2(s[2 * kb + 1][2], s[2 * kb + 1][3], ph[kb][3], pl[kb][3]);
+    for (int i = 0; i < 4; ++i) {
+      const int j = side * 32 + i * 8 + 2 * tq;
+      uint32_t wh, wl;
+      split2(j <= r_lo ? s[i][0] * pw[r_lo - j] : 0.f, j + 1 <= r_lo ? s[i][1] * pw[r_lo - j - 1] : 0.f, wh, wl);
+      *reinterpret_cast<uint32_t*>(ph + r_lo * VLD + j) = wh;
+      *reinterpret_cast<uint32_t*>(pl + r_lo * VLD + j) = wl;
+      split2(j <= r_hi ? s[i][2] * pw[r_hi - j] : 0.f, j + 1 <= r_hi ? s[i][3] * pw[r_hi - j - 1] : 0.f, wh, wl);
+      *reinterpret_cast<uint32_t*>(ph + r_hi * VLD + j) = wh;
+      *reinterpret_cast<uint32_t*>(pl + r_hi * VLD + j) = wl;
     }
   }
   const uint32_t* St = a.chunks + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
   const float f_lo = pw[r_lo + 1], f_hi = pw[r_hi + 1];
-  float o[NS][8][4];
+  float o[NS][4][4];
   float ss_lo = 0.f, ss_hi = 0.f;
 #pragma unroll
   for (int sl = 0; sl < NS; ++sl) {
@@ -798,10 +800,10 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
       }
     }
     __syncthreads();
-    float (&oc)[8][4] = o[sl];
+    float (&oc)[4][4] = o[sl];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) oc[i][0] = oc[i][1] = oc[i][2] = oc[i][3] = 0.f;
-    if (!busy) continue;
+    for (int i = 0; i < 4; ++i) oc[i][0] = oc[i][1] = oc[i][2] = oc[i][3] = 0.f;
+    if (!busy || c0 + side * 32 >= a.dv) continue;
 #pragma unroll
     for (int kk = 0; kk < DKP / 16; ++kk) {
       if (kk * 16 >= a.dk) continue;
@@ -809,9 +811,9 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
       ldsm4(qh + q_at + kk * 16, ah);
       ldsm4(ql + q_at + kk * 16, al);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
+      for (int np = 0; np < 2; ++np) {
         uint32_t bh[4], bl[4];
-        const int at = (kk * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + np * 16 + 8 * (lane / 16);
+        const int at = (kk * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + side * 32 + np * 16 + 8 * (lane / 16);
         ldsm4_t(kh + at, bh);
         ldsm4_t(kl + at, bl);
         mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
@@ -819,22 +821,26 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) { oc[i][0] *= f_lo; oc[i][1] *= f_lo; oc[i][2] *= f_hi; oc[i][3] *= f_hi; }
+    for (int i = 0; i < 4; ++i) { oc[i][0] *= f_lo; oc[i][1] *= f_lo; oc[i][2] *= f_hi; oc[i][3] *= f_hi; }
 #pragma unroll
     for (int kb = 0; kb < 4; ++kb) {
-      if (kb > warp) continue;
+      if (kb > rb) continue;
+      uint32_t ah[4], al[4];
+      const int pat = (rb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + kb * 16 + 8 * (lane / 16);
+      ldsm4(ph + pat, ah);
+      ldsm4(pl + pat, al);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
+      for (int np = 0; np < 2; ++np) {
         uint32_t bh[4], bl[4];
-        const int at = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + np * 16 + 8 * (lane / 16);
+        const int at = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + side * 32 + np * 16 + 8 * (lane / 16);
         ldsm4_t(vh + at, bh);
         ldsm4_t(vl + at, bl);
-        mma_terms(oc[2 * np], ph[kb], pl[kb], bh[0], bh[1], bl[0], bl[1]);
-        mma_terms(oc[2 * np + 1], ph[kb], pl[kb], bh[2], bh[3], bl[2], bl[3]);
+        mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+        mma_terms(oc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {                  // (columns beyond dv are zero)
+    for (int i = 0; i < 4; ++i) {                  // (columns beyond dv are zero)
       ss_lo = fmaf(oc[i][0], oc[i][0], fmaf(oc[i][1], oc[i][1], ss_lo));
       ss_hi = fmaf(oc[i][2], oc[i][2], fmaf(oc[i][3], oc[i][3], ss_hi));
     }
@@ -843,27 +849,33 @@ __global__ void __launch_bounds__(CK_THREADS) retention_chunk_out_kernel(RetArgs
   ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
   ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 1);
   ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 2);
-  const float n_lo = rsqrtf(ss_lo / (float)a.dv + a.eps), n_hi = rsqrtf(ss_hi / (float)a.dv + a.eps);
+  if (tq == 0) {
+    squares[side][r_lo] = ss_lo;
+    squares[side][r_hi] = ss_hi;
+  }
+  __syncthreads();
+  const float n_lo = rsqrtf((squares[0][r_lo] + squares[1][r_lo]) / (float)a.dv + a.eps);
+  const float n_hi = rsqrtf((squares[0][r_hi] + squares[1][r_hi]) / (float)a.dv + a.eps);
 #pragma unroll
   for (int sl = 0; sl < NS; ++sl)
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int col = sl * 64 + i * 8 + 2 * tq;
-      if (col >= a.dv) continue;
+    for (int half = 0; half < 2; ++half) {
+      const int r = half ? r_hi : r_lo;
+      if (r >= n) continue;
+      const float rn = half ? n_hi : n_lo;
+      const float* gp = a.proj + (size_t)(row0 + r) * a.ld + a.g0 + (size_t)h * a.dv;
+      const size_t at = ((size_t)(row0 + r) * a.H + h) * a.dv;
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int r = half ? r_hi : r_lo;
-        if (r >= n) continue;
-        const float rn = half ? n_hi : n_lo;
-        const float* gp = a.proj + (size_t)(row0 + r) * a.ld + a.g0 + (size_t)h * a.dv + col;
-        const size_t at = ((size_t)(row0 + r) * a.H + h) * a.dv + col;
+      for (int i = 0; i < 4; ++i) {
+        const int col = sl * 64 + side * 32 + i * 8 + 2 * tq;
+        if (col >= a.dv) continue;
         const float x = o[sl][i][2 * half] * rn, y = o[sl][i][2 * half + 1] * rn;
         if (a.v2 && a.out_dt == NV_DT_BF16) {
-          const float2 gg = *reinterpret_cast<const float2*>(gp);
-          *reinterpret_cast<__nv_bfloat162*>((bf16*)a.out + at) = __floats2bfloat162_rn(x * silu_of(gg.x), y * silu_of(gg.y));
+          const float2 gg = *reinterpret_cast<const float2*>(gp + col);
+          *reinterpret_cast<__nv_bfloat162*>((bf16*)a.out + at + col) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
         } else {
-          st_dt(a.out, a.out_dt, at, x * silu_of(gp[0]));
-          if (col + 1 < a.dv) st_dt(a.out, a.out_dt, at + 1, y * silu_of(gp[1]));
+          st_dt(a.out, a.out_dt, at + col, x * silu_fast(gp[col]));
+          if (col + 1 < a.dv) st_dt(a.out, a.out_dt, at + col + 1, y * silu_fast(gp[col + 1]));
         }
       }
     }
@@ -886,7 +898,7 @@ size_t chunk_sum_smem() { return sizeof(bf16) * (2 * (size_t)RC * (DKP + 8) + 2 
 template <int DKP>
 size_t chunk_out_smem() {
   const size_t ks = std::max((size_t)RC * (DKP + 8), (size_t)DKP * VLD);
-  return sizeof(bf16) * (2 * (size_t)RC * (DKP + 8) + 2 * ks + 2 * (size_t)RC * VLD);
+  return sizeof(bf16) * (2 * (size_t)RC * (DKP + 8) + 2 * ks + 4 * (size_t)RC * VLD);
 }
 
 template <int DKP, int NS>
