@@ -274,7 +274,11 @@ NV_API int nv_stream_mix_norm(float* x, int T, int S, int H, const float* branch
   const int chunks = H / vec;
   int threads = 32;
   if (kind == 2) {
-    while (threads < SM_RMS_THREADS && threads < chunks) threads *= 2;
+    // Few rows: as many threads as the row has chunks.  Many rows: smaller blocks, of which more share a multiprocessor,
+    // so that one's reduction runs beside another's loads (16,384 rows of two copies of 2,048: 160 -> 133 us); the sum
+    // of squares is then added up in another order, which is all that a row's result may differ by.
+    const int most = T > 512 ? SM_RMS_THREADS / 2 : SM_RMS_THREADS;
+    while (threads < most && threads < chunks) threads *= 2;
     const size_t smem = sizeof(float) * (size_t)vec * (size_t)(chunks > threads ? chunks - threads : 0);
     if (smem > 160 * 1024) return NV_ERR_UNSUPPORTED;
 #define NV_STREAM_RMS(VEC, SMAX)                                                                                          \
