@@ -326,7 +326,8 @@ __global__ void __launch_bounds__((WARPS + 1) * 32) attention_decode_kernel(DecA
 }
 
 // ---------------------------------------------------------------------------------------------
-// The tensor-core form, for bfloat16 caches whose head dimension is a multiple of 64.
+// The tensor-core form, for bfloat16 caches whose head dimension is a multiple of 16 from 64 on.  Between two multiples of 64
+// the next larger form runs: the boxes reach beyond the pages' rows there and are filled with zeros.
 //
 // The lane-per-chunk kernel above spends a few hundred instructions per key and page, and on this
 // GPU the instruction issue rate, not memory, then bounds it at about half of the memory speed.
@@ -356,7 +357,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 
 constexpr int TC_ROWS = 16;      // query heads per block (rows of the MMA)
 
-// D: head dimension, a multiple of 64 (compile time: it sizes the fragments).
+// D: head dimension rounded up to a multiple of 64 (compile time: it sizes the fragments); a.D: the head's own elements.
 template <int D, int TERMS>
 __global__ void __launch_bounds__((WARPS + 1) * 32, D <= 128 ? 3 : 1)
 attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
@@ -411,7 +412,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
     for (int i = threadIdx.x; i < TC_ROWS * D; i += WARPS * 32) {
       const int g = i / D, d = i % D;
       float v = 0.f;
-      if (g < ng) v = ld_dt(a.qkv, a.q_dt, (size_t)t * a.q_stride + (size_t)(kvh * G + g0 + g) * D + d);
+      if (g < ng && d < a.D) v = ld_dt(a.qkv, a.q_dt, (size_t)t * a.q_stride + (size_t)(kvh * G + g0 + g) * a.D + d);
       q_s[g * QLD + d] = __float2bfloat16_rn(v);
     }
     asm volatile("bar.sync 1, %0;" ::"n"(WARPS * 32) : "memory");      // the consumer warps only
@@ -597,6 +598,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
   // merge the warps (fixed order) and write this split's result; scores are in log2 units here
   for (int i = threadIdx.x; i < ng * D; i += (WARPS + 1) * 32) {
     const int gg = i / D, d = i % D;
+    if (d >= a.D) continue;
     float mm = mrg_m[0][gg];
 #pragma unroll
     for (int w = 1; w < WARPS; ++w) mm = fmaxf(mm, mrg_m[w][gg]);
@@ -610,17 +612,17 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
     }
     const int h = kvh * G + g0 + gg;
     if (a.splits == 1) {
-      st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * D + d, ll > 0.f ? ov / ll * head_gate_of(a.gate, t, h) : 0.f);
+      st_dt(a.out, a.out_dt, ((size_t)t * a.Hq + h) * a.D + d, ll > 0.f ? ov / ll * head_gate_of(a.gate, t, h) : 0.f);
     } else {
       const size_t pi = ((size_t)r * a.Hq + h) * a.splits + split;
-      a.part_o[pi * D + d] = ov;
+      a.part_o[pi * a.D + d] = ov;
       if (d == 0) {                                             // the merge kernel works in natural-log units
         a.part_ml[pi * 2] = mm == -INFINITY ? -1e30f : mms * 0.6931471805599453f;
         a.part_ml[pi * 2 + 1] = ll;
       }
     }
   }
-  if (a.splits > 1 && a.split_count) merge_when_last(a, r, t, kvh * G + g0, ng, D);
+  if (a.splits > 1 && a.split_count) merge_when_last(a, r, t, kvh * G + g0, ng, a.D);
 }
 
 // Combines the splits of one (row, head) in split order.
@@ -669,9 +671,9 @@ int launch_decode_tc(DecArgs a, int R, const void* kc, const void* vc, int num_p
   const int G = a.Hq / a.Hkv;
   CUtensorMap tm_k, tm_v;
   const long long rows = (long long)num_pages * a.Hkv * a.page;
-  int rc = nv_tensor_map_bf16(kc, rows, D, D, a.page, &tm_k);
+  int rc = nv_tensor_map_bf16(kc, rows, a.D, a.D, a.page, &tm_k);
   if (rc) return rc;
-  rc = nv_tensor_map_bf16(vc, rows, D, D, a.page, &tm_v);
+  rc = nv_tensor_map_bf16(vc, rows, a.D, a.D, a.page, &tm_v);
   if (rc) return rc;
   a.scale = scale * 1.4426950408889634f;            // the kernel works in log2 units
   const size_t ring = (size_t)a.stages * (a.same_kv ? 1 : 2) * a.page * D * 2;
@@ -792,29 +794,30 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
   // A ring of up to 64 KB: with pages of 16 keys of 128 elements that is eight stages, two per warp, so that a warp's
   // next page is on its way while it works on one (with one stage per warp a warp sat out the whole memory latency
   // between two pages), and three CTAs of 76 KB still share a multiprocessor.  Deeper rings lose CTAs and time.
-  int tc_stages = stages / WARPS * WARPS;
+  const int DT = (D + 63) / 64 * 64;               // the form's head dimension
+  int tc_stages = decode_stages(page, DT, esize) / WARPS * WARPS;
   a.same_kv = 0;
   if (kc == vc && cache_dt == NV_DT_BF16) {        // one array is keys and values: a page is fetched once
-    long long s2 = (64 * 1024) / ((long long)page * D * esize);
+    long long s2 = (64 * 1024) / ((long long)page * DT * esize);
     if (s2 > MAX_STAGES) s2 = MAX_STAGES;
     if (s2 / WARPS * WARPS >= WARPS) {
       tc_stages = (int)(s2 / WARPS * WARPS);
       a.same_kv = 1;
     }
   }
-  if (cache_dt == NV_DT_BF16 && D % 64 == 0 && page <= 256 && num_pages > 0 && tc_stages >= WARPS && !has_sink && !(softcap > 0.f)) {
+  if (cache_dt == NV_DT_BF16 && D >= 64 && D % 16 == 0 && page <= 256 && num_pages > 0 && tc_stages >= WARPS && !has_sink && !(softcap > 0.f)) {
     a.stages = tc_stages;
     // tensor-core form (a page of keys per warp); its blocks take up to 16 query heads of a kv head; with
     // float_weights the weights enter the product with the values as three bfloat16 terms
     if (float_weights)
-      rc = D == 64 ? launch_decode_tc<64, 3>(a, R, kc, vc, num_pages, scale, stream)
-         : D == 128 ? launch_decode_tc<128, 3>(a, R, kc, vc, num_pages, scale, stream)
-         : D == 192 ? launch_decode_tc<192, 3>(a, R, kc, vc, num_pages, scale, stream)
+      rc = DT == 64 ? launch_decode_tc<64, 3>(a, R, kc, vc, num_pages, scale, stream)
+         : DT == 128 ? launch_decode_tc<128, 3>(a, R, kc, vc, num_pages, scale, stream)
+         : DT == 192 ? launch_decode_tc<192, 3>(a, R, kc, vc, num_pages, scale, stream)
                     : launch_decode_tc<256, 3>(a, R, kc, vc, num_pages, scale, stream);
     else
-      rc = D == 64 ? launch_decode_tc<64, 1>(a, R, kc, vc, num_pages, scale, stream)
-         : D == 128 ? launch_decode_tc<128, 1>(a, R, kc, vc, num_pages, scale, stream)
-         : D == 192 ? launch_decode_tc<192, 1>(a, R, kc, vc, num_pages, scale, stream)
+      rc = DT == 64 ? launch_decode_tc<64, 1>(a, R, kc, vc, num_pages, scale, stream)
+         : DT == 128 ? launch_decode_tc<128, 1>(a, R, kc, vc, num_pages, scale, stream)
+         : DT == 192 ? launch_decode_tc<192, 1>(a, R, kc, vc, num_pages, scale, stream)
                     : launch_decode_tc<256, 1>(a, R, kc, vc, num_pages, scale, stream);
   } else if (cache_dt == NV_DT_BF16) {
     a.same_kv = 0;

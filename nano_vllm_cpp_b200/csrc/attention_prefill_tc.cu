@@ -27,8 +27,12 @@
 // 384 columns of tensor memory and 177 KB of shared memory (209 KB with three terms), so one CTA lives on a
 // multiprocessor.
 //
-// Takes bfloat16, head_dim 64, 128 or 256, pages of 16, 32 or 64 keys; everything else goes to the mma.sync kernel
-// (attention_prefill.cu), which is also this kernel's twin in the tests.  (The reference's kernel:
+// A head size between these (a multiple of 16) runs the next larger form: the boxes of keys and values reach beyond the
+// pages' rows there and are filled with zeros, so what the query boxes read of the next head meets zeros, and the
+// output's columns beyond the head are not stored.
+//
+// Takes bfloat16, head_dim 64 or a multiple of 16 up to 256 beyond it, pages of 16, 32 or 64 keys; everything else goes to
+// the mma.sync kernel (attention_prefill.cu), which is also this kernel's twin in the tests.  (The reference's kernel:
 // src/hip_ops.hip:473-551.)
 #include "tcgen05.cuh"
 
@@ -54,6 +58,7 @@ struct PtArgs {
   float sink_log2;          // the sink's score times log2(e)
   HeadGate gate;            // multiplies a head's output as it is written
   int S, max_blocks, window, Hq, Hkv, page;
+  int D;                    // elements of a head: the form's own number or fewer
   int min_rows;             // entries with fewer rows are left to another kernel
   int first_wave;           // CTAs that start alone on a multiprocessor (their number), before the second ones join them
 };
@@ -164,7 +169,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       if (lane == 0) {
         mbar_expect_tx(&q_full, SL * Q_SLAB);
 #pragma unroll
-        for (int s = 0; s < SL; ++s) tma_load_2d(Qs + s * Q_SLAB, &tm_q, &q_full, h * D + s * 64, row0);
+        for (int s = 0; s < SL; ++s) tma_load_2d(Qs + s * Q_SLAB, &tm_q, &q_full, h * a.D + s * 64, row0);
       }
       const int pages = TKB >> page_shift;
       const uint32_t box = (uint32_t)a.page * 128;
@@ -350,9 +355,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         float o[32];
         tmem_ld32(tmem_o + lane_off + c * 32, o);
         if (live) {
-          bf16* dst = a.out + ((size_t)(row0 + r) * a.Hq + h) * D + c * 32;
+          bf16* dst = a.out + ((size_t)(row0 + r) * a.Hq + h) * a.D + c * 32;
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
+            if (c * 32 + j >= a.D) continue;
             uint4 v;
             __nv_bfloat162 t0 = __floats2bfloat162_rn(o[j + 0] * inv, o[j + 1] * inv);
             __nv_bfloat162 t1 = __floats2bfloat162_rn(o[j + 2] * inv, o[j + 3] * inv);
@@ -377,9 +383,9 @@ int launch_prefill_tc(const PtArgs& a, const void* qkv, int q_stride, int T, con
   int rc = nv_tensor_map_bf16(qkv, T, q_stride, q_stride, TQ, &tm_q);
   if (rc) return rc;
   const long long rows = (long long)num_pages * a.Hkv * a.page;
-  rc = nv_tensor_map_bf16(kc, rows, D, D, a.page, &tm_k);
+  rc = nv_tensor_map_bf16(kc, rows, a.D, a.D, a.page, &tm_k);
   if (rc) return rc;
-  rc = nv_tensor_map_bf16(vc, rows, D, D, a.page, &tm_v);
+  rc = nv_tensor_map_bf16(vc, rows, a.D, a.D, a.page, &tm_v);
   if (rc) return rc;
   constexpr int SL = D / 64;
   const size_t smem = (size_t)SL * TQ * 128 + 3 * (size_t)SL * TKB * 128 + (size_t)TERMS * TQ * 128 + 1024;
@@ -398,7 +404,7 @@ int launch_prefill_tc(const PtArgs& a, const void* qkv, int q_stride, int T, con
 }  // namespace
 
 NV_API int nv_attention_prefill_tc_usable(int D, int page) {
-  return (D == 64 || D == 128 || D == 256) && (page == 16 || page == 32 || page == 64);
+  return D >= 64 && D <= 256 && D % 16 == 0 && (page == 16 || page == 32 || page == 64);
 }
 
 // Same contract as nv_attention_prefill (max_tiles counts tiles of nv_attention_prefill_tile_rows() = 64 rows, an
@@ -435,13 +441,14 @@ NV_API int nv_attention_prefill_tc(const void* qkv, int q_stride, int T, const v
       num_sms = 148;
   }
   a.first_wave = num_sms;
+  a.D = D;
   const int tiles = (max_tiles + S + 1) / 2;
   if (weight_terms == 3) {
     if (D == 64) return launch_prefill_tc<64, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
-    if (D == 256) return launch_prefill_tc<256, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
+    if (D > 128) return launch_prefill_tc<256, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
     return launch_prefill_tc<128, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
   }
   if (D == 64) return launch_prefill_tc<64, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
-  if (D == 256) return launch_prefill_tc<256, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
+  if (D > 128) return launch_prefill_tc<256, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
   return launch_prefill_tc<128, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
 }

@@ -437,7 +437,12 @@ ATTENTIONS = [ps.attention_layer(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2
               ps.attention_layer(heads=20, kv_heads=1, dim=64, vdim=32, scale=0.12),
               ps.attention_layer(heads=2, kv_heads=1, dim=256, vdim=256, scale=0.06),
               ps.attention_layer(heads=2, kv_heads=1, dim=192, vdim=80, scale=0.07),
-              ps.attention_layer(heads=1, kv_heads=1, dim=8, vdim=16, scale=0.5)]
+              ps.attention_layer(heads=1, kv_heads=1, dim=8, vdim=16, scale=0.5),
+              # between the sizes that the tensor-core forms are made for: the next larger form, its rest filled with zeros
+              ps.attention_layer(heads=4, kv_heads=2, dim=80, vdim=80, scale=0.11),
+              ps.attention_layer(heads=3, kv_heads=3, dim=112, vdim=104, scale=0.1),
+              ps.attention_layer(heads=17, kv_heads=1, dim=144, vdim=136, scale=0.08),
+              ps.attention_layer(heads=2, kv_heads=2, dim=208, vdim=208, scale=0.07)]
 PAGES = [[7, 3, 11, 0, 9], [5, 2, 8, 10]]
 
 
@@ -489,7 +494,7 @@ def test_keys_and_values_of_another_layer(layer, dtype):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("decoded", [False, True])
 @pytest.mark.parametrize("dim,i,j", [(32, 50, 0), (32, 50, 15), (32, 50, 16), (32, 330, 1), (64, 330, 127), (64, 330, 128),
-                                     (64, 700, 0), (128, 300, 63), (96, 500, 64), (96, 333, 2)])
+                                     (64, 700, 0), (128, 300, 63), (96, 500, 64), (96, 333, 2), (80, 400, 65), (176, 290, 17)])
 def test_one_key_stands_out(dim, i, j, decoded, dtype):
     """Row i's softmax falls in halves on key j and on itself (row j's input is row i's plus something that the key
     projection does not see, so its key is the same and its value another): the first tokens, page and tile borders,
