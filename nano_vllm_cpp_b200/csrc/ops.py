@@ -460,8 +460,8 @@ def attention_prefill(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, m
                       window: int, out, Hq: int, Hkv: int, D: int, err=None, min_rows: int = 1,
                       kernel: str = "auto", sink_score=None, weight_terms: int = 1, softcap: float = 0.0,
                       gate=None) -> None:
-    """bfloat16 rows of any mix of portions against their paged keys: the tcgen05 kernel for head sizes 64 and
-    128 and pages of 16, 32 or 64 keys, else the mma.sync kernel (``kernel="mma"`` asks for that one).  Entries
+    """bfloat16 rows of any mix of portions against their paged keys: the tcgen05 kernel for head sizes from
+    64 to 256 (multiples of 16) and pages of 16, 32 or 64 keys, else the mma.sync kernel (``kernel="mma"`` asks for that one).  Entries
     with fewer than ``min_rows`` rows are skipped and their rows of ``out`` left as they are.
     ``weight_terms`` = 3: the float32 weights enter the product with the values as three bfloat16 terms, all their
     bits (either kernel).  ``sink_score``: a further key with that score and no value in every softmax; ``softcap``
