@@ -3,7 +3,7 @@
 For every call of the model's order that owns a cache entry there is a pair of tensors ``k, v`` shaped
 ``[pages, kv_heads, page_size, head_dim]`` (values may have a head size of their own) — a page's rows of one
 head are contiguous —, or a state tensor ``[slots, *shape]``, or several of these for a mixer that keeps several
-things (``CompositeCacheSpec``: its view holds one view per part).  Calls whose attention has the same window
+things (``CompositeCacheSpec``: its view holds one view per part).  Calls whose attention has the same window or chunk size
 form a group and share page ids (the same page index addresses the same slice in each of them, as in the
 reference's pool: src/model.cpp:642-645).  All state arrays of a dtype are slices of one buffer ``[slots,
 words]``, so that a request's whole state is one stretch of memory and one launch zeroes it.
@@ -36,7 +36,9 @@ class CacheView:
 
 def _group_key(spec: KVCacheSpec):
     """What layers must share to share page ids: the window, and with a window the number of first positions that
-    stay readable behind it."""
+    stay readable behind it; or the chunk size."""
+    if spec.chunk > 0:
+        return ("chunk", spec.chunk)
     return (spec.window, spec.keep_first) if spec.window > 0 and spec.keep_first > 0 else spec.window
 
 
@@ -53,7 +55,7 @@ class DeviceCache:
     def __init__(self, cache_specs: list, page_size: int, max_slots: int, device, dtype):
         self.page_size, self.device, self.dtype, self.max_slots = page_size, device, dtype, max_slots
         self.specs = cache_specs
-        self.windows: list = []                    # one per group: the window, or (window, kept first positions)
+        self.windows: list = []                    # one per group: the window, (window, kept first positions) or ("chunk", size)
         for s in cache_specs:
             for leaf in _leaves(s):
                 if isinstance(leaf, KVCacheSpec) and _group_key(leaf) not in self.windows:

@@ -3,8 +3,9 @@
 The class lives in native code (csrc/host_core.cpp, ``CacheManager``); this is its Python face.
 Layers with the same needs form a *group* with pages and block tables of its own: one group for
 layers that read every earlier key, one for each window size (and number of first positions that stay
-readable behind the window).  A group with a window gives a page back as soon as every position in it lies
-before the window of the next row to run, unless the page holds one of the kept first positions.  A
+readable behind the window), one for each chunk size.  A group with a window gives a page back as soon as every position in it lies
+before the window of the next row to run, unless the page holds one of the kept first positions; a group with
+chunks gives a page back once the next row to run lies in a later chunk than all of the page.  A
 request also holds one *state slot* (an index into fixed-size per-request arrays) from ``open``
 to ``close``.
 
@@ -70,23 +71,30 @@ class CacheManager:
     def __init__(self, windows: list, num_pages, page_size: int, max_requests: int,
                  prefix_caching: bool = False, has_state: bool = False):
         """``windows``: one entry per group (0 = reads every key; ``(window, keep_first)`` for a window behind which
-        the first ``keep_first`` positions stay readable); it may be empty for a model without paged
+        the first ``keep_first`` positions stay readable; ``("chunk", n)``: a row reads the positions of its own chunk
+        of n, counted from the sequence's start); it may be empty for a model without paged
         layers, whose requests hold a state slot and nothing else.  ``num_pages``: an int for all groups or a
         list.  ``has_state``: some layer keeps a fixed-size state per request; prefix sharing is then refused
         (a request that adopted another's pages would skip tokens its state never saw)."""
         if isinstance(num_pages, int):
             num_pages = [num_pages] * len(windows)
-        self.keeps = [int(w[1]) if isinstance(w, (tuple, list)) else 0 for w in windows]
-        self.windows = [int(w[0]) if isinstance(w, (tuple, list)) else int(w) for w in windows]
+        self.windows, self.keeps, self.chunks = [], [], []
+        for w in windows:
+            pair = isinstance(w, (tuple, list))
+            chunked = pair and w[0] == "chunk"
+            self.chunks.append(int(w[1]) if chunked else 0)
+            self.windows.append(0 if chunked else int(w[0]) if pair else int(w))
+            self.keeps.append(int(w[1]) if pair and not chunked else 0)
         self.page_size = page_size
         self.max_requests = max_requests
         self.num_groups = len(windows)
         w, _ = host.ints(self.windows)
         n, _ = host.ints(list(num_pages))
         k, _ = host.ints(self.keeps)
+        c, _ = host.ints(self.chunks)
         L = host.lib()
         self._h = L.nvh_manager_create(w, n, self.num_groups, page_size, max_requests, 1 if prefix_caching else 0,
-                                       1 if has_state else 0, k)
+                                       1 if has_state else 0, k, c)
         self.pools = [BlockPool(num_pages[g], page_size, _handle=L.nvh_manager_pool(self._h, g))
                       for g in range(self.num_groups)]
         self.prefix_caching = bool(L.nvh_manager_prefix_caching(self._h))

@@ -71,6 +71,9 @@ struct DecArgs {
   int has_sink;           // the softmax's denominator also holds exp(sink): a key with that score and no value
   float sink;             // (the lane-per-chunk kernel and the merges add it; the tensor-core form does not know it)
   HeadGate gate;          // multiplies a head's output where its final value is written (here or in the merge)
+  int chunk;              // > 0: a row sees its own chunk of so many positions (and there is no window)
+  ScoreBias bias;         // what the distance gives to a score, after the cap
+  ScoreMap map;           // MOD kernels: how a raw score becomes a capped one in base-2 units
 };
 
 // Called by every thread of a block once the block has written its split's partial results for the query heads
@@ -130,7 +133,7 @@ __global__ void __launch_bounds__((WARPS + 1) * 32) attention_decode_kernel(DecA
   const int D = a.D, chunks = D / 8;
 
   const int n = a.positions[t] + 1;
-  const int lo = a.window > 0 ? max(0, n - a.window) : 0;
+  const int lo = first_visible(n - 1, a.window, a.chunk);
   // this split's pages
   const int p_lo = lo / a.page, p_hi = (n - 1) / a.page + 1;
   const int per = (p_hi - p_lo + a.splits - 1) / a.splits;
@@ -239,6 +242,7 @@ __global__ void __launch_bounds__((WARPS + 1) * 32) attention_decode_kernel(DecA
           sc += __shfl_xor_sync(0xffffffffu, sc, 4);
           if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
           if (live) {
+            if (a.bias.slope || a.bias.table) sc += score_bias_of(a.bias, kvh * G + g0 + g, n - 1 - j);
             if (sc > m[g]) {                       // a new maximum (rare after the first keys): rescale what was summed
               const float alpha = __expf(m[g] - sc);
               l[g] *= alpha;
@@ -326,7 +330,7 @@ __global__ void __launch_bounds__((WARPS + 1) * 32) attention_decode_kernel(DecA
 }
 
 // ---------------------------------------------------------------------------------------------
-// The tensor-core form, for bfloat16 caches whose head dimension is a multiple of 16 from 64 on.  Between two multiples of 64
+// The tensor-core form, for bfloat16 caches whose head dimension is a multiple of 16 from 32 on.  Between two multiples of 64
 // the next larger form runs: the boxes reach beyond the pages' rows there and are filled with zeros.
 //
 // The lane-per-chunk kernel above spends a few hundred instructions per key and page, and on this
@@ -358,7 +362,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 constexpr int TC_ROWS = 16;      // query heads per block (rows of the MMA)
 
 // D: head dimension rounded up to a multiple of 64 (compile time: it sizes the fragments); a.D: the head's own elements.
-template <int D, int TERMS>
+// MOD: scores pass a cap and a bias by distance; they are then in base-2 units (and a.scale is 1).
+template <int D, int TERMS, bool MOD>
 __global__ void __launch_bounds__((WARPS + 1) * 32, D <= 128 ? 3 : 1)
 attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                            DecArgs a) {
@@ -381,7 +386,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
 
   const int n = a.positions[t] + 1;
-  const int lo = a.window > 0 ? max(0, n - a.window) : 0;
+  const int lo = first_visible(n - 1, a.window, a.chunk);
   const int p_lo = lo / a.page, p_hi = (n - 1) / a.page + 1;
   const int per = (p_hi - p_lo + a.splits - 1) / a.splits;
   const int pb = p_lo + split * per;
@@ -467,6 +472,12 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
     int s = warp % a.stages;                       // stage of page i (the ring is a multiple of WARPS stages deep)
     uint32_t ph = (warp / a.stages) & 1;
     const uint32_t smem0 = smem_u32(dec_smem);
+    // MOD: this thread's rows of the tile are the query heads g and g + 8
+    const int h_lo = kvh * G + g0 + min(g, ng - 1), h_hi = kvh * G + g0 + min(g + 8, ng - 1);
+    const float slope_lo = MOD && a.bias.slope ? a.bias.slope[h_lo] * 1.4426950408889634f : 0.f;
+    const float slope_hi = MOD && a.bias.slope ? a.bias.slope[h_hi] * 1.4426950408889634f : 0.f;
+    const float* tab_lo = MOD && a.bias.table ? a.bias.table + (size_t)h_lo * (a.bias.last + 1) : nullptr;
+    const float* tab_hi = MOD && a.bias.table ? a.bias.table + (size_t)h_hi * (a.bias.last + 1) : nullptr;
     for (int i = warp; i < n_pages; i += WARPS) {
       mbar_wait(&full_bar[s], ph, a.err, 0x7112);
       const uint32_t kbase = smem0 + (uint32_t)s * stage_bytes;
@@ -494,6 +505,27 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
             for (int u = 0; u < 4; ++u) {
               mma16816(s0, qa[k4 * 4 + u], b[u][0], b[u][1]);
               mma16816(s1, qa[k4 * 4 + u], b[u][2], b[u][3]);
+            }
+          }
+        }
+        if (MOD) {
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const int na = n - 1 - (j0 + 2 * tq + c), nb = na - 8;         // distances (negative ones are masked below)
+            if (a.map.cap1 > 0.f) {
+              s0[c] = capped_log2(a.map, s0[c]); s0[2 + c] = capped_log2(a.map, s0[2 + c]);
+              s1[c] = capped_log2(a.map, s1[c]); s1[2 + c] = capped_log2(a.map, s1[2 + c]);
+            } else {
+              s0[c] *= a.map.in; s0[2 + c] *= a.map.in; s1[c] *= a.map.in; s1[2 + c] *= a.map.in;
+            }
+            s0[c] = fmaf(-slope_lo, (float)na, s0[c]); s0[2 + c] = fmaf(-slope_hi, (float)na, s0[2 + c]);
+            s1[c] = fmaf(-slope_lo, (float)nb, s1[c]); s1[2 + c] = fmaf(-slope_hi, (float)nb, s1[2 + c]);
+            if (tab_lo) {
+              const int ia = min(max(na, 0), a.bias.last), ib = min(max(nb, 0), a.bias.last);
+              s0[c] = fmaf(__ldg(tab_lo + ia), 1.4426950408889634f, s0[c]);
+              s0[2 + c] = fmaf(__ldg(tab_hi + ia), 1.4426950408889634f, s0[2 + c]);
+              s1[c] = fmaf(__ldg(tab_lo + ib), 1.4426950408889634f, s1[c]);
+              s1[2 + c] = fmaf(__ldg(tab_hi + ib), 1.4426950408889634f, s1[2 + c]);
             }
           }
         }
@@ -666,7 +698,7 @@ int launch_decode(const DecArgs& a, int R, int G, size_t smem, cudaStream_t s) {
   return G == 1 ? launch_decode_g<TC, CPL, 1>(a, R, G, smem, s) : launch_decode_g<TC, CPL, 4>(a, R, G, smem, s);
 }
 
-template <int D, int TERMS>
+template <int D, int TERMS, bool MOD>
 int launch_decode_tc(DecArgs a, int R, const void* kc, const void* vc, int num_pages, float scale, cudaStream_t s) {
   const int G = a.Hq / a.Hkv;
   CUtensorMap tm_k, tm_v;
@@ -675,24 +707,32 @@ int launch_decode_tc(DecArgs a, int R, const void* kc, const void* vc, int num_p
   if (rc) return rc;
   rc = nv_tensor_map_bf16(vc, rows, a.D, a.D, a.page, &tm_v);
   if (rc) return rc;
-  a.scale = scale * 1.4426950408889634f;            // the kernel works in log2 units
+  a.scale = MOD ? 1.f : scale * 1.4426950408889634f;            // the kernel works in log2 units
   const size_t ring = (size_t)a.stages * (a.same_kv ? 1 : 2) * a.page * D * 2;
   const size_t merge = (size_t)WARPS * TC_ROWS * D * sizeof(float);
   const size_t smem = (ring > merge ? ring : merge) + 1024;
   static bool attr_done = false;
   if (!attr_done) {
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_tc_kernel<D, TERMS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attention_decode_tc_kernel<D, TERMS, MOD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          160 * 1024);
     if (e != cudaSuccess) return (int)e;
     // three CTAs with a 64 KB ring each need nearly all of a multiprocessor's shared memory
-    e = cudaFuncSetAttribute(attention_decode_tc_kernel<D, TERMS>, cudaFuncAttributePreferredSharedMemoryCarveout,
+    e = cudaFuncSetAttribute(attention_decode_tc_kernel<D, TERMS, MOD>, cudaFuncAttributePreferredSharedMemoryCarveout,
                              cudaSharedmemCarveoutMaxShared);
     if (e != cudaSuccess) return (int)e;
     attr_done = true;
   }
   dim3 grid(R, a.Hkv * ((G + TC_ROWS - 1) / TC_ROWS), a.splits);
-  NV_RETURN_IF(launch_dep(attention_decode_tc_kernel<D, TERMS>, grid, dim3((WARPS + 1) * 32), smem, s, tm_k, tm_v, a));
+  NV_RETURN_IF(launch_dep(attention_decode_tc_kernel<D, TERMS, MOD>, grid, dim3((WARPS + 1) * 32), smem, s, tm_k, tm_v, a));
   NV_RETURN_LAST();
+}
+
+template <int TERMS, bool MOD>
+int launch_decode_tc_d(const DecArgs& a, int DT, int R, const void* kc, const void* vc, int num_pages, float scale, cudaStream_t s) {
+  return DT == 64 ? launch_decode_tc<64, TERMS, MOD>(a, R, kc, vc, num_pages, scale, s)
+       : DT == 128 ? launch_decode_tc<128, TERMS, MOD>(a, R, kc, vc, num_pages, scale, s)
+       : DT == 192 ? launch_decode_tc<192, TERMS, MOD>(a, R, kc, vc, num_pages, scale, s)
+                   : launch_decode_tc<256, TERMS, MOD>(a, R, kc, vc, num_pages, scale, s);
 }
 
 // Stages of the page ring for a page of `page` keys of `D` elements of `esize` bytes: as many as fit in
@@ -746,11 +786,13 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
                                const int* rows, int R, float scale, int window, void* out, int out_dt, int Hq,
                                int Hkv, int D, int page, int num_pages, int splits, float* scratch, int* err,
                                int* split_count, int split_count_len, int has_sink, float sink_score,
-                               int float_weights, float softcap, const float* gate, long long gate_ld,
-                               cudaStream_t stream) {
+                               int float_weights, float softcap, const float* gate, long long gate_ld, int chunk,
+                               const float* slopes, const float* bias_table, int bias_len, cudaStream_t stream) {
   // gate: head h's output of batch row t is multiplied by sigmoid(gate[t * gate_ld + h]) (nullptr: it is not); the
   // gates must have been written before the kernel that precedes this one on the stream.
-  // softcap > 0: scaled scores are capped, s -> softcap * tanh(s / softcap); like a sink it keeps the tensor-core form out.
+  // softcap > 0: scaled scores are capped, s -> softcap * tanh(s / softcap).  chunk > 0: a row at position p sees the
+  // positions from p / chunk * chunk on (and there is no window).  slopes [Hq]: head h's score with a key at distance n loses
+  // slopes[h] * n; bias_table [Hq, bias_len]: it gains bias_table[h][min(n, bias_len - 1)]; both after the cap.
   // has_sink: a further key with the score sink_score and no value in every softmax; it keeps the tensor-core form
   // out.  float_weights: the weights keep all their bits in their product with the values (the lane-per-chunk
   // kernel multiplies in float32; the tensor-core form takes them as three bfloat16 terms instead of one).
@@ -758,6 +800,7 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
   if (D <= 0 || D > 256 || D % 8 || Hkv <= 0 || Hq % Hkv || page % 16) return NV_ERR_UNSUPPORTED;
   const int esize = cache_dt == NV_DT_BF16 ? 2 : 4;
   const int stages = decode_stages(page, D, esize);
+  if (chunk < 0 || (chunk > 0 && window > 0) || (bias_table && bias_len < 1)) return NV_ERR_BAD_SIZE;
   if (stages == 0) return NV_ERR_UNSUPPORTED;          // a page of this size does not fit the ring twice
   if (((uintptr_t)kc & 15) || ((uintptr_t)vc & 15)) return NV_ERR_UNSUPPORTED;
   if (R == 0) return NV_OK;
@@ -773,6 +816,9 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
   a.has_sink = has_sink; a.sink = sink_score;
   a.softcap = softcap > 0.f ? softcap : 0.f;
   a.gate = HeadGate{gate, gate_ld};
+  a.chunk = chunk;
+  a.bias = ScoreBias{slopes, bias_table, bias_len - 1};
+  a.map = score_map(scale, a.softcap);
   // `split_count`: zeros (R * Hq of them are enough), kept zero from launch to launch by the kernel: the splits are
   // then added up by the block that finishes last instead of by a second kernel.  For a few rows only: with many,
   // the last blocks' sums lengthen the kernel's tail by more than the second kernel's launch costs (measured per
@@ -805,20 +851,17 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
       a.same_kv = 1;
     }
   }
-  if (cache_dt == NV_DT_BF16 && D >= 64 && D % 16 == 0 && page <= 256 && num_pages > 0 && tc_stages >= WARPS && !has_sink && !(softcap > 0.f)) {
+  if (cache_dt == NV_DT_BF16 && D >= 32 && D % 16 == 0 && page <= 256 && num_pages > 0 && tc_stages >= WARPS && !has_sink) {
     a.stages = tc_stages;
     // tensor-core form (a page of keys per warp); its blocks take up to 16 query heads of a kv head; with
     // float_weights the weights enter the product with the values as three bfloat16 terms
+    const bool mod = a.softcap > 0.f || slopes || bias_table;
     if (float_weights)
-      rc = DT == 64 ? launch_decode_tc<64, 3>(a, R, kc, vc, num_pages, scale, stream)
-         : DT == 128 ? launch_decode_tc<128, 3>(a, R, kc, vc, num_pages, scale, stream)
-         : DT == 192 ? launch_decode_tc<192, 3>(a, R, kc, vc, num_pages, scale, stream)
-                    : launch_decode_tc<256, 3>(a, R, kc, vc, num_pages, scale, stream);
+      rc = mod ? launch_decode_tc_d<3, true>(a, DT, R, kc, vc, num_pages, scale, stream)
+               : launch_decode_tc_d<3, false>(a, DT, R, kc, vc, num_pages, scale, stream);
     else
-      rc = DT == 64 ? launch_decode_tc<64, 1>(a, R, kc, vc, num_pages, scale, stream)
-         : DT == 128 ? launch_decode_tc<128, 1>(a, R, kc, vc, num_pages, scale, stream)
-         : DT == 192 ? launch_decode_tc<192, 1>(a, R, kc, vc, num_pages, scale, stream)
-                    : launch_decode_tc<256, 1>(a, R, kc, vc, num_pages, scale, stream);
+      rc = mod ? launch_decode_tc_d<1, true>(a, DT, R, kc, vc, num_pages, scale, stream)
+               : launch_decode_tc_d<1, false>(a, DT, R, kc, vc, num_pages, scale, stream);
   } else if (cache_dt == NV_DT_BF16) {
     a.same_kv = 0;
     rc = D <= 64 ? launch_decode<bf16, 1>(a, R, G, smem, stream)
@@ -891,7 +934,7 @@ NV_API int nv_attention_decode_noalloc(const void* qkv, int q_dt, int q_stride, 
   }
   return nv_attention_decode(qkv, q_dt, q_stride, kc, vc, cache_dt, block_table, max_blocks, row_entry, positions,
                              rows, R, scale, window, out, out_dt, Hq, Hkv, D, page, num_pages, splits,
-                             g_noalloc_ptr[dev], g_noalloc_err_ptr[dev], nullptr, 0, 0, 0.f, 0, 0.f, nullptr, 0, stream);
+                             g_noalloc_ptr[dev], g_noalloc_err_ptr[dev], nullptr, 0, 0, 0.f, 0, 0.f, nullptr, 0, 0, nullptr, nullptr, 0, stream);
 }
 
 NV_API int nv_attention_decode_noalloc_status(void) {

@@ -10,7 +10,7 @@
 // of two or three bfloat16 numbers, each term a product of its own into the same accumulators, so that with three
 // terms a weight enters with all the bits of the float.  A sink (a further key with a fixed score and no value)
 // is added to the softmax's denominator at the end.
-// Row at position p sees keys [max(0, p + 1 - window), p]; the mask is applied per element, so
+// Row at position p sees keys [max(0, p + 1 - window), p] (or from the start of its chunk on); the mask is applied per element, so
 // a tile may mix rows with different ranges.  The rows of this step are already in the cache when
 // the kernel runs, so a portion sees its own earlier rows there.
 //
@@ -35,7 +35,9 @@ struct PfArgs {
   int S, q_stride, max_blocks, window, Hq, Hkv, D, page;
   int min_rows;             // entries with fewer rows are left to another kernel
   float softcap, cap_in;    // softcap > 0: a score s becomes softcap * tanh(s * cap_in), cap_in = scale / softcap
-                            // (scale_log2 is then log2(e) alone)
+                            // (scale_log2 is then log2(e) alone, as it is with a bias)
+  ScoreBias bias;           // what the distance gives to a score, after the cap
+  int chunk;                // > 0: a row sees its own chunk of so many positions (and there is no window)
   int has_sink;             // the softmax's denominator also holds exp(sink): a key with that score and no value
   float sink_log2;          // the sink's score times log2(e)
   HeadGate gate;            // multiplies a head's output as it is written
@@ -107,7 +109,7 @@ __global__ void __launch_bounds__(BM * 2, DP <= 128 ? 2 : 1) attention_prefill_k
   const int row0 = tile_info[1], nrows = tile_info[2];
   const int pos0 = a.entry_pos0[e] + (row0 - a.cu_rows[e]);      // position of the tile's first row
   const int hi = pos0 + nrows;                                   // keys [.., hi) exist for this tile
-  const int lo = a.window > 0 ? max(0, pos0 + 1 - a.window) : 0; // first key any row of the tile sees
+  const int lo = first_visible(pos0, a.window, a.chunk);          // first key any row of the tile sees
   const int kv0 = lo / 16 * 16;
   const int n_tiles = (hi - kv0 + BN - 1) / BN;
   const int* bt = a.block_table + (size_t)e * a.max_blocks;
@@ -150,7 +152,7 @@ __global__ void __launch_bounds__(BM * 2, DP <= 128 ? 2 : 1) attention_prefill_k
   const int g = lane / 4, tq = lane % 4;
   const int r_lo = warp * 16 + g, r_hi = r_lo + 8;               // this thread's two rows in the tile
   const int p_lo = pos0 + r_lo, p_hi = pos0 + r_hi;
-  const int w_lo_lo = a.window > 0 ? p_lo + 1 - a.window : 0, w_lo_hi = a.window > 0 ? p_hi + 1 - a.window : 0;
+  const int w_lo_lo = first_visible(p_lo, a.window, a.chunk), w_lo_hi = first_visible(p_hi, a.window, a.chunk);
   const bool live_lo = r_lo < nrows, live_hi = r_hi < nrows;
 
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
@@ -171,7 +173,7 @@ __global__ void __launch_bounds__(BM * 2, DP <= 128 ? 2 : 1) attention_prefill_k
     // a warp whose 16 rows see none of this tile's keys (all later than its last row, or all before its
     // first row's window) only keeps the barriers
     const int warp_p_hi = pos0 + warp * 16 + 15, warp_p_lo = pos0 + warp * 16;
-    const bool warp_sees = j0 <= warp_p_hi && (a.window <= 0 || j0 + BN - 1 >= warp_p_lo + 1 - a.window) &&
+    const bool warp_sees = j0 <= warp_p_hi && j0 + BN - 1 >= first_visible(warp_p_lo, a.window, a.chunk) &&
                            warp * 16 < nrows;
     if (warp_sees) {
     // ---- S = Q K^T for this warp's 16 rows x 64 keys
@@ -203,8 +205,19 @@ __global__ void __launch_bounds__(BM * 2, DP <= 128 ? 2 : 1) attention_prefill_k
 #pragma unroll
         for (int c = 0; c < 4; ++c) s[nt][c] = a.softcap * tanhf(s[nt][c] * a.cap_in);
     }
+    if (a.bias.slope || a.bias.table) {
+      const float pre = a.softcap > 0.f ? 1.f : a.cap_in;          // (without a cap cap_in holds the scale)
+#pragma unroll
+      for (int nt = 0; nt < BN / 8; ++nt)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const int j = j0 + nt * 8 + 2 * tq + c;
+          s[nt][c] = fmaf(s[nt][c], pre, score_bias_of(a.bias, h, max(p_lo - j, 0)));
+          s[nt][2 + c] = fmaf(s[nt][2 + c], pre, score_bias_of(a.bias, h, max(p_hi - j, 0)));
+        }
+    }
     // ---- mask (only on tiles that some row of the warp sees partly), online softmax
-    const bool whole = j0 + BN - 1 <= warp_p_lo && (a.window <= 0 || j0 >= warp_p_hi + 1 - a.window) &&
+    const bool whole = j0 + BN - 1 <= warp_p_lo && j0 >= first_visible(warp_p_hi, a.window, a.chunk) &&
                        warp * 16 + 15 < nrows;
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
     if (!whole) {
@@ -372,22 +385,27 @@ int launch_prefill(const PfArgs& a, int max_tiles64, int num_sms, cudaStream_t s
 // ceil(rows / nv_attention_prefill_tile_rows()), the smallest tile the launcher may choose; surplus CTAs leave at once.
 // Entries with fewer than `min_rows` rows are skipped (their rows of `out` stay untouched): in a mixed step the
 // single rows go to the decode kernel.  gate: head h's output of row t is multiplied by sigmoid(gate[t * gate_ld + h]).
+// chunk, slopes, bias_table: see nv_attention_prefill_tc.
 NV_API int nv_attention_prefill_tile_rows() { return 64; }
 
 NV_API int nv_attention_prefill(const void* qkv, int q_stride, const void* kc, const void* vc,
                                 const int* block_table, int max_blocks, const int* cu_rows, const int* entry_pos0,
                                 int S, int max_tiles, float scale, int window, void* out, int Hq, int Hkv, int D,
                                 int page, int min_rows, int has_sink, float sink_score, int terms,
-                                float softcap, const float* gate, long long gate_ld, cudaStream_t stream) {
+                                float softcap, const float* gate, long long gate_ld, int chunk, const float* slopes,
+                                const float* bias_table, int bias_len, cudaStream_t stream) {
+  if (chunk < 0 || (chunk > 0 && window > 0) || (bias_table && bias_len < 1)) return NV_ERR_BAD_SIZE;
   if (D <= 0 || D > 256 || D % 16 || Hkv <= 0 || Hq % Hkv || (terms != 1 && terms != 3)) return NV_ERR_UNSUPPORTED;
   if (q_stride % 8 || ((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15)) return NV_ERR_UNSUPPORTED;
   if (S == 0 || max_tiles == 0) return NV_OK;
   PfArgs a;
   a.qkv = (const bf16*)qkv; a.kc = (const bf16*)kc; a.vc = (const bf16*)vc; a.block_table = block_table;
   a.cu_rows = cu_rows; a.entry_pos0 = entry_pos0; a.out = (bf16*)out;
-  a.scale_log2 = (softcap > 0.f ? 1.f : scale) * 1.4426950408889634f;
+  a.scale_log2 = (softcap > 0.f || slopes || bias_table ? 1.f : scale) * 1.4426950408889634f;
   a.softcap = softcap > 0.f ? softcap : 0.f;
-  a.cap_in = softcap > 0.f ? scale / softcap : 0.f;
+  a.cap_in = softcap > 0.f ? scale / softcap : scale;
+  a.bias = ScoreBias{slopes, bias_table, bias_len - 1};
+  a.chunk = chunk;
   a.S = S; a.q_stride = q_stride; a.max_blocks = max_blocks; a.window = window; a.Hq = Hq; a.Hkv = Hkv; a.D = D;
   a.page = page;
   a.min_rows = min_rows;

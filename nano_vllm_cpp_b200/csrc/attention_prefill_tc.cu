@@ -31,7 +31,7 @@
 // pages' rows there and are filled with zeros, so what the query boxes read of the next head meets zeros, and the
 // output's columns beyond the head are not stored.
 //
-// Takes bfloat16, head_dim 64 or a multiple of 16 up to 256 beyond it, pages of 16, 32 or 64 keys; everything else goes to
+// Takes bfloat16, head_dim a multiple of 16 from 32 to 256, pages of 16, 32 or 64 keys; everything else goes to
 // the mma.sync kernel (attention_prefill.cu), which is also this kernel's twin in the tests.  (The reference's kernel:
 // src/hip_ops.hip:473-551.)
 #include "tcgen05.cuh"
@@ -51,9 +51,11 @@ struct PtArgs {
   const int* entry_pos0;    // [S]
   bf16* out;
   int* err;
-  float scale_log2;         // scale * log2(e)
-  float softcap, cap_in;    // softcap > 0: a score s becomes softcap * tanh(s * cap_in), cap_in = scale / softcap
-                            // (scale_log2 is then log2(e) alone)
+  float scale_log2;         // scale * log2(e); 1 where the scores are mapped first
+  int mapped;               // scores pass a cap or a bias by distance before mask and softmax, and are then in base-2 units
+  ScoreMap map;
+  ScoreBias bias;
+  int chunk;                // > 0: a row sees its own chunk of so many positions (and there is no window)
   int has_sink;             // the softmax's denominator also holds exp(sink): a key with that score and no value
   float sink_log2;          // the sink's score times log2(e)
   HeadGate gate;            // multiplies a head's output as it is written
@@ -63,12 +65,7 @@ struct PtArgs {
   int first_wave;           // CTAs that start alone on a multiprocessor (their number), before the second ones join them
 };
 
-// 2^x by the special-function unit; exp2(-inf) = 0.
-__device__ __forceinline__ float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+__device__ __forceinline__ float ex2_approx(float x) { return ex2_fast(x); }      // (exp2(-inf) = 0)
 
 // Columns of tensor memory a CTA takes: two S buffers of 64 and O of D columns, rounded up to a power of two.
 template <int D>
@@ -152,7 +149,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     const int row0 = tile_info[1], nrows = tile_info[2];
     const int pos0 = a.entry_pos0[e] + (row0 - a.cu_rows[e]);      // position of the tile's first row
     const int hi = pos0 + nrows;                                   // keys [.., hi) exist for this tile
-    const int lo = a.window > 0 ? max(0, pos0 + 1 - a.window) : 0; // first key any row of the tile sees
+    const int lo = first_visible(pos0, a.window, a.chunk);          // first key any row of the tile sees
     const int kv0 = lo / TKB * TKB;
     const int n_blocks = (hi - kv0 + TKB - 1) / TKB;
     const uint32_t tmem_s = tmem_base, tmem_o = tmem_base + 2 * TKB;     // S(even), S(odd), O
@@ -250,7 +247,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       const int r = q * 32 + lane;
       const int p_row = pos0 + r;
       const bool live = r < nrows;
-      const int w_lo = a.window > 0 ? p_row + 1 - a.window : 0;
+      const int w_lo = first_visible(p_row, a.window, a.chunk);
+      const float slope = a.bias.slope ? a.bias.slope[h] * 1.4426950408889634f : 0.f;
+      const float* tab = a.bias.table ? a.bias.table + (size_t)h * (a.bias.last + 1) : nullptr;
       const uint32_t lane_off = (uint32_t)(q * 32) << 16;
       float m = -INFINITY, l = 0.f;
       for (int i = 0; i < n_blocks; ++i) {
@@ -262,9 +261,31 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         tmem_ld32_nowait(tmem_s + (i & 1) * TKB + lane_off + 32, s + 32);
         tmem_ld_wait();
         tmem_ld_fence<64>(s);
-        if (a.softcap > 0.f) {
+        if (a.mapped) {
+          const float d0 = (float)(p_row - j0);          // the distance to the block's first key (masked where negative)
+          if (a.map.cap1 > 0.f) {
 #pragma unroll
-          for (int c = 0; c < TKB; ++c) s[c] = a.softcap * tanhf(s[c] * a.cap_in);
+            for (int c = 0; c < TKB; ++c) s[c] = capped_log2(a.map, s[c]);
+          } else {
+#pragma unroll
+            for (int c = 0; c < TKB; ++c) s[c] *= a.map.in;
+          }
+          if (slope != 0.f) {
+            const float b0 = -slope * d0;
+#pragma unroll
+            for (int c = 0; c < TKB; ++c) s[c] += fmaf(slope, (float)c, b0);
+          }
+          if (tab) {
+            if (p_row - j0 - (TKB - 1) >= a.bias.last) {   // every key of the block is as far as the table goes, or farther
+              const float b = __ldg(tab + a.bias.last) * 1.4426950408889634f;
+#pragma unroll
+              for (int c = 0; c < TKB; ++c) s[c] += b;
+            } else {
+#pragma unroll
+              for (int c = 0; c < TKB; ++c)
+                s[c] = fmaf(__ldg(tab + min(max(p_row - j0 - c, 0), a.bias.last)), 1.4426950408889634f, s[c]);
+            }
+          }
         }
         if (!live || j0 + TKB - 1 > p_row || j0 < w_lo) {
 #pragma unroll
@@ -404,7 +425,7 @@ int launch_prefill_tc(const PtArgs& a, const void* qkv, int q_stride, int T, con
 }  // namespace
 
 NV_API int nv_attention_prefill_tc_usable(int D, int page) {
-  return D >= 64 && D <= 256 && D % 16 == 0 && (page == 16 || page == 32 || page == 64);
+  return D >= 32 && D <= 256 && D % 16 == 0 && (page == 16 || page == 32 || page == 64);
 }
 
 // Same contract as nv_attention_prefill (max_tiles counts tiles of nv_attention_prefill_tile_rows() = 64 rows, an
@@ -415,19 +436,25 @@ NV_API int nv_attention_prefill_tc(const void* qkv, int q_stride, int T, const v
                                    const int* block_table, int max_blocks, const int* cu_rows, const int* entry_pos0,
                                    int S, int max_tiles, float scale, int window, void* out, int Hq, int Hkv, int D,
                                    int page, int min_rows, int weight_terms, int* err, int has_sink, float sink_score,
-                                   float softcap, const float* gate, long long gate_ld, cudaStream_t stream) {
+                                   float softcap, const float* gate, long long gate_ld, int chunk, const float* slopes,
+                                   const float* bias_table, int bias_len, cudaStream_t stream) {
   // has_sink: a further key with the score sink_score and no value in every softmax.  softcap > 0: a scaled score s
   // becomes softcap * tanh(s / softcap) before mask and softmax.  gate: head h's output of row t is multiplied by
-  // sigmoid(gate[t * gate_ld + h]).
+  // sigmoid(gate[t * gate_ld + h]).  chunk > 0: a row at position p sees the positions from p / chunk * chunk on (and there is
+  // no window).  slopes [Hq], bias_table [Hq, bias_len]: head h's score with a key at distance n loses slopes[h] * n and
+  // gains bias_table[h][min(n, bias_len - 1)], after the cap.
+  if (chunk < 0 || (chunk > 0 && window > 0) || (bias_table && bias_len < 1)) return NV_ERR_BAD_SIZE;
   if (!nv_attention_prefill_tc_usable(D, page) || Hkv <= 0 || Hq % Hkv) return NV_ERR_UNSUPPORTED;
   if (weight_terms != 1 && weight_terms != 3) return NV_ERR_UNSUPPORTED;
   if (q_stride % 8 || ((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15)) return NV_ERR_UNSUPPORTED;
   if (S == 0 || max_tiles == 0 || T == 0) return NV_OK;
   PtArgs a;
   a.block_table = block_table; a.cu_rows = cu_rows; a.entry_pos0 = entry_pos0; a.out = (bf16*)out; a.err = err;
-  a.scale_log2 = (softcap > 0.f ? 1.f : scale) * 1.4426950408889634f;
-  a.softcap = softcap > 0.f ? softcap : 0.f;
-  a.cap_in = softcap > 0.f ? scale / softcap : 0.f;
+  a.mapped = (softcap > 0.f || slopes || bias_table) ? 1 : 0;
+  a.scale_log2 = a.mapped ? 1.f : scale * 1.4426950408889634f;
+  a.map = score_map(scale, softcap);
+  a.bias = ScoreBias{slopes, bias_table, bias_len - 1};
+  a.chunk = chunk;
   a.gate = HeadGate{gate, gate_ld};
   a.has_sink = has_sink ? 1 : 0;
   a.sink_log2 = sink_score * 1.4426950408889634f;
@@ -444,11 +471,11 @@ NV_API int nv_attention_prefill_tc(const void* qkv, int q_stride, int T, const v
   a.D = D;
   const int tiles = (max_tiles + S + 1) / 2;
   if (weight_terms == 3) {
-    if (D == 64) return launch_prefill_tc<64, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
+    if (D <= 64) return launch_prefill_tc<64, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
     if (D > 128) return launch_prefill_tc<256, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
     return launch_prefill_tc<128, 3>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
   }
-  if (D == 64) return launch_prefill_tc<64, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
+  if (D <= 64) return launch_prefill_tc<64, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
   if (D > 128) return launch_prefill_tc<256, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
   return launch_prefill_tc<128, 1>(a, qkv, q_stride, T, kc, vc, num_pages, tiles, stream);
 }

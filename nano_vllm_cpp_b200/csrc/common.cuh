@@ -78,7 +78,9 @@ __device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f +
 #define NV_EPI_RELU2 7
 // 8: a third pairing of gate and up rows, gelu in its tanh form on the gate: out = gelu_tanh(g) u.
 #define NV_EPI_GEGLU_TANH 8
-#define NV_EPI_LAST NV_EPI_GEGLU_TANH
+// 9: silu on the first p0 outputs of a row only; the others pass (a stacked projection of which some columns are activated).
+#define NV_EPI_SILU_FIRST 9
+#define NV_EPI_LAST NV_EPI_SILU_FIRST
 // Which codes pair a gate row with an up row (two accumulators per output), and the pairings themselves.
 __host__ __device__ __forceinline__ int epi_pair(int code) {
   return (code == NV_EPI_SWIGLU || code == NV_EPI_GLU_CLAMPED || code == NV_EPI_GEGLU_TANH) ? code : 0;
@@ -105,6 +107,11 @@ __device__ __forceinline__ float epilogue_act(int act, float v, float p0 = 0.f, 
   return v / (1.f + expf(-v));
 }
 
+// The unary activation of output feature n, for the codes that do not treat all features alike.
+__device__ __forceinline__ int epi_at(int act, int n, float p0) {
+  return act == NV_EPI_SILU_FIRST ? (n < (int)p0 ? NV_EPI_SILU : 0) : act;
+}
+
 // What multiplies a query head's attention output before it is stored: sigmoid of `gate[t * ld + h]` (t the batch row, h
 // the query head), or one without a gate (gate == nullptr).
 struct HeadGate {
@@ -113,6 +120,53 @@ struct HeadGate {
 };
 __device__ __forceinline__ float head_gate_of(const HeadGate& g, long long t, int h) {
   return g.gate ? 1.f / (1.f + expf(-g.gate[t * g.ld + h])) : 1.f;
+}
+
+// What the distance between a row and a key gives to their score, after the cap and before the softmax: -slope[h] * n, and
+// table[h * (last + 1) + min(n, last)], for query head h and distance n (either array may be nullptr).
+struct ScoreBias {
+  const float* slope;
+  const float* table;
+  int last;
+};
+__device__ __forceinline__ float score_bias_of(const ScoreBias& b, int h, int n) {
+  float v = b.slope ? -b.slope[h] * (float)n : 0.f;
+  if (b.table) v += b.table[(size_t)h * (b.last + 1) + min(n, b.last)];
+  return v;
+}
+// The first position that a row at position p sees: a sliding window (0: none), or the start of its chunk (0: no chunks).
+__host__ __device__ __forceinline__ int first_visible(int p, int window, int chunk) {
+  if (chunk > 0) return p / chunk * chunk;
+  return window > 0 && p + 1 > window ? p + 1 - window : 0;
+}
+__device__ __forceinline__ float ex2_fast(float x) {         // 2^x by the special-function unit
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// A score on its way to base-2 units in the tensor-core kernels.  cap tanh(x / cap) = cap - 2 cap / (e^(2 x / cap) + 1), whose
+// absolute error is a few units of the cap's last place, as the difference's is whatever x is.
+struct ScoreMap {
+  float in;                 // without a cap: scale * log2(e)
+  float cap_k, cap1, cap2;  // with a cap (cap1 > 0): 2 log2(e) scale / cap, cap log2(e), 2 cap log2(e)
+};
+static inline ScoreMap score_map(float scale, float softcap) {
+  const float l2e = 1.4426950408889634f;
+  ScoreMap m = {scale * l2e, 0.f, 0.f, 0.f};
+  if (softcap > 0.f) {
+    m.cap_k = 2.f * l2e * scale / softcap;
+    m.cap1 = softcap * l2e;
+    m.cap2 = 2.f * softcap * l2e;
+  }
+  return m;
+}
+__device__ __forceinline__ float capped_log2(const ScoreMap& m, float s) {
+  return fmaf(-m.cap2, rcp_fast(ex2_fast(s * m.cap_k) + 1.f), m.cap1);
 }
 
 // Programmatic dependent launch.  A kernel launched with the programmatic-serialization attribute may start

@@ -148,11 +148,13 @@ class BlockPool {
 // ------------------------------------------------------------------------------------------ CacheManager
 // Which pages and which state slot every live request holds.  Layers with the same needs form a group
 // with pages and block tables of its own (one group for layers that read every earlier key, one per
-// window size and number of kept first positions); a group with a window gives a page back as soon as every
+// window size and number of kept first positions, one per chunk size); a group with a window gives a page back as soon as every
 // position in it lies before the window of the next row to run, except the pages that hold one of the group's kept
-// first positions, which a request holds to its end.  A request also holds one state slot from open to close.  Hashing
+// first positions, which a request holds to its end.  A group with chunks (rows see the positions of their own chunk of
+// so many, counted from the sequence's start) gives a page back once the next row to run lies in a later chunk than all
+// of the page.  A request also holds one state slot from open to close.  Hashing
 // of full pages, so that requests with a common prefix share them (src/block_manager.cpp:56-98,
-// 121-134), is offered only for a single group without a window.
+// 121-134), is offered only for a single group that reads every earlier key.
 struct RequestCache {
   int64_t rid = 0;
   int slot = 0;
@@ -168,6 +170,7 @@ class CacheManager {
  public:
   std::vector<int> windows;
   std::vector<int> keeps;                 // per group: the first so many positions stay readable behind the window
+  std::vector<int> chunks;                // per group: rows read the positions of their own chunk of so many (0: no chunks)
   int page_size, max_requests;
   std::vector<BlockPool> pools;
   std::vector<int> free_slots;            // a stack: slot 0 is handed out first
@@ -179,12 +182,13 @@ class CacheManager {
   // prefix sharing is refused then, as it is for more than one group or a window.  `groups` may be 0 (a model
   // without paged layers): requests then hold a state slot and nothing else.
   CacheManager(const int* w, const int* n_pages, int groups, int ps, int max_req, bool prefix, bool has_state,
-               const int* keep = nullptr)
-      : windows(w, w + groups), keeps(groups, 0), page_size(ps), max_requests(max_req) {
+               const int* keep = nullptr, const int* chunk = nullptr)
+      : windows(w, w + groups), keeps(groups, 0), chunks(groups, 0), page_size(ps), max_requests(max_req) {
     if (keep) keeps.assign(keep, keep + groups);
+    if (chunk) chunks.assign(chunk, chunk + groups);
     for (int g = 0; g < groups; ++g) pools.emplace_back(n_pages[g], ps);
     for (int s = max_req - 1; s >= 0; --s) free_slots.push_back(s);
-    prefix_caching = prefix && !has_state && groups == 1 && windows[0] == 0;
+    prefix_caching = prefix && !has_state && groups == 1 && windows[0] == 0 && chunks[0] == 0;
   }
   RequestCache* find(int64_t rid) {
     auto it = requests.find(rid);
@@ -218,8 +222,9 @@ class CacheManager {
     requests.erase(it);
     return OK;
   }
-  int first_needed_page(int g, int start) const {    // lowest page of the window that rows from position `start` on read
+  int first_needed_page(int g, int start) const {    // lowest page of the window or chunk that rows from position `start` on read
     const int w = windows[g];
+    if (chunks[g] > 0) return start / chunks[g] * chunks[g] / page_size;
     if (w <= 0) return 0;
     return std::max(0, start + 1 - w) / page_size;
   }
@@ -580,9 +585,9 @@ NVH_API int nvh_pool_check(void* p, const int* held) {
 
 // ---- the cache manager
 NVH_API void* nvh_manager_create(const int* windows, const int* num_pages, int groups, int page_size, int max_requests,
-                                 int prefix_caching, int has_state, const int* keep_first) {
+                                 int prefix_caching, int has_state, const int* keep_first, const int* chunks) {
   return new CacheManager(windows, num_pages, groups, page_size, max_requests, prefix_caching != 0, has_state != 0,
-                          keep_first);
+                          keep_first, chunks);
 }
 NVH_API void nvh_manager_destroy(void* m) { delete (CacheManager*)m; }
 NVH_API void* nvh_manager_pool(void* m, int g) { return &((CacheManager*)m)->pools[g]; }

@@ -8,15 +8,24 @@
 // How a row's router logits become choices and weights.  mode 0: p = softmax(logits + bias) (bias may be nullptr), the
 // K largest p are chosen and weigh p (or p / their sum, which is the softmax over the chosen logits).  mode 1: s = sigmoid(logit) in float32; the K largest s + bias[e] are chosen
 // (bias may be nullptr) and weigh s, without the bias.  Either way the weights are multiplied by `scale`.
+// groups > 0: the experts form that many equal groups of neighbours; a group counts as its largest choice score, and only
+// the experts of the `keep` best groups (the lower index on a tie) can be chosen.
 struct RouteRule {
   int mode;
   const float* bias;
   float scale;
+  int groups, keep;
 };
+
+// Whether E experts can be grouped so (groups 0: they are not) and K of them be chosen from the groups that are kept.
+static inline bool route_groups_ok(int E, int K, int groups, int keep) {
+  if (groups == 0) return true;
+  return groups > 0 && E % groups == 0 && keep >= 1 && keep <= groups && K <= keep * (E / groups);
+}
 
 // One warp routes one row: p = softmax(logits) over all E in double, then K rounds of "largest
 // remaining, lowest index on a tie", optional renormalisation of the K weights in double
-// (src/hip_ops.hip:813-841); or the sigmoid rule of RouteRule.  `pr` is E doubles of scratch for this warp.
+// (src/hip_ops.hip:813-841); or the sigmoid rule of RouteRule.  `pr` is E + rule.groups doubles of scratch for this warp.
 // With C > 0 the row also gets C "always on" experts E .. E+C-1 with weight sigmoid(gate_logit), or 1 without a
 // gate: the chunks of a shared expert that is computed as C more experts (src/model.cpp:803-811 computes it
 // separately).  idx and score rows are K + C wide.
@@ -45,6 +54,24 @@ __device__ __forceinline__ void route_row(const float* __restrict__ r, int E, in
     for (int e = lane; e < E; e += 32) pr[e] /= s;
   }
   __syncwarp();
+  if (rule.groups > 0 && rule.keep < rule.groups) {
+    const int n = E / rule.groups;
+    double* best_of = pr + E;
+    for (int g = lane; g < rule.groups; g += 32) {
+      double m = -INFINITY;
+      for (int e = g * n; e < (g + 1) * n; ++e) m = fmax(m, pr[e]);
+      best_of[g] = m;
+    }
+    __syncwarp();
+    for (int g = lane; g < rule.groups; g += 32) {
+      const double m = best_of[g];
+      int better = 0;                       // groups that go before this one
+      for (int o = 0; o < rule.groups; ++o) better += best_of[o] > m || (best_of[o] == m && o < g);
+      if (better >= rule.keep)
+        for (int e = g * n; e < (g + 1) * n; ++e) pr[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
   double wsum = 0.0;
   double mine = 0.0;  // lane k keeps the k-th weight (K <= 32)
   for (int k = 0; k < K; ++k) {
@@ -60,6 +87,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ r, int E, in
       int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
     }
+    if (bi >= E) { bi = 0; best = 0.0; }    // (no number among the scores: keep every index inside the arrays)
     if (rule.mode == 1) best = (double)(1.f / (1.f + expf(-r[bi])));     // the weight is the score without the bias
     if (lane == k) { mine = best; idx_row[k] = bi; }
     wsum += best;

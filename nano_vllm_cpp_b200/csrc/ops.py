@@ -265,8 +265,8 @@ def embedding(ids, table, out, err: ErrorFlag, feed=None, copies: int = 1, scale
 
 
 def add_rmsnorm(x, branch, w, eps: float, out, out32=None, *, mix=None, branch2=None, branch_weight=None,
-                branch_eps: float = 0.0) -> None:
-    """x (+= branch (+ branch2)); out = rmsnorm(x) * w; optional float32 copy of out.
+                branch_eps: float = 0.0, branch_scale: float = 1.0, branch2_scale: float = 1.0) -> None:
+    """x (+= branch_scale * branch (+ branch2_scale * branch2)); out = rmsnorm(x) * w; optional float32 copy of out.
 
     ``mix`` = (rows, index, weight, dense, gate_logit) gives the branch as a sum that has not been taken yet:
     ``sigmoid(gate_logit[t]) * dense[t] + sum_r weight[t, r] * rows[index[t, r]]`` (dense and gate_logit may be
@@ -282,6 +282,7 @@ def add_rmsnorm(x, branch, w, eps: float, out, out32=None, *, mix=None, branch2=
     _need(x.dtype == torch.float32, "add_rmsnorm: the residual stream is float32")
     _need(branch2 is None or (branch is not None and branch2.dtype == torch.float32 and branch2.shape == x.shape),
           "add_rmsnorm: a second branch comes with a first and is float32 and shaped like x")
+    _need((branch_scale == 1.0 and branch2_scale == 1.0) or branch2 is not None, "add_rmsnorm: scales come with two branches")
     _need(branch is None or (branch.dtype == torch.float32 and branch.shape == x.shape),
           "add_rmsnorm: branch must be float32 and shaped like x")
     _need(w.numel() == H and out.shape == x.shape, "add_rmsnorm: shape mismatch")
@@ -306,7 +307,8 @@ def add_rmsnorm(x, branch, w, eps: float, out, out32=None, *, mix=None, branch2=
             _need(t_ is None or t_.data_ptr() % 16 == 0, "add_rmsnorm: rows must start on 16-byte boundaries")
     _check(lib().nv_add_rmsnorm(_p(x), _p(branch), _p(branch2), _p(w), dt(w), eps, _p(out), dt(out),
                                 _p(out32), T, H, _p(rows), _p(index), _p(weight), R, _p(dense),
-                                _p(gate), gate_ld, _p(branch_weight), float(branch_eps), _stream()), "add_rmsnorm")
+                                _p(gate), gate_ld, _p(branch_weight), float(branch_eps), float(branch_scale),
+                                float(branch2_scale), _stream()), "add_rmsnorm")
 
 
 ADD_RMSNORM_MAX_MIX = 64
@@ -317,6 +319,7 @@ EPILOGUE_ACTS = {"gelu_erf": 2, "gelu_tanh": 3, "silu": 4, "relu2": 7}
 EPILOGUE_XIELU = 5          # given as the tuple ("xielu", p0, p1) with its two positive numbers
 EPILOGUE_GLU_CLAMPED = 6    # with ``swiglu``: the tuple ("glu_clamped", limit, slope) makes the pairing of gate and up rows
                             # g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(slope g) (u + 1)
+EPILOGUE_SILU_FIRST = 9     # the tuple ("silu_first", n): silu on the first n outputs of a row, the others pass
 
 
 def _epilogue(swiglu: bool, act) -> int:
@@ -324,6 +327,9 @@ def _epilogue(swiglu: bool, act) -> int:
     of a unary activation that every output value passes after the bias."""
     if act is None:
         return 1 if swiglu else 0
+    if isinstance(act, tuple) and act[0] == "silu_first":
+        _need(not swiglu and len(act) == 2 and act[1] >= 0, "silu on the first outputs is ('silu_first', how many)")
+        return EPILOGUE_SILU_FIRST
     if isinstance(act, tuple):
         if swiglu:
             _need(len(act) == 3 and act[0] == "glu_clamped" and act[1] > 0, "a pairing with numbers is ('glu_clamped', limit, slope)")
@@ -338,7 +344,7 @@ def _epilogue(swiglu: bool, act) -> int:
 
 def _act_numbers(act):
     """The two numbers that a product's launcher takes beside the activation's code (0, 0 where it has none)."""
-    return (float(act[1]), float(act[2])) if isinstance(act, tuple) else (0.0, 0.0)
+    return (float(act[1]), float(act[2]) if len(act) > 2 else 0.0) if isinstance(act, tuple) else (0.0, 0.0)
 
 
 def gemm_plain(a, w, out, *, bias=None, a_rows=None, swiglu=False, M=None, tiles=None, act=None) -> None:
@@ -402,19 +408,22 @@ def attention_decode_usable(k_cache, D: int) -> bool:
 
 def attention_decode(qkv, k_cache, v_cache, block_table, row_entry, positions, scale: float, window: int, out,
                      Hq: int, Hkv: int, D: int, max_context: int, rows=None, err=None, sink_score=None,
-                     float_weights: bool = False, softcap: float = 0.0, gate=None) -> None:
+                     float_weights: bool = False, softcap: float = 0.0, gate=None, chunk: int = 0, slopes=None,
+                     bias_table=None) -> None:
     """One query row per request (``rows``: which batch rows; None = all) against its paged keys.  ``qkv``: rows
     whose first Hq * D elements are the query heads.  ``sink_score``: a further key with that score and no value
     in every softmax.  ``float_weights``: the weights keep all their bits in the product with the values (the
     tensor-core form takes them as three bfloat16 terms instead of one rounded one; the kernel that gives a lane a
     chunk of a key, which other head sizes and a sink go to, multiplies in float32).  ``softcap`` > 0: a scaled score s
-    becomes ``softcap * tanh(s / softcap)`` (the lane-per-chunk kernel).  ``gate``: see ``_head_gates``."""
+    becomes ``softcap * tanh(s / softcap)``.  ``gate``: see ``_head_gates``.  ``chunk``, ``slopes``, ``bias_table``: see
+    ``_score_bias``."""
     _cuda_contig(qkv, k_cache, v_cache, block_table, row_entry, positions, out, rows)
     _i32(block_table, row_entry, positions, rows)
     R = qkv.shape[0] if rows is None else rows.numel()
     page = k_cache.shape[2]
     L = lib()
-    splits = L.nv_attention_decode_splits(R, Hq, Hkv, max_context, num_sms())
+    seen = min([max_context] + [n for n in (window, chunk) if n > 0])        # the most keys a row reads
+    splits = L.nv_attention_decode_splits(R, Hq, Hkv, seen, num_sms())
     scratch = counts = None
     if splits > 1:
         scratch = torch.empty(R * Hq * splits * (D + 2), dtype=torch.float32, device=qkv.device)
@@ -427,7 +436,18 @@ def attention_decode(qkv, k_cache, v_cache, block_table, row_entry, positions, s
                                  _p(counts), (counts.numel() if counts is not None else 0),
                                  (0 if sink_score is None else 1), float(sink_score or 0.0),
                                  (1 if float_weights else 0), float(softcap), *_head_gates(gate, qkv.shape[0], Hq),
-                                 _stream()), "attention_decode")
+                                 *_score_bias(chunk, slopes, bias_table, Hq), _stream()), "attention_decode")
+
+
+def _score_bias(chunk: int, slopes, table, Hq: int):
+    """``chunk`` > 0: a row at position p sees the positions from ``p // chunk * chunk`` on (and there is no window).
+    ``slopes`` (float32 [Hq]) and ``table`` (float32 [Hq, n]): the score of query head h with a key at distance d loses
+    ``slopes[h] * d`` and gains ``table[h, min(d, n - 1)]``, behind the cap.  What the attention launchers take for them."""
+    _cuda_contig(slopes, table)
+    _f32(slopes, table)
+    _need(slopes is None or slopes.numel() == Hq, "attention: one slope per query head")
+    _need(table is None or (table.dim() == 2 and table.shape[0] == Hq and table.shape[1] >= 1), "attention: a row of biases per query head")
+    return chunk, _p(slopes), _p(table), (table.shape[1] if table is not None else 0)
 
 
 def _head_gates(gate, T: int, Hq: int):
@@ -459,19 +479,19 @@ def attention_prefill_tile_rows() -> int:
 def attention_prefill(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, max_tiles: int, scale: float,
                       window: int, out, Hq: int, Hkv: int, D: int, err=None, min_rows: int = 1,
                       kernel: str = "auto", sink_score=None, weight_terms: int = 1, softcap: float = 0.0,
-                      gate=None) -> None:
+                      gate=None, chunk: int = 0, slopes=None, bias_table=None) -> None:
     """bfloat16 rows of any mix of portions against their paged keys: the tcgen05 kernel for head sizes from
-    64 to 256 (multiples of 16) and pages of 16, 32 or 64 keys, else the mma.sync kernel (``kernel="mma"`` asks for that one).  Entries
+    32 to 256 (multiples of 16) and pages of 16, 32 or 64 keys, else the mma.sync kernel (``kernel="mma"`` asks for that one).  Entries
     with fewer than ``min_rows`` rows are skipped and their rows of ``out`` left as they are.
     ``weight_terms`` = 3: the float32 weights enter the product with the values as three bfloat16 terms, all their
     bits (either kernel).  ``sink_score``: a further key with that score and no value in every softmax; ``softcap``
     > 0: a scaled score s becomes ``softcap * tanh(s / softcap)`` before mask and softmax (either kernel).  ``gate``: see
-    ``_head_gates``."""
+    ``_head_gates``; ``chunk``, ``slopes``, ``bias_table``: see ``_score_bias`` (either kernel)."""
     _cuda_contig(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, out)
     _i32(block_table, cu_rows, entry_pos0)
     _need(qkv.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16,
           "attention_prefill: bfloat16 only")
-    _need(out.shape == (qkv.shape[0], Hq * D), "attention_prefill: out shape")
+    _need(out.shape == (qkv.shape[0], Hq * D) and qkv.shape[1] >= Hq * D, "attention_prefill: shapes")
     S = entry_pos0.numel()
     L = lib()
     page = k_cache.shape[2]
@@ -484,14 +504,16 @@ def attention_prefill(qkv, k_cache, v_cache, block_table, cu_rows, entry_pos0, m
                                          window, _p(out), Hq, Hkv, D, page,
                                          min_rows, weight_terms, _p(err.t if err is not None else _global_err().t),
                                          (0 if sink_score is None else 1), float(sink_score or 0.0), float(softcap),
-                                         *_head_gates(gate, qkv.shape[0], Hq), _stream()),
+                                         *_head_gates(gate, qkv.shape[0], Hq),
+                                         *_score_bias(chunk, slopes, bias_table, Hq), _stream()),
                "attention_prefill_tc")
         return
     _check(L.nv_attention_prefill(_p(qkv), qkv.shape[1], _p(k_cache), _p(v_cache), _p(block_table),
                                   block_table.shape[1], _p(cu_rows), _p(entry_pos0), S,
                                   max_tiles, scale, window, _p(out), Hq, Hkv,
                                   D, page, min_rows, (0 if sink_score is None else 1), float(sink_score or 0.0),
-                                  weight_terms, float(softcap), *_head_gates(gate, qkv.shape[0], Hq), _stream()),
+                                  weight_terms, float(softcap), *_head_gates(gate, qkv.shape[0], Hq),
+                                  *_score_bias(chunk, slopes, bias_table, Hq), _stream()),
            "attention_prefill")
 
 
@@ -615,16 +637,18 @@ ROUTE_SCORES = {"softmax": 0, "sigmoid": 1}
 
 
 def _route_rule(rule, E: int):
-    """``rule`` = None (softmax, no bias, weights as they are) or (score kind, bias [E] float32 or None, weight scale):
-    what the routing kernels take as their last three arguments.  With sigmoid scores the bias steers the choice only;
-    with softmax scores it is added to the logits."""
+    """``rule`` = None (softmax, no bias, weights as they are) or (score kind, bias [E] float32 or None, weight scale) or
+    the same with (groups, kept groups) behind it: what the routing kernels take as their last five arguments.  With
+    sigmoid scores the bias steers the choice only; with softmax scores it is added to the logits.  With groups (equal
+    runs of neighbouring experts) only the experts of the kept groups, those with the largest members, can be chosen."""
     if rule is None:
-        return 0, None, 1.0
-    kind, bias, scale = rule
+        return 0, None, 1.0, 0, 0
+    kind, bias, scale = rule[:3]
+    groups, keep = rule[3] if len(rule) > 3 and rule[3] is not None else (0, 0)
     _need(kind in ROUTE_SCORES, f"router: the score is one of {sorted(ROUTE_SCORES)}")
     _need(bias is None or (bias.is_cuda and bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == E),
           "router: the bias is float32 [E]")
-    return ROUTE_SCORES[kind], bias, float(scale)
+    return ROUTE_SCORES[kind], bias, float(scale), int(groups), int(keep)
 
 
 def router_topk(logits, K: int, renorm: bool, idx, score, C: int = 0, gate_logit=None, rule=None) -> None:
@@ -638,11 +662,11 @@ def router_topk(logits, K: int, renorm: bool, idx, score, C: int = 0, gate_logit
     _i32(idx)
     _need(idx.shape == (T, K + C) and score.shape == (T, K + C), "router: output shapes")
     _need(gate_logit is None or gate_logit.dtype == torch.float32, "router: gate logits")
-    mode, bias, wscale = _route_rule(rule, E)
+    mode, bias, wscale, groups, keep = _route_rule(rule, E)
     _check(lib().nv_router_topk(_p(logits), logits.stride(0), T, E, K,
                                 (1 if renorm else 0), _p(idx), _p(score), C, _p(gate_logit),
                                 (gate_logit.stride(0) if gate_logit is not None else 0), mode, _p(bias), wscale,
-                                _stream()),
+                                groups, keep, _stream()),
            "router_topk")
 
 
@@ -716,8 +740,8 @@ def moe_align(idx, K: int, al: MoeAlignment, err: ErrorFlag, spread_last: int = 
            "moe_align")
 
 
-def moe_route_small_usable(T: int, E: int, K: int, C: int, H: int) -> bool:
-    return bool(lib().nv_moe_route_small_usable(T, E, K, C, H))
+def moe_route_small_usable(T: int, E: int, K: int, C: int, H: int, groups: int = 0) -> bool:
+    return bool(lib().nv_moe_route_small_usable(T, E, K, C, H, groups))
 
 
 def moe_route_small(logits, K: int, renorm: bool, C: int, gate_logit, idx, score, al: "MoeAlignment", err, x=None,
@@ -736,7 +760,7 @@ def moe_route_small(logits, K: int, renorm: bool, C: int, gate_logit, idx, score
         _need(x.dtype == torch.bfloat16 and x.is_contiguous(), "route: bfloat16 rows")
         H = x.shape[1]
         xs = torch.empty((T * KT, H), dtype=x.dtype, device=x.device)
-    mode, bias, wscale = _route_rule(rule, E)
+    mode, bias, wscale, groups, keep = _route_rule(rule, E)
     _check(lib().nv_moe_route_small(_p(logits), logits.stride(0), T, E, K,
                                     (1 if renorm else 0), C, _p(gate_logit),
                                     (gate_logit.stride(0) if gate_logit is not None else 0), _p(idx),
@@ -744,7 +768,7 @@ def moe_route_small(logits, K: int, renorm: bool, C: int, gate_logit, idx, score
                                     _p(al.pair_pos), _p(al.tile_expert), _p(al.tile_row0), _p(al.tile_rows),
                                     _p(al.num_tiles), _p(err.t), _p(x), _p(xs), H, (C if static else 0),
                                     _p(zero), (zero.numel() if zero is not None else 0), mode, _p(bias), wscale,
-                                    _stream()), "moe_route_small")
+                                    groups, keep, _stream()), "moe_route_small")
     return xs
 
 
@@ -1107,14 +1131,15 @@ def qk_prepare_store(src, q0: int, k0: int, v0: int, positions, row_entry, block
 def paged_attention_general(q, k_cache, v_cache, block_table, row_entry, positions, scale: float, window: int, out,
                             Hq: int, Hkv: int, D: int, Dv: int, sink_score=None, *, sinks=None, keep_first: int = 0,
                             key_span: int = 1, value_heads: int | None = None, softcap: float = 0.0,
-                            gate=None) -> None:
+                            gate=None, chunk: int = 0, slopes=None, bias_table=None) -> None:
     """Causal softmax attention of every row over its request's paged keys; values may be wider or narrower than
     keys; ``sink_score``: a further key with that score and no value in every softmax (None: none), ``sinks``
     (float32 [Hq]): one such score per head; ``keep_first``: with a window, the sequence's first so many positions
     stay visible; ``key_span`` = Hkv: a query row holds Hkv * D elements per head and a score is the sum of its
     parts' products with all kv heads' keys (see ``mix_query_heads``); ``v_cache`` None: the values are read where
     the keys are; ``value_heads``: kv heads of the values where that is not ``Hkv``; ``softcap`` > 0: a scaled score
-    s becomes ``softcap * tanh(s / softcap)`` before mask and softmax; ``gate``: see ``_head_gates``."""
+    s becomes ``softcap * tanh(s / softcap)`` before mask and softmax; ``gate``: see ``_head_gates``; ``chunk``,
+    ``slopes``, ``bias_table``: see ``_score_bias``."""
     if v_cache is None:
         v_cache = k_cache
     Hv = Hkv if value_heads is None else value_heads
@@ -1130,7 +1155,8 @@ def paged_attention_general(q, k_cache, v_cache, block_table, row_entry, positio
                                             block_table.shape[1], _p(row_entry), _p(positions), scale, window,
                                             keep_first, (0 if sink_score is None else 1), float(sink_score or 0.0),
                                             _p(sinks), _p(out), dt(out), T, Hq, Hkv, Hv, D, Dv, key_span,
-                                            k_cache.shape[2], float(softcap), *_head_gates(gate, T, Hq), _stream()),
+                                            k_cache.shape[2], float(softcap), *_head_gates(gate, T, Hq),
+                                            *_score_bias(chunk, slopes, bias_table, Hq), _stream()),
            "paged_attention_general")
 
 
@@ -1169,12 +1195,31 @@ def causal_conv_add(h, w, batch, state, out) -> None:
     _need(w.shape == (taps, H) and out.shape == (T, H) and out.data_ptr() != h.data_ptr(), "causal_conv_add: shapes")
     _need(taps == 1 or (state is not None and state.shape[1:] == (taps - 1, H)), "causal_conv_add: state")
     single = taps > 1 and batch.decode_only
-    _check(lib().nv_causal_conv_add(_p(h), _p(w), taps, _p(batch.row_entry), _p(batch.cu_rows), _p(batch.entry_slot),
-                                    _p(state) if taps > 1 else None, _slot_stride(state) if taps > 1 else 0, _p(out), dt(out),
-                                    T, H, 1 if single else 0, _stream()), "causal_conv_add",
+    _check(lib().nv_causal_conv(_p(h), H, _p(w), None, 0, taps, _p(batch.row_entry), _p(batch.cu_rows), _p(batch.entry_slot),
+                                _p(state) if taps > 1 else None, _slot_stride(state) if taps > 1 else 0, _p(out), dt(out),
+                                T, H, 1 if single else 0, _stream()), "causal_conv_add",
            nbytes=float(T) * H * (4 + out.element_size()))
     if taps > 1 and not single:
         conv_state_update(h, 0, H, taps, batch, state)
+
+
+def causal_conv_silu(src, col0: int, w, bias, batch, state, out) -> None:
+    """``out[t, c] = silu(bias[c] + sum_j w[j, c] * src[t - (taps - 1) + j, col0 + c])``: a causal convolution over time on the
+    channels ``col0 .. col0 + C`` of float32 rows.  ``w`` float32 [taps, C] (the last row the current token's), ``bias`` [C] or
+    None, ``state`` [slots, taps - 1, C] as in ``causal_conv_add``."""
+    _cuda_contig(w, bias, out)
+    _f32(src, w, bias)
+    (taps, C), T = w.shape, src.shape[0]
+    _need(src.is_cuda and src.stride(1) == 1 and src.shape[1] >= col0 + C and out.shape == (T, C)
+          and (bias is None or bias.numel() == C), "causal_conv_silu: shapes")
+    _need(taps == 1 or (state is not None and state.shape[1:] == (taps - 1, C)), "causal_conv_silu: state")
+    single = taps > 1 and batch.decode_only
+    _check(lib().nv_causal_conv(src.data_ptr() + 4 * col0, src.stride(0), _p(w), _p(bias), 1, taps, _p(batch.row_entry),
+                                _p(batch.cu_rows), _p(batch.entry_slot), _p(state) if taps > 1 else None,
+                                _slot_stride(state) if taps > 1 else 0, _p(out), dt(out), T, C, 1 if single else 0, _stream()),
+           "causal_conv_silu", nbytes=float(T) * C * (4 + out.element_size()))
+    if taps > 1 and not single:
+        conv_state_update(src, col0, C, taps, batch, state)
 
 
 def retention_usable(form: str, dk: int, dv: int) -> bool:
@@ -1193,25 +1238,56 @@ def retention(proj, cols: dict, batch, S, powers, inv_freq, rot_dim: int, H: int
     ``dk^-1/2``; ``out = o / sqrt(mean(o^2) + eps) * silu(gate)``.  ``proj`` float32 [T, P] holds q, k, v and the gate at
     ``cols``; ``powers`` float32 [H, 65]: the decays to the power 0 .. 64.  ``fast``: entries of one row in one launch,
     the others in chunks on the tensor cores; else (or where those do not take the sizes) the scan."""
-    _cuda_contig(proj, powers, inv_freq, out)
-    _f32(proj, powers, inv_freq)
+    _need(out.shape == (proj.shape[0], H * dv), "retention: shapes")
+    _decayed_memory("retention", proj, cols, batch, S, H, H, dk, dv, powers=powers, k_scale=float(dk) ** -0.5,
+                    inv_freq=inv_freq, rot_dim=rot_dim, eps=eps, out=out, fast=fast)
+
+
+def decayed_memory(src, cols: dict, batch, S, H: int, dk: int, dv: int, raw, *, q_heads: int | None = None, powers=None,
+                   steps=None, fast: bool = True) -> None:
+    """The same recurrence without rotation, scaling, head norm and gate: ``raw`` [T, H, dv] float32 receives every head's
+    ``o``.  ``src`` float32 [T, P] holds q, k and v at ``cols``; ``q_heads``: q and k have so many heads, and head h reads
+    number ``h // (H / q_heads)``.  Decays: ``powers`` as in ``retention``, or ``steps`` = (z [T, >= col + H] float32, col,
+    A_log [H], bias [H]): a step size per row and head, ``dt = softplus(z + bias)``, by which k is multiplied, and the decay
+    ``exp(-exp(A_log) dt)``."""
+    _need(raw.shape == (src.shape[0], H, dv) and (powers is None) != (steps is None), "decayed_memory: shapes")
+    _decayed_memory("decayed_memory", src, cols, batch, S, H, H if q_heads is None else q_heads, dk, dv, powers=powers,
+                    k_scale=1.0, raw=raw, steps=steps, fast=fast)
+
+
+def _decayed_memory(name, proj, cols, batch, S, H, G, dk, dv, *, powers=None, k_scale=1.0, inv_freq=None, rot_dim=0,
+                    eps=0.0, out=None, raw=None, steps=None, fast=True):
+    _cuda_contig(powers, inv_freq, out, raw)
+    _f32(proj, powers, inv_freq, raw)
+    _need(proj.is_cuda and proj.stride(1) == 1, f"{name}: float32 rows")
     T = proj.shape[0]
     rc = retention_chunk_rows()
-    _need(powers.shape == (H, rc + 1) and out.shape == (T, H * dv) and S.shape[1:] == (H, dk, dv), "retention: shapes")
-    _need(rot_dim % 2 == 0 and 0 <= rot_dim <= dk and inv_freq.numel() >= rot_dim // 2, "retention: rotation")
+    _need((powers is None or powers.shape == (H, rc + 1)) and S.shape[1:] == (H, dk, dv) and H % G == 0, f"{name}: shapes")
+    _need(rot_dim % 2 == 0 and 0 <= rot_dim <= dk and (rot_dim == 0 or inv_freq.numel() >= rot_dim // 2), f"{name}: rotation")
     half = rot_dim // 2
     dev = proj.device
+    dsrc, d_ld, d0, A_log, dt_bias = None, 0, 0, None, None
+    if steps is not None:
+        dsrc, d0, A_log, dt_bias = steps
+        _f32(dsrc, A_log, dt_bias)
+        _need(dsrc.stride(1) == 1 and dsrc.shape[0] == T and dsrc.shape[1] >= d0 + H and A_log.numel() == H
+              and dt_bias.numel() == H, f"{name}: step sizes")
+        d_ld = dsrc.stride(0)
+    to_raw = raw is not None
 
-    def launch(what, name, *, table=None, rows=None, R=0, raw=None, chunks=None, max_chunks=0, min_rows=1, flops=0.0):
-        _check(lib().nv_retention(what, _p(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols["g"], _p(table),
+    def launch(what, form, *, table=None, rows=None, R=0, scratch=None, chunks=None, decays=None, max_chunks=0, min_rows=1,
+               flops=0.0):
+        o = out if out is not None else raw
+        _check(lib().nv_retention(what, _p(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols.get("g", 0), _p(table),
                                   _p(batch.positions), _p(inv_freq), half, _p(batch.row_entry), _p(batch.cu_rows),
                                   _p(batch.entry_slot), batch.S, _p(rows), R, _p(S), _slot_stride(S), _p(powers),
-                                  float(dk) ** -0.5, float(eps), _p(out), dt(out), _p(raw), _p(chunks), max_chunks, T, H, dk,
-                                  dv, min_rows, _stream()), name, flops)
+                                  float(k_scale), float(eps), _p(o), dt(o), _p(raw if to_raw else scratch), _p(chunks),
+                                  max_chunks, T, H, dk, dv, min_rows, G, 1 if to_raw else 0, _p(dsrc), d_ld, d0, _p(A_log),
+                                  _p(dt_bias), _p(decays), _stream()), f"{name}_{form}", flops)
 
     single = batch.n_single if fast and retention_usable("step", dk, dv) else 0
     if single:
-        launch(0, "retention_step", rows=None if batch.decode_only else batch.single_rows, R=single)
+        launch(0, "step", rows=None if batch.decode_only else batch.single_rows, R=single)
     if single == batch.S:
         return
     table = None
@@ -1223,11 +1299,30 @@ def retention(proj, cols: dict, batch, S, powers, inv_freq, rot_dim: int, H: int
         # an upper bound of the entries' chunks that depends on the step's totals only (surplus blocks leave at once)
         most = (T - single) // rc + (batch.S - single)
         chunks = torch.empty((most, H, dk, dv), dtype=torch.int32, device=dev)
-        launch(1, "retention_chunks", table=table, chunks=chunks, max_chunks=most, min_rows=min_rows,
+        decays = torch.empty((most, H), dtype=torch.float32, device=dev) if steps is not None else None
+        launch(1, "chunks", table=table, chunks=chunks, decays=decays, max_chunks=most, min_rows=min_rows,
                flops=4.0 * T * H * dk * dv)
     else:
-        raw = torch.empty((T, H, dv), dtype=torch.float32, device=dev)
-        launch(2, "retention_scan", table=table, raw=raw, min_rows=min_rows)
+        scratch = None if to_raw else torch.empty((T, H, dv), dtype=torch.float32, device=dev)
+        launch(2, "scan", table=table, scratch=scratch, min_rows=min_rows)
+
+
+def gated_norm(raw, gate, gate_col: int, weight, eps: float, out, H: int, dv: int, *, parts: int = 1, gate_first: bool = False,
+               skip=None, x=None, x_col: int = 0) -> None:
+    """The row of all heads' outputs ``raw`` [T, H * dv] float32: with ``skip`` [H] first ``y = raw + skip[h] * x`` (``x`` float32
+    rows, heads from column ``x_col`` on).  ``gate_first``: ``rms(y silu(gate)) * weight``, else ``rms(y) * weight *
+    sigmoid(gate)``; the root mean square is taken over ``parts`` equal parts of the row.  ``gate``: float32 rows, the gates from
+    column ``gate_col`` on."""
+    _cuda_contig(raw, weight, out, skip)
+    _f32(raw, gate, weight, skip, x)
+    T, n = raw.shape[0], H * dv
+    _need(raw.numel() == T * n and out.shape == (T, n) and weight.numel() == n and n % parts == 0, "gated_norm: shapes")
+    _need(gate.stride(1) == 1 and gate.shape[0] == T and gate.shape[1] >= gate_col + n, "gated_norm: gates")
+    _need(skip is None or (skip.numel() == H and x is not None and x.stride(1) == 1 and x.shape[1] >= x_col + n), "gated_norm: skip")
+    _check(lib().nv_gated_norm(_p(raw), _p(skip), (x.data_ptr() + 4 * x_col if x is not None else None),
+                               (x.stride(0) if x is not None else 0), gate.data_ptr() + 4 * gate_col, gate.stride(0), _p(weight),
+                               _p(out), dt(out), T, H, dv, parts, 1 if gate_first else 0, float(eps), _stream()), "gated_norm",
+           nbytes=float(T) * n * (8 + (4 if skip is not None else 0) + out.element_size()))
 
 
 def cols_rmsnorm(src, col0: int, n: int, w, eps: float, out) -> None:

@@ -126,7 +126,7 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(GemmArgs g) {
       float v = acc[i][j];
       if (SWIGLU) v = pair_mul(g.swiglu, v, acc2[i][j], g.act_p0, g.act_p1);
       if (g.bias) v += ld_dt(g.bias, g.bias_dt, n);
-      st_dt(g.out, g.out_dt, orow + n, epilogue_act(g.act, v, g.act_p0, g.act_p1));
+      st_dt(g.out, g.out_dt, orow + n, epilogue_act(epi_at(g.act, n, g.act_p0), v, g.act_p0, g.act_p1));
     }
   }
 }

@@ -67,6 +67,7 @@ struct NormArgs {
   // its input: both norms in one pass over the row.)
   const float* bw;
   float b_eps;
+  float scale, scale2;      // with two branches: what they are multiplied by
 };
 
 template <int VEC>
@@ -119,10 +120,10 @@ __global__ void __launch_bounds__(NORM_THREADS) add_rmsnorm_kernel(NormArgs a) {
     Chunk<VEC> r;
     if (a.branch) {
       r = ld_chunk<VEC>(a.branch + base + (size_t)c * VEC);
-      if (a.branch2) {          // x + (b + b2): the branches are summed first
+      if (a.branch2) {          // x + (s b + s2 b2): the branches are summed first
         Chunk<VEC> b2 = ld_chunk<VEC>(a.branch2 + base + (size_t)c * VEC);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) r.v[j] += b2.v[j];
+        for (int j = 0; j < VEC; ++j) r.v[j] = fmaf(a.scale2, b2.v[j], a.scale * r.v[j]);
       }
       return r;
     }
@@ -363,6 +364,14 @@ __global__ void __launch_bounds__(256) rope_store_kernel(void* __restrict__ qkv,
   // what is copied as it is: the part of k beyond the rotated dimensions, and v
   const int tail = D - rotary_dim;
   const int k_lo = max(h_begin, Hq), k_hi = min(h_end, Hq + Hkv);
+  if (packed && rotary_dim == 0) {                 // keys that are not turned at all: 16-byte copies
+    const int cpd = D / 8;
+    for (int i = threadIdx.x; i < (k_hi - k_lo) * cpd; i += blockDim.x) {
+      const int h = k_lo + i / cpd, c = i % cpd;
+      const size_t cbase = (((size_t)blk * Hkv + (h - Hq)) * page + slot) * D;
+      *((uint4*)((bf16*)kc + cbase) + c) = *((const uint4*)((const bf16*)qkv + row + (size_t)h * D) + c);
+    }
+  } else
   for (int i = threadIdx.x; i < (k_hi - k_lo) * tail; i += blockDim.x) {
     const int h = k_lo + i / tail, d = rotary_dim + i % tail;
     const size_t cbase = (((size_t)blk * Hkv + (h - Hq)) * page + slot) * D;
@@ -465,7 +474,7 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, long long l
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
   const int t = blockIdx.x * (blockDim.x / 32) + warp;
   if (t >= T) return;
-  route_row(logits + (size_t)t * ld, E, K, renorm, sm + (size_t)warp * E, lane, idx + (size_t)t * (K + C),
+  route_row(logits + (size_t)t * ld, E, K, renorm, sm + (size_t)warp * (E + rule.groups), lane, idx + (size_t)t * (K + C),
             score + (size_t)t * (K + C), C, (C && gate_logit) ? gate_logit + (size_t)t * gate_ld : nullptr, rule);
 }
 
@@ -622,8 +631,8 @@ NV_API int nv_embedding(const int* ids, const int* feed, const void* table, int 
 NV_API int nv_add_rmsnorm(float* x, const float* branch, const float* branch2, const void* w, int w_dt, float eps, void* out,
                           int out_dt, float* out32, int T, int H, const float* rows, const int* index,
                           const float* weight, int R, const float* dense, const float* gate_logit,
-                          long long gate_ld, const float* branch_w, float branch_eps, cudaStream_t s) {
-  // branch_w: the branch passes an RMS norm with this weight (and branch_eps) before it is added
+                          long long gate_ld, const float* branch_w, float branch_eps, float scale, float scale2, cudaStream_t s) {
+  // scale, scale2: what two branches are multiplied by.  branch_w: the branch passes an RMS norm with this weight (and branch_eps) before it is added
   if (!dt_ok(w_dt) || !dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
   if (branch_w && !(branch || R > 0 || dense)) return NV_ERR_BAD_SIZE;
   if (R < 0 || R > NORM_MAX_R || (R > 0 && (!rows || !index || !weight))) return NV_ERR_BAD_SIZE;
@@ -634,7 +643,7 @@ NV_API int nv_add_rmsnorm(float* x, const float* branch, const float* branch2, c
   a.x = x; a.branch = branch; a.branch2 = branch2; a.w = w; a.out = out; a.out32 = out32; a.rows = rows; a.index = index;
   a.weight = weight; a.dense = dense; a.gate_logit = gate_logit; a.gate_ld = gate_ld; a.eps = eps;
   a.w_dt = w_dt; a.out_dt = out_dt; a.H = H; a.R = R;
-  a.bw = branch_w; a.b_eps = branch_eps;
+  a.bw = branch_w; a.b_eps = branch_eps; a.scale = scale; a.scale2 = scale2;
   if (branch_w) {
     if (H % 4 == 0) NV_RETURN_IF(launch_dep(add_rmsnorm_kernel<4, true>, dim3(T), dim3(NORM_THREADS), 0, s, a));
     else NV_RETURN_IF(launch_dep(add_rmsnorm_kernel<1, true>, dim3(T), dim3(NORM_THREADS), 0, s, a));
@@ -684,15 +693,16 @@ NV_API int nv_paged_attention_plain(const void* qkv, int dt, int q_stride, const
 
 NV_API int nv_router_topk(const float* logits, long long ld, int T, int E, int K, int renorm, int* idx,
                           float* score, int C, const float* gate_logit, long long gate_ld, int mode,
-                          const float* choice_bias, float weight_scale, cudaStream_t s) {
+                          const float* choice_bias, float weight_scale, int groups, int keep, cudaStream_t s) {
   if (K < 1 || K > E || K > 32 || C < 0 || C > 32 || mode < 0 || mode > 1) return NV_ERR_UNSUPPORTED;
+  if (!route_groups_ok(E, K, groups, keep)) return NV_ERR_BAD_SIZE;
   if (T == 0) return NV_OK;
-  const int warps = 4;
-  size_t smem = (size_t)warps * E * sizeof(double);
-  if (smem > 48 * 1024) return NV_ERR_UNSUPPORTED;  // E <= 1536
+  const int warps = E + groups <= 1536 ? 4 : 2;
+  size_t smem = (size_t)warps * (E + groups) * sizeof(double);
+  if (smem > 48 * 1024) return NV_ERR_UNSUPPORTED;
   router_topk_kernel<<<(T + warps - 1) / warps, warps * 32, smem, s>>>(logits, ld, T, E, K, renorm, idx, score, C,
                                                                        gate_logit, gate_ld,
-                                                                       RouteRule{mode, choice_bias, weight_scale});
+                                                                       RouteRule{mode, choice_bias, weight_scale, groups, keep});
   NV_RETURN_LAST();
 }
 

@@ -1,16 +1,24 @@
-// Retention (linear attention with one fixed decay per head) and the causal convolution over a mixer's input.
+// Matrix memories that decay by one number per head (retention, lightning attention, the state-space dual form), and the
+// causal convolution over time.
 //
-//   causal_conv_add        out = h + conv(h), a short convolution over time on every channel, its history kept per request
+//   causal_conv            out = h + conv(h) or silu(conv(h) + bias), a short convolution over time on every channel, its
+//                          history kept per request
 //   rotary_table           cosine and sine of every row's angles, shared by the heads
-//   retention_step         entries of one row: rotation, state update, output, head norm and gate in one launch
+//   retention_step         entries of one row: rotation, state update, output (and head norm and gate) in one launch
 //   retention_scan         any sizes, row by row (the twin of the others; float32 runs)
 //   retention_chunk_*      entries of many rows on the tensor cores, 64 rows at a time
+//   gated_norm             a row's outputs of all heads: skip term, gate and RMS norm over equal parts of the row
 //
-// Per head with the decay d, keys k (turned by their positions, times dk^-1/2) and values v:
-//   S_t = d S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t,   y_t = o_t / sqrt(mean(o_t^2) + eps) * silu(gate_t).
+// Per head with the decay d, keys k (turned by their positions, times a constant) and values v:
+//   S_t = d S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t.
+// What follows is either y_t = o_t / sqrt(mean(o_t^2) + eps) * silu(gate_t) per head, in the same kernels, or o_t goes out in
+// float32 (gated_norm takes it).  The decay is a constant of the head, or it follows from a step size that every row has
+// per head (row decays): dt = softplus(z + bias), d = exp(-exp(a) dt), and the row's key is multiplied by dt.  Several heads
+// may share their q and k.
 // S lives in float32.  The chunked form writes the recurrence for the rows i = 0 .. n - 1 of a chunk that starts from S:
 //   o_i = d^(i+1) S^T q_i + sum_{j <= i} d^(i-j) (q_i . k_j) v_j,   S' = d^n S + sum_j d^(n-1-j) k_j v_j^T
-// in three launches: every chunk's own sum over j (all chunks at once), a pass over each entry's chunks that turns
+// (with row decays d^(i-j) is the product of the rows' decays from j + 1 to i, taken as a difference of running sums of
+// their logarithms) in three launches: every chunk's own sum over j (all chunks at once), a pass over each entry's chunks that turns
 // these into the states the chunks start from, and every chunk's outputs (all chunks at once).  All operands of the
 // tensor-core products are float32 numbers split into two bfloat16 terms (hi, and what its rounding left), with the
 // three products hi hi, hi lo and lo hi, so that a product carries sixteen bits of each operand; sums are float32.
@@ -22,15 +30,17 @@ namespace {
 
 // ------------------------------------------------------------------ causal convolution
 struct ConvArgs {
-  const float* h;           // [T, H]
+  const float* h;           // [T, H], rows `ld` apart
+  long long ld;
   const float* w;           // [taps, H]: row j multiplies the input taps - 1 - j positions back
+  const float* bias;        // [H] or nullptr
   const int* row_entry;
   const int* cu_rows;
   const int* entry_slot;
   float* state;             // per slot [taps - 1, H]: the inputs of the request's last taps - 1 positions
   long long slot_stride;
   void* out;
-  int out_dt, T, H, taps, rows, update;
+  int out_dt, T, H, taps, rows, update, act;           // act 0: h + conv(h); 1: silu(conv(h) + bias)
 };
 
 template <int VEC>
@@ -77,7 +87,7 @@ __device__ __forceinline__ void st_out(void* out, int dt, size_t i, const Vals<V
 // brought up to date here too, which is safe where every entry has one row (nobody else reads it).
 // The taps are added in ascending order of time, whatever the cut, so a row's result does not depend on it.
 template <int VEC, int TAPS>
-__global__ void __launch_bounds__(256) causal_conv_add_kernel(ConvArgs a) {
+__global__ void __launch_bounds__(256) causal_conv_kernel(ConvArgs a) {
   grid_dep_wait();
   grid_dep_launch();
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -96,12 +106,26 @@ __global__ void __launch_bounds__(256) causal_conv_add_kernel(ConvArgs a) {
     const int j = t - a.cu_rows[e];
     float* st = a.state + (size_t)a.entry_slot[e] * a.slot_stride + col;
     auto back = [&](int d) {
-      return j >= d ? ldv<VEC>(a.h + (size_t)(t - d) * a.H + col) : ldv<VEC>(st + (size_t)(taps - 1 + j - d) * a.H);
+      return j >= d ? ldv<VEC>(a.h + (size_t)(t - d) * a.ld + col) : ldv<VEC>(st + (size_t)(taps - 1 + j - d) * a.H);
     };
-    const Vals<VEC> cur = ldv<VEC>(a.h + (size_t)t * a.H + col);
+    const Vals<VEC> cur = ldv<VEC>(a.h + (size_t)t * a.ld + col);
     Vals<VEC> acc;
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc.v[i] = 0.f;
+    auto finish = [&](const Vals<VEC>& last) {         // the current token's tap, then what the mode adds or applies
+      if (a.act) {
+        Vals<VEC> b = acc;
+        if (a.bias) b = ldv<VEC>(a.bias + col);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          const float z = fmaf(last.v[i], cur.v[i], acc.v[i]) + (a.bias ? b.v[i] : 0.f);
+          acc.v[i] = z / (1.f + expf(-z));
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) acc.v[i] = cur.v[i] + fmaf(last.v[i], cur.v[i], acc.v[i]);
+      }
+    };
     if (TAPS > 0) {
       if (t == t0 || j == 0) {
 #pragma unroll
@@ -111,8 +135,7 @@ __global__ void __launch_bounds__(256) causal_conv_add_kernel(ConvArgs a) {
       for (int d = TAPS - 1; d >= 1; --d)
 #pragma unroll
         for (int i = 0; i < VEC; ++i) acc.v[i] = fmaf(w[TAPS - 1 - d].v[i], hist[d - 1].v[i], acc.v[i]);
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) acc.v[i] = cur.v[i] + fmaf(w[TAPS > 0 ? TAPS - 1 : 0].v[i], cur.v[i], acc.v[i]);
+      finish(w[TAPS > 0 ? TAPS - 1 : 0]);
       st_out<VEC>(a.out, a.out_dt, (size_t)t * a.H + col, acc);
 #pragma unroll
       for (int d = HN - 1; d >= 1; --d) hist[d] = hist[d - 1];
@@ -128,8 +151,7 @@ __global__ void __launch_bounds__(256) causal_conv_add_kernel(ConvArgs a) {
         for (int i = 0; i < VEC; ++i) acc.v[i] = fmaf(wd.v[i], x.v[i], acc.v[i]);
       }
       const Vals<VEC> wl = ldv<VEC>(a.w + (size_t)(taps - 1) * a.H + col);
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) acc.v[i] = cur.v[i] + fmaf(wl.v[i], cur.v[i], acc.v[i]);
+      finish(wl);
       st_out<VEC>(a.out, a.out_dt, (size_t)t * a.H + col, acc);
       if (a.update)
         for (int s = 0; s < taps - 1; ++s)
@@ -168,6 +190,16 @@ struct RetArgs {
   void* out;                // [T, H * dv]
   float* raw;               // scan: [T, H, dv]
   uint32_t* chunks;         // chunked form: per chunk and head dk * dv words (float32 sums, then the states' two terms)
+  int G;                    // heads of q and k: head h reads q/k head h / (H / G)
+  int raw_out;              // the outputs go to `raw` [T, H, dv] in float32, without norm and gate
+  // Row decays (dsrc != nullptr): step size dt = softplus(dsrc[t, d0 + h] + dt_bias[h]), decay exp(-exp(A_log[h]) dt), and
+  // the row's k times dt instead of k_scale.
+  const float* dsrc;
+  long long d_ld;
+  int d0;
+  const float* A_log;
+  const float* dt_bias;
+  float* chunk_decay;       // chunked form with row decays: [chunks, H], what a chunk multiplies its first state by
   // v2: the chunked form reads two neighbouring elements at a time; planes: the states' terms lie row by row (see the pass)
   int out_dt, H, dk, dv, num_entries, min_rows, slice, v2, planes;
 };
@@ -176,6 +208,10 @@ constexpr int RC = 64;                 // rows of a chunk
 constexpr int RT_THREADS = 256;
 
 __device__ __forceinline__ float silu_of(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float step_size_of(const RetArgs& a, int t, int h) {
+  const float z = a.dsrc[(size_t)t * a.d_ld + a.d0 + h] + a.dt_bias[h];
+  return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+}
 
 // ------------------------------------------------------------------ one row per entry
 // grid (rows, heads).  The head's matrix streams through registers once: a thread owns VEC neighbouring columns and every
@@ -205,22 +241,29 @@ __global__ void __launch_bounds__(RT_THREADS) retention_step_kernel(RetArgs a) {
   grid_dep_wait();
   grid_dep_launch();
   const int items = half + (dk - 2 * half);
+  const int gh = h / (a.H / a.G);
+  float d = 0.f, ks = a.k_scale;
+  if (a.dsrc) {
+    ks = step_size_of(a, t, h);
+    d = expf(-expf(a.A_log[h]) * ks);
+  } else {
+    d = a.powers[(size_t)h * (RC + 1) + 1];
+  }
   for (int i = tid; i < items; i += RT_THREADS) {
-    const float* pq = p + a.q0 + (size_t)h * dk;
-    const float* pk = p + a.k0 + (size_t)h * dk;
+    const float* pq = p + a.q0 + (size_t)gh * dk;
+    const float* pk = p + a.k0 + (size_t)gh * dk;
     if (i < half) {
       const float ang = (float)a.positions[t] * a.inv_freq[i];
       const float cs = cosf(ang), sn = sinf(ang);
       q[i] = pq[i] * cs - pq[i + half] * sn;
       q[i + half] = pq[i + half] * cs + pq[i] * sn;
-      k[i] = (pk[i] * cs - pk[i + half] * sn) * a.k_scale;
-      k[i + half] = (pk[i + half] * cs + pk[i] * sn) * a.k_scale;
+      k[i] = (pk[i] * cs - pk[i + half] * sn) * ks;
+      k[i + half] = (pk[i + half] * cs + pk[i] * sn) * ks;
     } else {
       q[i + half] = pq[i + half];
-      k[i + half] = pk[i + half] * a.k_scale;
+      k[i + half] = pk[i + half] * ks;
     }
   }
-  const float d = a.powers[(size_t)h * (RC + 1) + 1];
   __syncthreads();
   if (owner) {
     Vals<VEC> v, o;
@@ -258,8 +301,10 @@ __global__ void __launch_bounds__(RT_THREADS) retention_step_kernel(RetArgs a) {
     float o = 0.f;
     for (int i = 0; i < RS; ++i) o += share[(size_t)i * dv + c];
     share[c] = o;                      // (column c's shares are read by this thread alone)
+    if (a.raw_out) a.raw[((size_t)t * a.H + h) * dv + c] = o;
     ss = fmaf(o, o, ss);
   }
+  if (a.raw_out) return;
   ss = warp_sum(ss);
   if ((tid & 31) == 0) red[tid >> 5] = ss;
   __syncthreads();
@@ -285,22 +330,27 @@ __global__ void __launch_bounds__(RT_THREADS) retention_scan_kernel(RetArgs a) {
   float* share = k + dk;
   float* Sg = a.S + (size_t)a.entry_slot[e] * a.S_stride + (size_t)h * dk * dv;
   for (int r = rs; r < dk; r += RS) S[r * W + c] = col < dv ? Sg[(size_t)r * dv + col] : 0.f;
-  const float d = a.powers[(size_t)h * (RC + 1) + 1];
-  const int items = half + (dk - 2 * half);
+  const int items = half + (dk - 2 * half), gh = h / (a.H / a.G);
+  const float rate = a.dsrc ? expf(a.A_log[h]) : 0.f;
+  float d = a.dsrc ? 0.f : a.powers[(size_t)h * (RC + 1) + 1], ks = a.k_scale;
   for (int t = row0; t < row1; ++t) {
     const float* p = a.proj + (size_t)t * a.ld;
-    const float* pq = p + a.q0 + (size_t)h * dk;
-    const float* pk = p + a.k0 + (size_t)h * dk;
+    const float* pq = p + a.q0 + (size_t)gh * dk;
+    const float* pk = p + a.k0 + (size_t)gh * dk;
+    if (a.dsrc) {
+      ks = step_size_of(a, t, h);
+      d = expf(-rate * ks);
+    }
     for (int i = tid; i < items; i += RT_THREADS) {
       if (i < half) {
         const float2 cs = a.table[(size_t)t * half + i];
         q[i] = pq[i] * cs.x - pq[i + half] * cs.y;
         q[i + half] = pq[i + half] * cs.x + pq[i] * cs.y;
-        k[i] = (pk[i] * cs.x - pk[i + half] * cs.y) * a.k_scale;
-        k[i + half] = (pk[i + half] * cs.x + pk[i] * cs.y) * a.k_scale;
+        k[i] = (pk[i] * cs.x - pk[i + half] * cs.y) * ks;
+        k[i + half] = (pk[i + half] * cs.x + pk[i] * cs.y) * ks;
       } else {
         q[i + half] = pq[i + half];
-        k[i + half] = pk[i + half] * a.k_scale;
+        k[i + half] = pk[i + half] * ks;
       }
     }
     __syncthreads();
@@ -411,6 +461,27 @@ __device__ __forceinline__ void find_chunk(const int* cu_rows, int S, int min_ro
   if (lane == 0) info[0] = -1;
 }
 
+// Row decays of a chunk, worked out by warp 0: dt[i] the rows' step sizes, cl[i] the base-2 logarithm of the product of the
+// decays of rows 0 .. i.  Rows beyond n neither decay nor count.
+__device__ __forceinline__ void chunk_row_decays(const RetArgs& a, int h, int row0, int n, float* cl, float* dt) {
+  const int lane = threadIdx.x & 31, i = 2 * lane;
+  const float rate2 = expf(a.A_log[h]) * 1.4426950408889634f;
+  const float d0 = i < n ? step_size_of(a, row0 + i, h) : 0.f, d1 = i + 1 < n ? step_size_of(a, row0 + i + 1, h) : 0.f;
+  const float l0 = -rate2 * d0, l1 = -rate2 * d1;
+  float inc = l0 + l1;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float up = __shfl_up_sync(0xffffffffu, inc, o);
+    if (lane >= o) inc += up;
+  }
+  const float before = __shfl_up_sync(0xffffffffu, inc, 1);
+  const float first = (lane ? before : 0.f) + l0;
+  dt[i] = d0;
+  dt[i + 1] = d1;
+  cl[i] = first;
+  cl[i + 1] = first + l1;
+}
+
 // Rows row0 .. row0 + n - 1 of one q or k head, turned, times factor(row), as two bfloat16 terms in shared memory
 // [RC][LDS]; rows beyond n and elements beyond dk are zero.
 template <int DKP, typename F>
@@ -516,7 +587,7 @@ __device__ __forceinline__ void load_values(const RetArgs& a, const float* src, 
 }
 
 // Every chunk's own sum: U = sum_j d^(n-1-j) k_j v_j^T, float32 [dk][dv].  grid (chunks, heads).
-template <int DKP>
+template <int DKP, bool VAR>
 __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 ? 3 : 1) retention_chunk_sum_kernel(RetArgs a) {
   constexpr int LDS = DKP + 8;
   extern __shared__ __align__(16) uint8_t ck_smem[];
@@ -525,17 +596,24 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 ? 3 : 1) retention_chun
   bf16* vh = kl + RC * LDS;
   bf16* vl = vh + RC * VLD;
   __shared__ int info[3];
-  __shared__ float pw[RC + 1];
-  const int h = blockIdx.y, tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+  __shared__ float pw[RC + 1], dts[VAR ? RC : 1];      // powers of the decay; with row decays their running logarithms
+  const int h = blockIdx.y, gh = h / (a.H / a.G), tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
   grid_dep_wait();
   grid_dep_launch();
-  if (warp == 0) find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
-  for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
+  if (warp == 0) {
+    find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
+    __syncwarp();
+    if (VAR && info[0] >= 0) chunk_row_decays(a, h, info[1], info[2], pw, dts);
+  }
+  if (!VAR)
+    for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
   __syncthreads();
   if (info[0] < 0) return;
   const int row0 = info[1], n = info[2];
   const float ks = a.k_scale;
-  load_turned<DKP>(a, a.proj + a.k0 + (size_t)h * a.dk, row0, n, [&](int r) { return pw[n - 1 - r] * ks; }, kh, kl);
+  if (VAR && tid == 0) a.chunk_decay[(size_t)blockIdx.x * a.H + h] = exp2f(pw[n - 1]);
+  load_turned<DKP>(a, a.proj + a.k0 + (size_t)gh * a.dk, row0, n,
+                   [&](int r) { return VAR ? exp2f(pw[n - 1] - pw[r]) * dts[VAR ? r : 0] : pw[n - 1 - r] * ks; }, kh, kl);
   float* U = reinterpret_cast<float*>(a.chunks) + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
   const int g = lane / 4, tq = lane % 4;
   const bool even = (a.dv & 1) == 0;
@@ -620,7 +698,10 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs 
   const size_t size = (size_t)a.dk * dv, step = (size_t)a.H * size;
   uint32_t* p = a.chunks + ((size_t)first_s * a.H + h) * size + (size_t)d * dv;
   float* Sg = a.S + (size_t)a.entry_slot[e] * a.S_stride + (size_t)h * size + (size_t)d * dv;
-  const float full = a.powers[(size_t)h * (RC + 1) + RC], last = a.powers[(size_t)h * (RC + 1) + n - (count - 1) * RC];
+  const bool var = a.chunk_decay != nullptr;
+  const float full = var ? 0.f : a.powers[(size_t)h * (RC + 1) + RC];
+  const float last = var ? 0.f : a.powers[(size_t)h * (RC + 1) + n - (count - 1) * RC];
+  const float* dec = a.chunk_decay + (size_t)first_s * a.H + h;
   Vals<4> S[NJ];
 #pragma unroll
   for (int j = 0; j < NJ; ++j)
@@ -638,7 +719,7 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs 
 #pragma unroll
     for (int i = 0; i < U; ++i)
       if (c0 + i < count) {
-        const float f = c0 + i + 1 < count ? full : last;
+        const float f = var ? dec[(size_t)(c0 + i) * a.H] : (c0 + i + 1 < count ? full : last);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const int c = 4 * (lane + 32 * j);
@@ -675,7 +756,10 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
   const size_t step = (size_t)a.H * size;
   uint32_t* p = a.chunks + ((size_t)first_s * a.H + h) * size + i;
   float* Sg = a.S + (size_t)a.entry_slot[e] * a.S_stride + (size_t)h * size + i;
-  const float full = a.powers[(size_t)h * (RC + 1) + RC], last = a.powers[(size_t)h * (RC + 1) + n - (count - 1) * RC];
+  const bool var = a.chunk_decay != nullptr;
+  const float full = var ? 0.f : a.powers[(size_t)h * (RC + 1) + RC];
+  const float last = var ? 0.f : a.powers[(size_t)h * (RC + 1) + n - (count - 1) * RC];
+  const float* dec = a.chunk_decay + (size_t)first_s * a.H + h;
   float S = *Sg;
   constexpr int U = 8;                 // chunk sums in flight
   for (int c0 = 0; c0 < count; c0 += U) {
@@ -688,7 +772,7 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
         const bf16 hi = __float2bfloat16_rn(S);
         const __nv_bfloat162 pk = __halves2bfloat162(hi, __float2bfloat16_rn(S - __bfloat162float(hi)));
         p[(size_t)(c0 + j) * step] = *reinterpret_cast<const uint32_t*>(&pk);
-        S = fmaf(c0 + j + 1 < count ? full : last, S, u[j]);
+        S = fmaf(var ? dec[(size_t)(c0 + j) * a.H] : (c0 + j + 1 < count ? full : last), S, u[j]);
       }
   }
   *Sg = S;
@@ -699,7 +783,7 @@ __device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f +
 // Every chunk's outputs, its heads normed and gated.  grid (chunks, heads).  Two warps share sixteen rows: each takes half
 // of the keys for the weights, which both then read from shared memory, and half of every slab's columns.  NS: slabs of
 // 64 value columns.
-template <int DKP, int NS>
+template <int DKP, int NS, bool VAR>
 __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) retention_chunk_out_kernel(RetArgs a) {
   constexpr int LDS = DKP + 8;
   constexpr int KS = RC * LDS > DKP * VLD ? RC * LDS : DKP * VLD;      // the keys' place is the state's afterwards
@@ -714,18 +798,23 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
   bf16* pl = ph + RC * VLD;
   __shared__ float squares[2][RC];
   __shared__ int info[3];
-  __shared__ float pw[RC + 1];
-  const int h = blockIdx.y, tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+  __shared__ float pw[RC + 1], dts[VAR ? RC : 1];      // powers of the decay; with row decays their running logarithms
+  const int h = blockIdx.y, gh = h / (a.H / a.G), tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
   grid_dep_wait();
   grid_dep_launch();
-  if (warp == 0) find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
-  for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
+  if (warp == 0) {
+    find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
+    __syncwarp();
+    if (VAR && info[0] >= 0) chunk_row_decays(a, h, info[1], info[2], pw, dts);
+  }
+  if (!VAR)
+    for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
   __syncthreads();
   if (info[0] < 0) return;
   const int row0 = info[1], n = info[2];
   const float ks = a.k_scale;
-  load_turned<DKP>(a, a.proj + a.q0 + (size_t)h * a.dk, row0, n, [](int) { return 1.f; }, qh, ql);
-  load_turned<DKP>(a, a.proj + a.k0 + (size_t)h * a.dk, row0, n, [&](int) { return ks; }, kh, kl);
+  load_turned<DKP>(a, a.proj + a.q0 + (size_t)gh * a.dk, row0, n, [](int) { return 1.f; }, qh, ql);
+  load_turned<DKP>(a, a.proj + a.k0 + (size_t)gh * a.dk, row0, n, [&](int r) { return VAR ? dts[VAR ? r : 0] : ks; }, kh, kl);
   __syncthreads();
   const int g = lane / 4, tq = lane % 4;
   const int rb = warp >> 1, side = warp & 1;         // rows 16 rb .. 16 rb + 15; which half of the keys and columns
@@ -760,16 +849,17 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
     for (int i = 0; i < 4; ++i) {
       const int j = side * 32 + i * 8 + 2 * tq;
       uint32_t wh, wl;
-      split2(j <= r_lo ? s[i][0] * pw[r_lo - j] : 0.f, j + 1 <= r_lo ? s[i][1] * pw[r_lo - j - 1] : 0.f, wh, wl);
+      auto since = [&](int r, int from) { return VAR ? exp2f(pw[r] - pw[from]) : pw[r - from]; };   // decay from row `from` to r
+      split2(j <= r_lo ? s[i][0] * since(r_lo, j) : 0.f, j + 1 <= r_lo ? s[i][1] * since(r_lo, j + 1) : 0.f, wh, wl);
       *reinterpret_cast<uint32_t*>(ph + r_lo * VLD + j) = wh;
       *reinterpret_cast<uint32_t*>(pl + r_lo * VLD + j) = wl;
-      split2(j <= r_hi ? s[i][2] * pw[r_hi - j] : 0.f, j + 1 <= r_hi ? s[i][3] * pw[r_hi - j - 1] : 0.f, wh, wl);
+      split2(j <= r_hi ? s[i][2] * since(r_hi, j) : 0.f, j + 1 <= r_hi ? s[i][3] * since(r_hi, j + 1) : 0.f, wh, wl);
       *reinterpret_cast<uint32_t*>(ph + r_hi * VLD + j) = wh;
       *reinterpret_cast<uint32_t*>(pl + r_hi * VLD + j) = wl;
     }
   }
   const uint32_t* St = a.chunks + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
-  const float f_lo = pw[r_lo + 1], f_hi = pw[r_hi + 1];
+  const float f_lo = VAR ? exp2f(pw[r_lo]) : pw[r_lo + 1], f_hi = VAR ? exp2f(pw[r_hi]) : pw[r_hi + 1];
   float o[NS][4][4];
   float ss_lo = 0.f, ss_hi = 0.f;
 #pragma unroll
@@ -845,6 +935,27 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
       ss_hi = fmaf(oc[i][2], oc[i][2], fmaf(oc[i][3], oc[i][3], ss_hi));
     }
   }
+  if (a.raw_out) {
+#pragma unroll
+    for (int sl = 0; sl < NS; ++sl)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = half ? r_hi : r_lo;
+        if (r >= n) continue;
+        float* to = a.raw + ((size_t)(row0 + r) * a.H + h) * a.dv;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int col = sl * 64 + side * 32 + i * 8 + 2 * tq;
+          if (col >= a.dv) continue;
+          if (a.v2) *reinterpret_cast<float2*>(to + col) = make_float2(o[sl][i][2 * half], o[sl][i][2 * half + 1]);
+          else {
+            to[col] = o[sl][i][2 * half];
+            if (col + 1 < a.dv) to[col + 1] = o[sl][i][2 * half + 1];
+          }
+        }
+      }
+    return;
+  }
   ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 1);
   ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
   ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 1);
@@ -881,6 +992,87 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
     }
 }
 
+// ------------------------------------------------------------------ the row of all heads: skip, gate, norm
+struct GatedNormArgs {
+  const float* raw;         // [T, n]
+  const float* skip;        // [H] or nullptr: y += skip[h] * x[t, c]
+  const float* x;           // [T, x_ld]
+  long long x_ld;
+  const float* gate;        // [T, gate_ld]
+  long long gate_ld;
+  const float* w;           // [n]
+  void* out;                // [T, n]
+  int out_dt, n, dv, parts, gate_first;
+  float eps;
+};
+
+// gate_first: the parts of (o + skip x) silu(gate), each over its root mean square, times w; else the parts of o + skip x over
+// their root mean square, times w sigmoid(gate).  One block per (row, part); a thread keeps its first GN_KEEP chunks in
+// registers between the two passes and works further ones out again.  Sums in a fixed order.
+constexpr int GN_THREADS = 256, GN_KEEP = 4;
+template <int VEC>
+__global__ void __launch_bounds__(GN_THREADS) gated_norm_kernel(GatedNormArgs a) {
+  __shared__ float red[GN_THREADS / 32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  const int m = a.n / a.parts, base = blockIdx.y * m, chunks = m / VEC;
+  grid_dep_wait();
+  grid_dep_launch();
+  const float* raw = a.raw + (size_t)t * a.n + base;
+  const float* gate = a.gate + (size_t)t * a.gate_ld + base;
+  const float* x = a.x + (size_t)t * a.x_ld + base;
+  auto value = [&](int c) {
+    Vals<VEC> v = ldv<VEC>(raw + c * VEC);
+    if (a.skip) {
+      const Vals<VEC> xv = ldv<VEC>(x + c * VEC);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.skip[(base + c * VEC + i) / a.dv], xv.v[i], v.v[i]);
+    }
+    if (a.gate_first) {
+      const Vals<VEC> g = ldv<VEC>(gate + c * VEC);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v.v[i] *= silu_of(g.v[i]);
+    }
+    return v;
+  };
+  Vals<VEC> keep[GN_KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < GN_KEEP; ++u) {
+    const int c = tid + u * nt;
+    if (c < chunks) {
+      keep[u] = value(c);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(keep[u].v[i], keep[u].v[i], ss);
+    }
+  }
+  for (int c = tid + GN_KEEP * nt; c < chunks; c += nt) {
+    const Vals<VEC> v = value(c);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v.v[i], v.v[i], ss);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float sum = 0.f;
+  for (int i = 0; i < nt / 32; ++i) sum += red[i];
+  const float r = rsqrtf(sum / (float)m + a.eps);
+  auto emit = [&](int c, Vals<VEC> v) {
+    const Vals<VEC> wv = ldv<VEC>(a.w + base + c * VEC);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v.v[i] = v.v[i] * r * wv.v[i];
+    if (!a.gate_first) {
+      const Vals<VEC> g = ldv<VEC>(gate + c * VEC);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v.v[i] *= 1.f / (1.f + expf(-g.v[i]));
+    }
+    st_out<VEC>(a.out, a.out_dt, (size_t)t * a.n + base + (size_t)c * VEC, v);
+  };
+#pragma unroll
+  for (int u = 0; u < GN_KEEP; ++u)
+    if (tid + u * nt < chunks) emit(tid + u * nt, keep[u]);
+  for (int c = tid + GN_KEEP * nt; c < chunks; c += nt) emit(c, value(c));
+}
+
 template <typename K>
 int allow(K kernel, size_t bytes) {
   if (bytes > 227 * 1024) return NV_ERR_UNSUPPORTED;
@@ -901,46 +1093,52 @@ size_t chunk_out_smem() {
   return sizeof(bf16) * (2 * (size_t)RC * (DKP + 8) + 2 * ks + 4 * (size_t)RC * VLD);
 }
 
-template <int DKP, int NS>
+template <int DKP, int NS, bool VAR>
 int launch_chunks(const RetArgs& a, int max_chunks, cudaStream_t s) {
-  int rc = allow(retention_chunk_sum_kernel<DKP>, chunk_sum_smem<DKP>());
+  int rc = allow(retention_chunk_sum_kernel<DKP, VAR>, chunk_sum_smem<DKP>());
   if (rc) return rc;
-  rc = allow(retention_chunk_out_kernel<DKP, NS>, chunk_out_smem<DKP>());
+  rc = allow(retention_chunk_out_kernel<DKP, NS, VAR>, chunk_out_smem<DKP>());
   if (rc) return rc;
   const dim3 grid(max_chunks, a.H);
-  NV_RETURN_IF(launch_dep(retention_chunk_sum_kernel<DKP>, grid, dim3(CK_THREADS), chunk_sum_smem<DKP>(), s, a));
+  NV_RETURN_IF(launch_dep(retention_chunk_sum_kernel<DKP, VAR>, grid, dim3(CK_THREADS), chunk_sum_smem<DKP>(), s, a));
   const dim3 rows(a.num_entries, a.H, (a.dk + 7) / 8);
   if (a.planes && a.dv <= 128) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<1>, rows, dim3(256), 0, s, a));
   else if (a.planes) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<2>, rows, dim3(256), 0, s, a));
   else NV_RETURN_IF(launch_dep(retention_chunk_pass_kernel, dim3(a.num_entries, a.H, (a.dk * a.dv + 255) / 256), dim3(256), 0, s, a));
-  NV_RETURN_IF(launch_dep(retention_chunk_out_kernel<DKP, NS>, grid, dim3(CK_THREADS), chunk_out_smem<DKP>(), s, a));
+  NV_RETURN_IF(launch_dep(retention_chunk_out_kernel<DKP, NS, VAR>, grid, dim3(CK_THREADS), chunk_out_smem<DKP>(), s, a));
   NV_RETURN_LAST();
 }
 
-template <int DKP>
+template <int DKP, bool VAR>
 int launch_chunks_ns(const RetArgs& a, int max_chunks, cudaStream_t s) {
-  if (a.dv <= 64) return launch_chunks<DKP, 1>(a, max_chunks, s);
-  if (a.dv <= 128) return launch_chunks<DKP, 2>(a, max_chunks, s);
-  return launch_chunks<DKP, 4>(a, max_chunks, s);
+  if (a.dv <= 64) return launch_chunks<DKP, 1, VAR>(a, max_chunks, s);
+  if (a.dv <= 128) return launch_chunks<DKP, 2, VAR>(a, max_chunks, s);
+  return launch_chunks<DKP, 4, VAR>(a, max_chunks, s);
+}
+template <int DKP>
+int launch_chunks_dk(const RetArgs& a, int max_chunks, cudaStream_t s) {
+  return a.dsrc ? launch_chunks_ns<DKP, true>(a, max_chunks, s) : launch_chunks_ns<DKP, false>(a, max_chunks, s);
 }
 
 }  // namespace
 
-// out = h + conv(h).  h: [T, H] float32; w: [taps, H] float32; state: per slot [taps - 1, H] float32 (nullptr with one
-// tap).  `update` (allowed where every entry of the step has one row): the state is brought up to date as well.
-NV_API int nv_causal_conv_add(const float* h, const float* w, int taps, const int* row_entry, const int* cu_rows,
-                              const int* entry_slot, float* state, long long slot_stride, void* out, int out_dt, int T,
-                              int H, int update, cudaStream_t s) {
+// act 0: out = h + conv(h); act 1: out = silu(conv(h) + bias).  h: [T, H] float32, rows `ld` apart; w: [taps, H] float32;
+// bias: [H] or nullptr; state: per slot [taps - 1, H] float32 (nullptr with one tap).  `update` (allowed where every entry
+// of the step has one row): the state is brought up to date as well.
+NV_API int nv_causal_conv(const float* h, long long ld, const float* w, const float* bias, int act, int taps,
+                          const int* row_entry, const int* cu_rows, const int* entry_slot, float* state,
+                          long long slot_stride, void* out, int out_dt, int T, int H, int update, cudaStream_t s) {
   if (!dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
-  if (taps < 1 || H < 1 || (taps > 1 && !state)) return NV_ERR_BAD_SIZE;
+  if (taps < 1 || H < 1 || ld < H || (taps > 1 && !state) || act < 0 || act > 1 || (bias && !act)) return NV_ERR_BAD_SIZE;
   if (T == 0) return NV_OK;
-  ConvArgs a = {h, w, row_entry, cu_rows, entry_slot, state, slot_stride, out, out_dt, T, H, taps, T > 512 ? 8 : 1, update};
-  const bool vec = H % 4 == 0 && slot_stride % 4 == 0 && !((uintptr_t)h & 15) && !((uintptr_t)w & 15) && !((uintptr_t)state & 15)
+  ConvArgs a = {h, ld, w, bias, row_entry, cu_rows, entry_slot, state, slot_stride, out, out_dt, T, H, taps,
+                T > 512 ? 8 : 1, update, act};
+  const bool vec = H % 4 == 0 && ld % 4 == 0 && slot_stride % 4 == 0 && !((uintptr_t)bias & 15) && !((uintptr_t)h & 15) && !((uintptr_t)w & 15) && !((uintptr_t)state & 15)
                    && !((uintptr_t)out & 15);
   const int chunks = vec ? H / 4 : H;
   const int threads = chunks < 256 ? (chunks + 31) / 32 * 32 : 256;
   const dim3 grid((T + a.rows - 1) / a.rows, (chunks + threads - 1) / threads);
-#define NV_CONV(VEC, TAPS) NV_RETURN_IF(launch_dep(causal_conv_add_kernel<VEC, TAPS>, grid, dim3(threads), 0, s, a))
+#define NV_CONV(VEC, TAPS) NV_RETURN_IF(launch_dep(causal_conv_kernel<VEC, TAPS>, grid, dim3(threads), 0, s, a))
 #define NV_CONV_TAPS(VEC)            \
   switch (taps) {                    \
     case 2: NV_CONV(VEC, 2); break;  \
@@ -984,8 +1182,14 @@ NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k
                         const int* positions, const float* inv_freq, int half, const int* row_entry, const int* cu_rows,
                         const int* entry_slot, int num_entries, const int* rows, int R, float* S, long long S_stride,
                         const float* powers, float k_scale, float eps, void* out, int out_dt, float* raw, void* chunks,
-                        int max_chunks, int T, int H, int dk, int dv, int min_rows, cudaStream_t s) {
+                        int max_chunks, int T, int H, int dk, int dv, int min_rows, int G, int raw_out, const float* dsrc,
+                        long long d_ld, int d0, const float* A_log, const float* dt_bias, float* chunk_decay,
+                        cudaStream_t s) {
+  // G: heads of q and k.  raw_out: the outputs go to `raw` in float32, without norm and gate (any `what`; `out` is then not
+  // written).  dsrc: row decays, from the step sizes' pre-activations [T, d_ld] at column d0 (head h's at d0 + h), with
+  // A_log [H] and dt_bias [H]; `powers` may then be nullptr, and what 1 takes chunk_decay [max_chunks, H] as scratch.
   if (!dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
+  if (G < 1 || H % G || (raw_out && !raw) || (!dsrc && !powers) || (dsrc && (!A_log || !dt_bias))) return NV_ERR_BAD_SIZE;
   if (H < 1 || half < 0 || 2 * half > dk || num_entries < 0) return NV_ERR_BAD_SIZE;
   if (!nv_retention_usable(what, dk, dv)) return NV_ERR_UNSUPPORTED;
   if (T == 0 || num_entries == 0) return NV_OK;
@@ -995,6 +1199,8 @@ NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k
   a.entry_slot = entry_slot; a.rows = rows; a.S = S; a.S_stride = S_stride; a.powers = powers; a.k_scale = k_scale;
   a.eps = eps; a.out = out; a.raw = raw; a.chunks = (uint32_t*)chunks; a.out_dt = out_dt; a.H = H; a.dk = dk; a.dv = dv;
   a.num_entries = num_entries; a.min_rows = min_rows;
+  a.G = G; a.raw_out = raw_out; a.dsrc = dsrc; a.d_ld = d_ld; a.d0 = d0; a.A_log = A_log; a.dt_bias = dt_bias;
+  a.chunk_decay = nullptr;
   if (what == 0) {
     if (R == 0) return NV_OK;
     const bool vec = step_vec(dv) == 4 && S_stride % 4 == 0 && !((uintptr_t)S & 15);
@@ -1009,14 +1215,15 @@ NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k
   }
   if (half > 0 && !table) return NV_ERR_BAD_SIZE;
   if (what == 1) {
-    if (!chunks || max_chunks < 1) return NV_ERR_BAD_SIZE;
+    if (!chunks || max_chunks < 1 || (dsrc && !chunk_decay)) return NV_ERR_BAD_SIZE;
+    if (dsrc) a.chunk_decay = chunk_decay;
     a.v2 = (half % 2 == 0 && dk % 2 == 0 && dv % 2 == 0 && ld % 2 == 0 && q0 % 2 == 0 && k0 % 2 == 0 && v0 % 2 == 0 &&
             g0 % 2 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)table & 15) && !((uintptr_t)chunks & 15) &&
-            !((uintptr_t)out & 15)) ? 1 : 0;
+            !((uintptr_t)out & 15) && !((uintptr_t)raw & 7)) ? 1 : 0;
     a.planes = (dv % 8 == 0 && S_stride % 4 == 0 && !((uintptr_t)S & 15) && !((uintptr_t)chunks & 15)) ? 1 : 0;
-    if (dk <= 64) return launch_chunks_ns<64>(a, max_chunks, s);
-    if (dk <= 128) return launch_chunks_ns<128>(a, max_chunks, s);
-    return launch_chunks_ns<256>(a, max_chunks, s);
+    if (dk <= 64) return launch_chunks_dk<64>(a, max_chunks, s);
+    if (dk <= 128) return launch_chunks_dk<128>(a, max_chunks, s);
+    return launch_chunks_dk<256>(a, max_chunks, s);
   }
   if (!raw) return NV_ERR_BAD_SIZE;
   a.slice = 32;
@@ -1026,7 +1233,29 @@ NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k
   retention_scan_kernel<<<dim3(num_entries, H, (dv + a.slice - 1) / a.slice), RT_THREADS, smem, s>>>(a);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
+  if (raw_out) return NV_OK;
   const long long items = (long long)T * H;
   retention_finish_kernel<<<(unsigned)((items + 7) / 8), 256, 0, s>>>(a, T);
+  NV_RETURN_LAST();
+}
+
+// out[t, :] from raw [T, n] (n = H * dv), see gated_norm_kernel.  skip: [H] with x [T, x_ld], or nullptr; gate: [T, gate_ld];
+// w: [n]; the norm is taken over `parts` equal parts of the row.  gate_first: silu(gate) before the norm, else sigmoid(gate)
+// behind it.
+NV_API int nv_gated_norm(const float* raw, const float* skip, const float* x, long long x_ld, const float* gate,
+                         long long gate_ld, const float* w, void* out, int out_dt, int T, int H, int dv, int parts,
+                         int gate_first, float eps, cudaStream_t s) {
+  if (!dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
+  if (H < 1 || dv < 1 || parts < 1 || parts > 65535 || (H * dv) % parts || (skip && !x)) return NV_ERR_BAD_SIZE;
+  if (T == 0) return NV_OK;
+  GatedNormArgs a = {raw, skip, x, x_ld, gate, gate_ld, w, out, out_dt, H * dv, dv, parts, gate_first, eps};
+  if (!x) a.x = raw;                     // (never read)
+  const int m = a.n / parts;
+  const bool vec = m % 4 == 0 && gate_ld % 4 == 0 && (!skip || (x_ld % 4 == 0 && !((uintptr_t)x & 15))) &&
+                   !((uintptr_t)raw & 15) && !((uintptr_t)gate & 15) && !((uintptr_t)w & 15) && !((uintptr_t)out & 15);
+  const int chunks = vec ? m / 4 : m;
+  const int threads = chunks < GN_THREADS ? (chunks + 31) / 32 * 32 : GN_THREADS;
+  if (vec) NV_RETURN_IF(launch_dep(gated_norm_kernel<4>, dim3(T, parts), dim3(threads), 0, s, a));
+  else NV_RETURN_IF(launch_dep(gated_norm_kernel<1>, dim3(T, parts), dim3(threads), 0, s, a));
   NV_RETURN_LAST();
 }

@@ -619,7 +619,7 @@ __global__ void __launch_bounds__(ATTG_THREADS) paged_attention_general_kernel(
     const int* __restrict__ block_table, int max_blocks, const int* __restrict__ row_entry,
     const int* __restrict__ positions, float scale, int window, int keep_first, int has_sink, float sink_score,
     const float* __restrict__ sinks, void* __restrict__ out, int out_dt, int Hq, int Hkv, int Hv, int D, int Dv,
-    int KS, int page, float softcap, HeadGate gate) {
+    int KS, int page, float softcap, HeadGate gate, int chunk, ScoreBias bias) {
   extern __shared__ float qs[];      // KS * D
   __shared__ float p[ATTG_THREADS];
   __shared__ int pslot[ATTG_THREADS];
@@ -628,7 +628,7 @@ __global__ void __launch_bounds__(ATTG_THREADS) paged_attention_general_kernel(
   const int kvh = KS > 1 ? 0 : h / (Hq / Hkv);     // first key head of the score
   const int vh = h / (Hq / Hv);                    // the head's value head
   const int n = positions[t] + 1;
-  const int lo = window > 0 ? max(0, n - window) : 0;
+  const int lo = first_visible(n - 1, window, chunk);
   const int nkeep = min(keep_first, lo);           // kept positions that the window no longer covers
   const int total = nkeep + (n - lo);
   const int* bt = block_table + (size_t)row_entry[t] * max_blocks;
@@ -657,6 +657,7 @@ __global__ void __launch_bounds__(ATTG_THREADS) paged_attention_general_kernel(
       (void)slot;
       s = acc * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      if (bias.slope || bias.table) s += score_bias_of(bias, h, n - 1 - j);
     }
     // maximum over the chunk
     float mx = warp_max(s);
@@ -1401,7 +1402,11 @@ NV_API int nv_paged_attention_general(const void* q, int q_dt, const void* kc, c
                                       const int* positions, float scale, int window, int keep_first, int has_sink,
                                       float sink_score, const float* sinks, void* out, int out_dt, int T, int Hq,
                                       int Hkv, int Hv, int D, int Dv, int key_span, int page, float softcap,
-                                      const float* gate, long long gate_ld, cudaStream_t s) {
+                                      const float* gate, long long gate_ld, int chunk, const float* slopes,
+                                      const float* bias_table, int bias_len, cudaStream_t s) {
+  // chunk > 0: a row at position p sees the positions from p / chunk * chunk on; slopes [Hq], bias_table [Hq, bias_len]: what
+  // the distance n takes off a head's score, slopes[h] * n, and gives to it, bias_table[h][min(n, bias_len - 1)], after the cap
+  if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0)) || (bias_table && bias_len < 1)) return NV_ERR_BAD_SIZE;
   if (!dt_ok(q_dt) || !dt_ok(cache_dt) || !dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
   if (D <= 0 || Dv <= 0 || Dv > ATTG_NV * ATTG_THREADS || Hkv <= 0 || Hv <= 0 || Hq % Hv || keep_first < 0)
     return NV_ERR_UNSUPPORTED;
@@ -1412,7 +1417,8 @@ NV_API int nv_paged_attention_general(const void* q, int q_dt, const void* kc, c
   if (rc) return rc;
   paged_attention_general_kernel<<<dim3(T, Hq), ATTG_THREADS, smem, s>>>(
       q, q_dt, kc, vc, cache_dt, block_table, max_blocks, row_entry, positions, scale, window, keep_first, has_sink,
-      sink_score, sinks, out, out_dt, Hq, Hkv, Hv, D, Dv, key_span, page, softcap, HeadGate{gate, gate_ld});
+      sink_score, sinks, out, out_dt, Hq, Hkv, Hv, D, Dv, key_span, page, softcap, HeadGate{gate, gate_ld}, chunk,
+      ScoreBias{slopes, bias_table, bias_len - 1});
   NV_RETURN_LAST();
 }
 

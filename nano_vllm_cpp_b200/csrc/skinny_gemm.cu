@@ -162,7 +162,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32, 1) skinny_kernel(SkArgs a) {
       if (feat < a.N && row < a.R) {
         float out = SWIGLU ? pair_mul(a.pair, v[0], v[NA - 1], a.act_p0, a.act_p1) : v[0];
         if (!SWIGLU && a.bias) out += ld_dt(a.bias, a.bias_dt, feat);
-        st_dt(a.out, a.out_dt, (size_t)row * a.ldo + feat, SWIGLU ? out : epilogue_act(a.act, out, a.act_p0, a.act_p1));
+        st_dt(a.out, a.out_dt, (size_t)row * a.ldo + feat, SWIGLU ? out : epilogue_act(epi_at(a.act, feat, a.act_p0), out, a.act_p0, a.act_p1));
       }
     }
   };

@@ -207,11 +207,11 @@ __global__ void __launch_bounds__(1024) moe_route_small_kernel(
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
   const int KT = K + C;
   for (int t = warp; t < T; t += 32)
-    route_row(logits + (size_t)t * ld, E, K, renorm, rs_smem + (size_t)warp * E, lane, idx + (size_t)t * KT,
+    route_row(logits + (size_t)t * ld, E, K, renorm, rs_smem + (size_t)warp * (E + rule.groups), lane, idx + (size_t)t * KT,
               score + (size_t)t * KT, C, (C && gate_logit) ? gate_logit + (size_t)t * gate_ld : nullptr, rule);
   __threadfence_block();
   __syncthreads();
-  int* al_s = (int*)(rs_smem + (size_t)32 * E);
+  int* al_s = (int*)(rs_smem + (size_t)32 * (E + rule.groups));
   align_block(idx, T * KT, KT, E + C, tile_m, counts, offsets, sorted_token, pair_pos, tile_expert, tile_row0,
               tile_rows, num_tiles, err, al_s, 0, nullptr, nullptr, nullptr, nullptr, n_static);
   if (!x_sorted) return;
@@ -301,8 +301,8 @@ NV_API int nv_rowdot(const float* a, long long lda, const void* w, int w_dt, flo
 }
 
 // Largest batch the fused routing kernel takes: rows and pairs one block can walk in a few microseconds.
-NV_API int nv_moe_route_small_usable(int T, int E, int K, int C, int H) {
-  const size_t smem = (size_t)32 * E * sizeof(double) + (size_t)4 * (E + C) * sizeof(int);
+NV_API int nv_moe_route_small_usable(int T, int E, int K, int C, int H, int groups) {
+  const size_t smem = (size_t)32 * (E + groups) * sizeof(double) + (size_t)4 * (E + C) * sizeof(int);
   return T <= 64 && T * (K + C) <= 1024 && smem <= 48 * 1024 && H % 8 == 0 && K <= 32 && C <= 32;
 }
 
@@ -311,15 +311,16 @@ NV_API int nv_moe_route_small(const float* logits, long long ld, int T, int E, i
                               int* counts, int* offsets, int* sorted_token, int* pair_pos, int* tile_expert,
                               int* tile_row0, int* tile_rows, int* num_tiles, int* err, const void* x,
                               void* x_sorted, int H, int n_static, int* zero, int n_zero, int mode,
-                              const float* choice_bias, float weight_scale, cudaStream_t s) {
-  if (!nv_moe_route_small_usable(T, E, K, C, H) || K < 1 || K > E || mode < 0 || mode > 1) return NV_ERR_UNSUPPORTED;
+                              const float* choice_bias, float weight_scale, int groups, int keep, cudaStream_t s) {
+  if (!route_groups_ok(E, K, groups, keep)) return NV_ERR_BAD_SIZE;
+  if (!nv_moe_route_small_usable(T, E, K, C, H, groups) || K < 1 || K > E || mode < 0 || mode > 1) return NV_ERR_UNSUPPORTED;
   if (n_zero < 0 || n_zero > 1024 || (n_zero && !zero)) return NV_ERR_BAD_SIZE;
   if (n_static != 0 && n_static != C) return NV_ERR_UNSUPPORTED;
   if (T == 0) return NV_OK;
-  const size_t smem = (size_t)32 * E * sizeof(double) + (size_t)4 * (E + C) * sizeof(int);
+  const size_t smem = (size_t)32 * (E + groups) * sizeof(double) + (size_t)4 * (E + C) * sizeof(int);
   NV_RETURN_IF(launch_dep(moe_route_small_kernel, dim3(1), dim3(1024), smem, s, logits, ld, T, E, K, renorm, C,
                           gate_logit, gate_ld, idx, score, tile_m, counts, offsets, sorted_token, pair_pos, tile_expert,
                           tile_row0, tile_rows, num_tiles, err, (const bf16*)x, (bf16*)x_sorted, H, n_static, zero,
-                          n_zero, RouteRule{mode, choice_bias, weight_scale}));
+                          n_zero, RouteRule{mode, choice_bias, weight_scale, groups, keep}));
   NV_RETURN_LAST();
 }

@@ -195,8 +195,8 @@ __device__ __forceinline__ void epilogue_chunk(const TcArgs& a, const Tile& t, i
     for (int j = 0; j < W; ++j) {
       if (j < valid) {
         const float v = (a.swiglu ? pair_mul(a.swiglu, g[j], u[j], a.act_p0, a.act_p1) : g[j]) + bias;
-        st_dt(a.out, a.out_dt, (row + j) * a.ldo + t.o_col0 + n, epilogue_act(a.act, v, a.act_p0, a.act_p1));
-        if (n2_ok) st_dt(a.out, a.out_dt, (row + j) * a.ldo + t.o_col0 + n2, epilogue_act(a.act, u[j] + bias2, a.act_p0, a.act_p1));
+        st_dt(a.out, a.out_dt, (row + j) * a.ldo + t.o_col0 + n, epilogue_act(epi_at(a.act, n, a.act_p0), v, a.act_p0, a.act_p1));
+        if (n2_ok) st_dt(a.out, a.out_dt, (row + j) * a.ldo + t.o_col0 + n2, epilogue_act(epi_at(a.act, n2, a.act_p0), u[j] + bias2, a.act_p0, a.act_p1));
       }
     }
     return;
@@ -220,6 +220,16 @@ __device__ __forceinline__ void epilogue_chunk(const TcArgs& a, const Tile& t, i
     case NV_EPI_GELU_TANH: chunk_act<W, NV_EPI_GELU_TANH>(g, u, a.act_p0, a.act_p1); break;
     case NV_EPI_SILU: chunk_act<W, NV_EPI_SILU>(g, u, a.act_p0, a.act_p1); break;
     case NV_EPI_XIELU: chunk_act<W, NV_EPI_XIELU>(g, u, a.act_p0, a.act_p1); break;
+    case NV_EPI_SILU_FIRST:
+      if (n < (int)a.act_p0) {
+#pragma unroll
+        for (int j = 0; j < W; ++j) g[j] = epilogue_act(NV_EPI_SILU, g[j]);
+      }
+      if (n2_ok && n2 < (int)a.act_p0) {
+#pragma unroll
+        for (int j = 0; j < W; ++j) u[j] = epilogue_act(NV_EPI_SILU, u[j]);
+      }
+      break;
     default: chunk_act<W, NV_EPI_RELU2>(g, u, a.act_p0, a.act_p1); break;
   }
   if (a.out_dt == NV_DT_BF16) {
@@ -491,8 +501,8 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
               if (n2_ok) p[n2] = u[j];
             } else {
               float v = a.swiglu ? pair_mul(a.swiglu, g[j], u[j], a.act_p0, a.act_p1) : g[j];
-              st_dt(a.out, a.out_dt, row * a.ldo + t.o_col0 + n, epilogue_act(a.act, v + bias, a.act_p0, a.act_p1));
-              if (n2_ok) st_dt(a.out, a.out_dt, row * a.ldo + t.o_col0 + n2, epilogue_act(a.act, u[j] + bias2, a.act_p0, a.act_p1));
+              st_dt(a.out, a.out_dt, row * a.ldo + t.o_col0 + n, epilogue_act(epi_at(a.act, n, a.act_p0), v + bias, a.act_p0, a.act_p1));
+              if (n2_ok) st_dt(a.out, a.out_dt, row * a.ldo + t.o_col0 + n2, epilogue_act(epi_at(a.act, n2, a.act_p0), u[j] + bias2, a.act_p0, a.act_p1));
             }
           }
         }
@@ -528,7 +538,7 @@ __global__ void tc_gemm_finish_kernel(const float* __restrict__ partial, int spl
   }
   float v = swiglu ? pair_mul(swiglu, g, u, act_p0, act_p1) : g;
   if (bias) v += ld_dt(bias, bias_dt, n);
-  st_dt(out, out_dt, t * ldo + n, epilogue_act(act, v, act_p0, act_p1));
+  st_dt(out, out_dt, t * ldo + n, epilogue_act(epi_at(act, n, act_p0), v, act_p0, act_p1));
 }
 
 // The same for a grouped product: only the rows that the tile list covers are finished (other rows of `out` belong
@@ -554,7 +564,7 @@ __global__ void tc_gemm_finish_grouped_kernel(const float* __restrict__ partial,
       g += p[n];
       if (swiglu) u += p[N + n];
     }
-    st_dt(out, out_dt, (long long)r * ldo + n, swiglu ? pair_mul(swiglu, g, u, act_p0, act_p1) : epilogue_act(act, g, act_p0, act_p1));
+    st_dt(out, out_dt, (long long)r * ldo + n, swiglu ? pair_mul(swiglu, g, u, act_p0, act_p1) : epilogue_act(epi_at(act, n, act_p0), g, act_p0, act_p1));
   }
 }
 

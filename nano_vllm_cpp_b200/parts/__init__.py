@@ -4,7 +4,7 @@ from .base import (TensorSpec, KVCacheSpec, StateCacheSpec, CompositeCacheSpec, 
 from .registry import register_part, build_part
 from . import norm, rotary, convolution, attention, latent_attention, feedforward, recurrent, parallel, token_input  # noqa: F401  (register themselves)
 from .block import Arrangement, LayerSpec, PreNormBlock, build_layer
-from . import streams  # noqa: F401
+from . import streams, passes  # noqa: F401
 from .model import LayerCall, ModelSpec, Model
 
 __all__ = ["TensorSpec", "KVCacheSpec", "StateCacheSpec", "CompositeCacheSpec", "SharedCacheSpec", "TokenInput", "InputFilter", "RunContext", "Part", "Norm", "PositionEncoding",

@@ -56,11 +56,22 @@ class PagedAttention(Mixer):
     ``sigmoid(Wg h)_h``, one number per head and row (tensor ``g`` [heads, hidden]), where the attention kernel writes
     it.  ``own_kv`` False: the layer has no k and v tensors; its call reads the pages of an earlier call (whose kv heads
     and head sizes are the same) with its own queries, and writes none.
+
+    Three more, of the same path.  ``chunk`` > 0 instead of a window: row i sees the positions of its own chunk of so many,
+    counted from the sequence's start (``j <= i`` and ``j // chunk == i // chunk``).  ``distance_slopes`` (one number per
+    query head): a score loses ``slope * (i - j)``, behind the cap.  ``distance_far``: a score gains a learned number that
+    depends on head and distance, also behind the cap: row ``bucket(i - j)`` of the tensor ``rel`` [rows, heads], where
+    distances below half of the rows have a row each and the others share the rest on a logarithmic scale that ends at
+    ``distance_far`` (``distance_buckets``); the number of rows is the file's (``distance_rows`` for random weights).
+
+    A layer of this path without head norms, positions, gates and borrowed keys skips the float32 projection in bfloat16
+    runs: its projection makes bfloat16 rows that the attention kernels read in place, heads padded to one size in the
+    weights.
     """
 
     _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
               "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias", "g": "g_proj.weight",
-              "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "head_mix": "head_mix", "sink": "sink"}
+              "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "head_mix": "head_mix", "sink": "sink", "rel": "rel"}
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, bias: bool,
                  position: PartSpec, window: int = 0, scale: float | None = None, v_head_dim: int | None = None,
@@ -69,7 +80,8 @@ class PagedAttention(Mixer):
                  keep_first: int = 0, learned_sink: bool = False, head_mix: bool = False,
                  value_position: PartSpec | None = None, qk_norm_weight: bool = True,
                  qk_norm_after_rotation: bool = False, score_softcap: float = 0.0, round_weights: bool = False,
-                 qk_norm_whole: bool = False, output_gate: bool = False, own_kv: bool = True):
+                 qk_norm_whole: bool = False, output_gate: bool = False, own_kv: bool = True, chunk: int = 0,
+                 distance_slopes: list | None = None, distance_far: int | None = None, distance_rows: int = 32):
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
         self.hidden, self.Hq, self.Hkv, self.D = hidden_size, num_heads, num_kv_heads, head_dim
@@ -108,6 +120,17 @@ class PagedAttention(Mixer):
             raise ValueError("a norm over all heads comes with its eps and precedes the turn")
         if not self.own_kv and (bias or self.values_from_keys):
             raise ValueError("a layer without keys and values of its own has no biases of theirs")
+        self.chunk = int(chunk)
+        self.distance_slopes = None if distance_slopes is None else [float(s) for s in distance_slopes]
+        self.distance_far = None if distance_far is None else int(distance_far)
+        self.distance_rows = int(distance_rows)
+        if self.chunk < 0 or (self.chunk and self.window):
+            raise ValueError("a layer sees a window or its own chunk, not both")
+        if self.distance_slopes is not None and len(self.distance_slopes) != num_heads:
+            raise ValueError("distance_slopes: one number per query head")
+        if self.distance_far is not None and self.distance_far < 1:
+            raise ValueError("distance_far must be positive")
+        scored = bool(self.chunk or self.distance_slopes is not None or self.distance_far is not None)
         # the options that only the general kernels know, whatever the dtype
         self.extended = bool(self.keep_first or self.learned_sink or self.head_mix or self.value_position is not None)
         if self.extended and self.softcap > 0:
@@ -115,7 +138,10 @@ class PagedAttention(Mixer):
         if self.extended and (self.qk_norm_whole or self.output_gate or not self.own_kv):
             raise ValueError("a norm over all heads, an output gate and borrowed keys are not supported together with kept "
                              "positions, learned sinks, mixed heads or turned values")
-        self.general = (self.extended or self.output_gate or not self.own_kv or self.softcap > 0 or self.values_from_keys or bool(exact_weights) or self.Dv != self.D or self.qk_norm_eps is not None or self.sink_score is not None
+        if self.extended and scored:
+            raise ValueError("chunks and biases by distance are not supported together with kept positions, learned sinks, "
+                             "mixed heads or turned values")
+        self.general = (scored or self.extended or self.output_gate or not self.own_kv or self.softcap > 0 or self.values_from_keys or bool(exact_weights) or self.Dv != self.D or self.qk_norm_eps is not None or self.sink_score is not None
                         or self.position.pairing != "halves" or self.position.amplitude != 1.0)
         if self.general:
             if self.extended:
@@ -153,6 +179,8 @@ class PagedAttention(Mixer):
             s[n["head_mix"]] = TensorSpec((self.Hq, self.Hq), init="identity", kind="vector")
         if self.learned_sink:
             s[n["sink"]] = TensorSpec((self.Hq,), init="zeros", kind="vector")
+        if self.distance_far is not None:       # the number of rows is the file's
+            s[n["rel"]] = TensorSpec((None if available is not None else self.distance_rows, self.Hq), kind="vector")
         s.update(self.position.tensor_specs(available))      # a position encoding may have tensors of its own
         return s
 
@@ -160,6 +188,13 @@ class PagedAttention(Mixer):
         self.ctx = ctx
         n = self.names
         self.position.load(fetch, ctx)
+        self.slopes = self.bias_table = None
+        if self.distance_slopes is not None:
+            self.slopes = torch.tensor(self.distance_slopes, dtype=torch.float32, device=ctx.device)
+        if self.distance_far is not None:       # spread out: one number per head and distance
+            rel = fetch(n["rel"]).float()
+            rows = torch.tensor(distance_buckets(rel.shape[0], self.distance_far), device=rel.device)
+            self.bias_table = rel[rows].t().contiguous()
         # q, k and v rows are stacked so that one product makes all three (src/model.cpp:508-513)
         rows = [fetch(n["q"])]
         if self.own_kv:
@@ -176,7 +211,7 @@ class PagedAttention(Mixer):
         # The tensor-core kernel wants one head size for q, k and v, a multiple of 16: a bfloat16 run of the general
         # path pads the three with zeros up to it (the scores and the sums are the same), and the output
         # projection gets zero columns for the padding.
-        self.pad = 0
+        self.pad, self.direct = 0, False
         self.mix_weight = fetch(n["head_mix"]).float().contiguous() if self.head_mix else None
         self.sinks = fetch(n["sink"]).float().contiguous() if self.learned_sink else None
         if self.value_position is not None:
@@ -184,6 +219,14 @@ class PagedAttention(Mixer):
         if (self.general and not self.extended and ctx.fast_kernels and ctx.act_dtype == torch.bfloat16
                 and self.o_weight.dtype == torch.bfloat16):
             self.pad = (max(self.D, self.Dv) + 15) // 16 * 16
+            self.direct = (self.qkv_weight.dtype == torch.bfloat16 and self.position.rotary_dim == 0 and self.own_kv
+                           and self.qk_norm_eps is None and not self.values_from_keys and not self.output_gate)
+            if self.direct:
+                self.pad = max(self.pad, 32)
+                sizes = [(self.Hq, self.D), (self.Hkv, self.D), (self.Hkv, self.Dv)]
+                self.qkv_weight = _pad_heads(self.qkv_weight, sizes, self.pad)
+                if self.qkv_bias is not None:
+                    self.qkv_bias = _pad_heads(self.qkv_bias, sizes, self.pad)
             if self.pad != self.Dv:
                 w = torch.zeros((self.hidden, self.Hq, self.pad), dtype=self.o_weight.dtype, device=self.o_weight.device)
                 w[:, :, :self.Dv] = self.o_weight.view(self.hidden, self.Hq, self.Dv)
@@ -194,8 +237,8 @@ class PagedAttention(Mixer):
 
     def cache_spec(self):
         if getattr(self, "pad", 0):
-            return KVCacheSpec(self.Hkv, self.pad, self.window)
-        return KVCacheSpec(self.Hkv, self.D, self.window, 0 if self.Dv == self.D else self.Dv, self.keep_first)
+            return KVCacheSpec(self.Hkv, self.pad, self.window, chunk=self.chunk)
+        return KVCacheSpec(self.Hkv, self.D, self.window, 0 if self.Dv == self.D else self.Dv, self.keep_first, chunk=self.chunk)
 
     # ------------------------------------------------------------------ forward
     def forward(self, h, batch, cache):
@@ -217,6 +260,8 @@ class PagedAttention(Mixer):
         and values in their pages, are in the activation dtype; scores, weights and sums are float32."""
         ctx, T = self.ctx, h.shape[0]
         Hq, Hkv, D, Dv = self.Hq, self.Hkv, self.D, self.Dv
+        if self.direct:
+            return self._forward_direct(h, batch, cache)
         proj = linear(ctx, h, self.qkv_weight, torch.float32, bias=self.qkv_bias)
         bt = batch.block_tables[cache.group]
         if self.extended:
@@ -234,29 +279,45 @@ class PagedAttention(Mixer):
         gate = proj[:, self.gate_col:self.gate_col + Hq] if self.output_gate else None
         att = torch.empty((T, Hq * (P or Dv)), dtype=ctx.act_dtype, device=h.device)
         if P:
-            # Entries of one row go to the split-key decode kernel (with weights that keep their float32 bits), the
-            # others to a tensor-core kernel (tcgen05 for head sizes from 64 on, else mma.sync), where
-            # the float32 weights enter the product with the values as three bfloat16 terms; the decode kernel and
-            # the mma.sync kernel add the sink to the softmax's denominator.
-            single = batch.n_single if ops.attention_decode_usable(cache.k, P) else 0
-            if single:
-                ops.attention_decode(q, cache.k, cache.v, bt, batch.row_entry, batch.positions, self.scale, self.window,
-                                     att, Hq, Hkv, P, batch.max_context if batch.decode_only else batch.max_single_context,
-                                     rows=None if batch.decode_only else batch.single_rows, err=ctx.err,
-                                     sink_score=self.sink_score, float_weights=self.weight_terms == 3,
-                                     softcap=self.softcap, gate=gate)
-            if single < batch.S:
-                tiles = (batch.T - single) // ops.attention_prefill_tile_rows() + (batch.S - single)
-                ops.attention_prefill(q, cache.k, cache.v, bt, batch.cu_rows, batch.entry_pos0, tiles, self.scale,
-                                      self.window, att, Hq, Hkv, P, err=ctx.err, min_rows=2 if single else 1,
-                                      kernel="mma" if self.sink_score is not None and self.weight_terms == 3 else "auto",
-                                      sink_score=self.sink_score, weight_terms=self.weight_terms, softcap=self.softcap,
-                                      gate=gate)
+            self._attend_general(q, cache, bt, batch, att, P, gate)
         else:
             ops.paged_attention_general(q, cache.k, cache.v, bt, batch.row_entry, batch.positions, self.scale,
                                         self.window, att, Hq, Hkv, D, Dv, sink_score=self.sink_score,
-                                        softcap=self.softcap, gate=gate)
+                                        softcap=self.softcap, gate=gate, chunk=self.chunk, slopes=self.slopes,
+                                        bias_table=self.bias_table)
         return linear(ctx, att, self.o_weight, torch.float32, bias=self.o_bias)
+
+    def _forward_direct(self, h, batch, cache):
+        """Heads that go from the projection to the scores as they are: one bfloat16 product makes q, k and v with all heads
+        padded to one size, keys and values are copied to their pages, and the attention kernels read q where it is."""
+        ctx, P = self.ctx, self.pad
+        qkv = linear(ctx, h, self.qkv_weight, torch.bfloat16, bias=self.qkv_bias)
+        bt = batch.block_tables[cache.group]
+        ops.rope_store(qkv, batch.positions, self.position.inv_freq(), 0, cache.k, cache.v, bt, batch.row_entry, self.Hq,
+                       self.Hkv, P, cache.write, ctx.err)
+        att = torch.empty((h.shape[0], self.Hq * P), dtype=torch.bfloat16, device=h.device)
+        self._attend_general(qkv, cache, bt, batch, att, P, None)
+        return linear(ctx, att, self.o_weight, torch.float32, bias=self.o_bias)
+
+    def _attend_general(self, q, cache, bt, batch, att, P, gate):
+        """Entries of one row go to the split-key decode kernel (with weights that keep their float32 bits, or as one
+        rounded term), the others to a tensor-core kernel (tcgen05, else mma.sync), where float32 weights enter the product
+        with the values as three bfloat16 terms; the decode kernel and the mma.sync kernel add the sink to the softmax's
+        denominator.  ``q``: rows whose first Hq * P elements are the query heads."""
+        ctx, Hq, Hkv = self.ctx, self.Hq, self.Hkv
+        scored = dict(softcap=self.softcap, gate=gate, chunk=self.chunk, slopes=self.slopes, bias_table=self.bias_table)
+        single = batch.n_single if ops.attention_decode_usable(cache.k, P) else 0
+        if single:
+            ops.attention_decode(q, cache.k, cache.v, bt, batch.row_entry, batch.positions, self.scale, self.window,
+                                 att, Hq, Hkv, P, batch.max_context if batch.decode_only else batch.max_single_context,
+                                 rows=None if batch.decode_only else batch.single_rows, err=ctx.err,
+                                 sink_score=self.sink_score, float_weights=self.weight_terms == 3, **scored)
+        if single < batch.S:
+            tiles = (batch.T - single) // ops.attention_prefill_tile_rows() + (batch.S - single)
+            ops.attention_prefill(q, cache.k, cache.v, bt, batch.cu_rows, batch.entry_pos0, tiles, self.scale,
+                                  self.window, att, Hq, Hkv, P, err=ctx.err, min_rows=2 if single else 1,
+                                  kernel="mma" if self.sink_score is not None and self.weight_terms == 3 else "auto",
+                                  sink_score=self.sink_score, weight_terms=self.weight_terms, **scored)
 
     def _forward_extended(self, proj, bt, batch, cache):
         """Kept first positions, learned sinks, mixed heads, turned values.  The queries stay float32 from the
@@ -336,6 +397,33 @@ class PagedAttention(Mixer):
             tiles = (batch.T - single) // tm + (batch.S - single)
             ops.attention_prefill(qkv, cache.k, cache.v, bt, batch.cu_rows, batch.entry_pos0, tiles, self.scale,
                                   self.window, att, self.Hq, self.Hkv, self.D, err=ctx.err, min_rows=min_rows)
+
+
+def distance_buckets(rows: int, far: int) -> list:
+    """For the distances 0, 1, ... up to the first that all farther ones share a row with: the row of a learned table of
+    ``rows`` rows.  Below ``half = rows // 2`` every distance has its own; distance n beyond has ``half + floor(ln(n / half) /
+    ln(far / half) * (rows - half))``, at most the last one.  Worked out in double."""
+    half = rows // 2
+    out = list(range(half))
+    while not out or out[-1] < rows - 1:
+        n = len(out)
+        if half == 0 or far <= half:            # (no room for a logarithmic part)
+            out.append(rows - 1)
+        else:
+            out.append(min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half))))
+    return out
+
+
+def _pad_heads(w, sizes, P: int):
+    """Rows (or entries) of stacked heads, ``sizes`` = [(heads, elements per head)], with zeros behind every head up to P."""
+    parts, at = [], 0
+    for heads, d in sizes:
+        block = w[at:at + heads * d].view(heads, d, *w.shape[1:])
+        at += heads * d
+        full = torch.zeros((heads, P, *w.shape[1:]), dtype=w.dtype, device=w.device)
+        full[:, :d] = block
+        parts.append(full.view(heads * P, *w.shape[1:]))
+    return torch.cat(parts, dim=0).contiguous()
 
 
 def _cat(ts):

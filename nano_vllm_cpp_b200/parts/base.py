@@ -47,13 +47,15 @@ class KVCacheSpec:
     """Keys and values in pages; ``window`` > 0: only the last ``window`` positions are read, and with
     ``keep_first`` > 0 also the sequence's first so many positions, whose pages are then never given back.
     ``v_head_dim`` > 0: values have that many elements per head instead of ``head_dim``.  ``values`` False: the
-    layer keeps one array per page (what it reads as values is what it reads as keys)."""
+    layer keeps one array per page (what it reads as values is what it reads as keys).  ``chunk`` > 0: a row at position
+    i reads the positions from ``i // chunk * chunk`` on only (and there is no window)."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
     v_head_dim: int = 0
     keep_first: int = 0
     values: bool = True
+    chunk: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -145,14 +147,19 @@ class RowMix:
 
 @dataclass
 class BranchSum:
-    """Two branch outputs that are both still to be added to the residual stream (the sublayers of a layer whose
-    mixer and feed-forward read the same normed rows).  A norm with ``accepts_sum`` adds them in its own kernel;
-    for every other consumer ``resolve_branch`` adds the second into the first."""
+    """Two branch outputs that are both still to be added to the residual stream, each times a constant (the sublayers of
+    a layer whose mixer and feed-forward read the same normed rows, two mixers side by side).  A norm with
+    ``accepts_sum`` adds them in its own kernel; for every other consumer ``resolve_branch`` adds the second into the
+    first."""
     first: torch.Tensor
     second: torch.Tensor
+    scale: float = 1.0          # of the first
+    scale2: float = 1.0         # of the second
 
     def sum(self) -> torch.Tensor:
-        return self.first.add_(self.second)
+        if self.scale != 1.0:
+            self.first.mul_(self.scale)
+        return self.first.add_(self.second, alpha=self.scale2)
 
 
 @dataclass

@@ -107,16 +107,23 @@ class PreNormBlock(Arrangement):
     The sum into the residual stream is fused with the next norm: a block hands its last branch
     output on as ``pending`` instead of adding it, and every norm adds what is pending first —
     the reference's ``rms_norm_add`` convention (src/hip_ops.hip:395-417).  With an ``input_filter`` the mixer reads
-    ``filter(norm1(x))``.
+    ``filter(norm1(x))``.  A layer may have no feed-forward (and then has no ``norm2``).
     """
     slots = {"norm1": "norm", "input_filter": "input_filter", "mixer": "mixer", "norm2": "norm",
              "feed_forward": "feed_forward"}
-    optional = ("input_filter",)
+    optional = ("input_filter", "norm2", "feed_forward")
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        if (self.norm2 is None) != (self.feed_forward is None):
+            raise ValueError("a pre-norm layer's feed-forward comes with its norm")
 
     def forward(self, x, pending, batch, cache):
         h, cache = self.mixer_input(lambda f32, rows: self.norm1.forward(x, resolve_branch(self.norm1, pending), want_f32=f32),
                                     batch, cache)
         pending = self.mixer.forward(h, batch, cache)
+        if self.feed_forward is None:
+            return pending
         h, h32 = self.norm2.forward(x, resolve_branch(self.norm2, pending), want_f32=self.feed_forward.wants_f32_input)
         pending = self.feed_forward.forward(h, h32, batch)
         return pending

@@ -117,7 +117,8 @@ class SparseMoeSwiGLU(FeedForward):
     Other routers are options.  ``score="sigmoid"``: every expert's score is ``s = sigmoid(r)`` by itself, in
     float32; the ``top_k`` largest ``s + correction`` are chosen (``choice_bias``: a learned vector ``correction``
     [experts] that steers the choice only), and the weights are the chosen experts' ``s`` without it.  ``route_scale``
-    multiplies the weights.  ``router_bias`` (softmax scores): a learned vector ``router_bias`` [experts] is added to the
+    multiplies the weights.  ``groups`` = (count, keep): the experts form ``count`` equal groups of neighbours, a group
+    counts as its largest score, and only experts of the ``keep`` best groups can be chosen.  ``router_bias`` (softmax scores): a learned vector ``router_bias`` [experts] is added to the
     logits before the softmax; with ``renormalize`` the weights are then the softmax over the chosen biased logits.
     ``shared_gate=False``: the shared expert has no gate and is added as it is.  ``names``
     gives the tensors' names where they are not the usual ones (keys: router, router_bias, correction, shared_gate, and the
@@ -137,7 +138,8 @@ class SparseMoeSwiGLU(FeedForward):
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, intermediate_size: int,
                  shared_intermediate_size: int = 0, renormalize: bool = False, score: str = "softmax",
                  route_scale: float = 1.0, choice_bias: bool = False, shared_gate: bool = True,
-                 names: dict | None = None, expert_activation: str | None = None, router_bias: bool = False):
+                 names: dict | None = None, expert_activation: str | None = None, router_bias: bool = False,
+                 groups: tuple | None = None):
         if not (1 <= top_k <= num_experts):
             raise ValueError("top_k must lie in 1..num_experts")
         if top_k > 32 or num_experts > 1536:
@@ -151,6 +153,11 @@ class SparseMoeSwiGLU(FeedForward):
         if router_bias and score != "softmax":
             raise ValueError("a bias on the router's logits goes with softmax scores")
         self.router_bias = bool(router_bias)
+        self.groups = (int(groups[0]), int(groups[1])) if groups is not None else None
+        if self.groups is not None:
+            n, keep = self.groups
+            if n < 1 or num_experts % n or not 1 <= keep <= n or top_k > keep * (num_experts // n):
+                raise ValueError("groups: the experts form equal groups, and the kept ones hold at least top_k experts")
         self.score, self.route_scale, self.choice_bias = score, float(route_scale), bool(choice_bias)
         self.shared_gate = bool(shared_gate) and shared_intermediate_size > 0
         if expert_activation is not None and expert_activation not in ops.EPILOGUE_ACTS:
@@ -199,8 +206,8 @@ class SparseMoeSwiGLU(FeedForward):
         bias = fetch(n["correction"]).float().contiguous() if self.choice_bias else None
         if self.router_bias:
             bias = fetch(n["router_bias"]).float().contiguous()
-        if self.score != "softmax" or bias is not None or self.route_scale != 1.0:
-            self.rule = (self.score, bias, self.route_scale)
+        if self.score != "softmax" or bias is not None or self.route_scale != 1.0 or self.groups is not None:
+            self.rule = (self.score, bias, self.route_scale, self.groups)
         stacked = self.gated and fetch.has("experts.gate_up_proj")
         G = 2 if self.gated else 1                       # matrices of an expert's first product
         first = fetch("experts.gate_up_proj") if stacked else fetch(n["expert_gate" if self.gated else "expert_up"].format(0))
@@ -290,7 +297,7 @@ class SparseMoeSwiGLU(FeedForward):
         al = self._alignment(T * KT, self.E + C, dev, fast)
         x_sorted = None
         if (fast and C and T <= SIDE_MAX_ROWS and al.secondary is None
-                and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden)):
+                and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden, self.groups[0] if self.groups else 0)):
             return self._forward_beside(h, logits, gate_logit, idx, score, al)
         if fast and C and T >= 256 and al.secondary is None:
             return self._forward_beside(h, logits, gate_logit, idx, score, al, many=True)
@@ -300,7 +307,7 @@ class SparseMoeSwiGLU(FeedForward):
             if self._counters is None:
                 self._counters = torch.zeros(2, dtype=torch.int32, device=dev)
             zero, c0, c1 = self._counters, self._counters[0:1], self._counters[1:2]
-        if fast and al.secondary is None and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden):
+        if fast and al.secondary is None and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden, self.groups[0] if self.groups else 0):
             x_sorted = ops.moe_route_small(logits, self.K, self.renorm, C, gate_logit, idx, score, al, ctx.err,
                                            x=None, zero=zero, rule=self.rule)   # one block copies rows slower than the copy kernel does
         else:

@@ -25,6 +25,7 @@ from .streams import StreamUpdate, read_streams
 class LayerCall:
     layer: int
     cache_of: Optional[int] = None     # index of an earlier call whose cache entry this call reads
+    pass_index: Optional[int] = None   # the call opens this pass over a stretch of layers (see ModelSpec.pass_input)
 
 
 @dataclass
@@ -46,6 +47,8 @@ class ModelSpec:
     logit_scale: float = 1.0            # logits = head(x) * logit_scale, then, with a cap,
     logit_softcap: float = 0.0          # logits = cap * tanh(logits / cap)
     embed_scale: float = 1.0            # the stream starts as embed[token] * embed_scale
+    pass_input: Optional[PartSpec] = None   # what the stream goes through before a call that opens a pass (parts.passes)
+    pass_input_prefix: str = "loop."
 
     def calls(self):
         if self.order is None:
@@ -83,6 +86,9 @@ class Model:
         self.spec = spec
         self.layers = [build_layer(ls) for ls in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm)
+        self.pass_input = build_part("pass_input", spec.pass_input) if spec.pass_input is not None else None
+        if self.pass_input is not None and spec.streams > 1:
+            raise ValueError("passes over a stretch of layers go with one copy of the residual stream")
         self.calls = spec.calls()
         self.after_call = None      # a hook (call index, stream, pending) for whoever wants to look at the stream layer by layer
         if spec.layer_ids is not None and len(spec.layer_ids) != len(spec.layers):
@@ -90,6 +96,8 @@ class Model:
         for i, c in enumerate(self.calls):
             if not (0 <= c.layer < len(self.layers)):
                 raise ValueError(f"call {i} names layer {c.layer}, which does not exist")
+            if c.pass_index is not None and self.pass_input is None:
+                raise ValueError(f"call {i} opens a pass, but the model has no pass input")
             if c.cache_of is not None and not (0 <= c.cache_of < i and self.calls[c.cache_of].cache_of is None):
                 raise ValueError(f"call {i}: cache_of must name an earlier call that owns its cache entry")
 
@@ -104,6 +112,8 @@ class Model:
             for sub, part in layer.parts():
                 yield lp + sub, part
         yield self.spec.final_norm_prefix, self.final_norm
+        if self.pass_input is not None:
+            yield self.spec.pass_input_prefix, self.pass_input
 
     def tensor_specs(self, has=None) -> dict:
         """Every tensor the model needs, by full name."""
@@ -150,7 +160,10 @@ class Model:
         x = torch.empty((batch.T, s.streams * s.hidden_size), dtype=torch.float32, device=ctx.device)
         ops.embedding(batch.input_ids, self.embed, x, ctx.err, feed=ctx.feed, copies=s.streams, scale=s.embed_scale)
         pending = None
+        recalled = self.pass_input.recall(x) if self.pass_input is not None else None
         for i, c in enumerate(self.calls):
+            if c.pass_index is not None:
+                x, pending = self.pass_input.forward(x, pending, recalled, c.pass_index)
             pending = self.layers[c.layer].forward(x, pending, batch, cache.view(i))
             if self.after_call is not None:
                 self.after_call(i, x, pending)

@@ -13,7 +13,7 @@ class RMSNorm(Norm):
 
     The residual stream and the statistics are float32; ``y`` is written in the activation dtype.
     A branch that is still a ``RowMix`` is summed by the same kernel, and so are the two outputs of a
-    ``BranchSum``.  A ``NormedBranch`` (a sublayer output with a norm of its own, ``n``) is taken in by one launch
+    ``BranchSum`` with their constants.  A ``NormedBranch`` (a sublayer output with a norm of its own, ``n``) is taken in by one launch
     that does both norms: ``x += rms_n(branch) * w_n; y = rms(x) * w``.
     """
     accepts_mix = True
@@ -62,6 +62,7 @@ class RMSNorm(Norm):
         if want_f32:
             out32 = out if out.dtype == torch.float32 else torch.empty_like(x)
         mix = branch2 = None
+        scale = scale2 = 1.0
         if isinstance(branch, NormedBranch):
             inner, first = branch.branch, branch.norm
             if isinstance(inner, RowMix) and inner.index.shape[1] <= ops.ADD_RMSNORM_MAX_MIX:
@@ -77,9 +78,9 @@ class RMSNorm(Norm):
             else:
                 branch = branch.sum()
         elif isinstance(branch, BranchSum):
-            branch, branch2 = branch.first, branch.second
+            branch, branch2, scale, scale2 = branch.first, branch.second, branch.scale, branch.scale2
         ops.add_rmsnorm(x, branch, self.weight, self.eps, out, None if out32 is out else out32, mix=mix,
-                        branch2=branch2)
+                        branch2=branch2, branch_scale=scale, branch2_scale=scale2)
         return out, out32
 
 

@@ -265,10 +265,7 @@ class Retention(Mixer):
         self.w_in = _stack([fetch(n["q"]), fetch(n["k"]), fetch(n["v"]), fetch(n["g"])])     # one float32 product
         self.cols = {"q": 0, "k": H * dk, "v": 2 * H * dk, "g": 2 * H * dk + H * dv}
         self.w_out = fetch(n["o"])
-        # d^0 .. d^64 per head, worked out in float64
-        d = torch.tensor(self.decay, dtype=torch.float64)[:, None]
-        e = torch.arange(ops.retention_chunk_rows() + 1, dtype=torch.float64)[None, :]
-        self.powers = torch.pow(d, e).float().to(ctx.device).contiguous()
+        self.powers = _decay_powers(self.decay, ctx.device)
 
     def cache_spec(self):
         return StateCacheSpec((self.H, self.dk, self.dv))
@@ -283,6 +280,139 @@ class Retention(Mixer):
         return linear(ctx, y, self.w_out, torch.float32)
 
 
+class LightningAttention(Mixer):
+    """Linear attention with one fixed decay per head, activated projections and one norm over the row of all heads.
+
+    ``q, k, v = silu(Wq h), silu(Wk h), silu(Wv h)`` (``heads`` heads of ``dim``, ``dim`` and ``vdim`` elements).  Per head
+    with the constant d = ``decay[h]``:
+
+        S = d S + k v^T;   o = S^T q
+
+    The heads side by side are divided by the root mean square of the whole row (``eps``), multiplied by the weight ``norm``
+    and by ``sigmoid(Wg h)``, and ``Wo`` projects back.  State per request: S, in float32.  ``names`` renames the tensors
+    (keys: q, k, v, g, o, norm)."""
+
+    _NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "norm": "norm"}
+
+    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, decay: list, eps: float, names: dict | None = None):
+        if min(heads, dim, vdim) < 1 or len(decay) != heads:
+            raise ValueError("lightning attention: every size must be positive, and there is one decay per head")
+        if dim > 1400:
+            raise ValueError(f"lightning attention keys of {dim} elements are not supported: the scan kernel takes up to 1400")
+        self.hidden, self.H, self.dk, self.dv, self.eps = hidden_size, heads, dim, vdim, float(eps)
+        self.decay = [float(d) for d in decay]
+        self.names = dict(self._NAMES, **(names or {}))
+
+    def tensor_specs(self, available=None):
+        W, H, dk, dv, n = self.hidden, self.H, self.dk, self.dv, self.names
+        return {n["q"]: TensorSpec((H * dk, W)), n["k"]: TensorSpec((H * dk, W)), n["v"]: TensorSpec((H * dv, W)),
+                n["g"]: TensorSpec((H * dv, W)), n["o"]: TensorSpec((W, H * dv)),
+                n["norm"]: TensorSpec((H * dv,), init="ones", kind="vector")}
+
+    def load(self, fetch, ctx):
+        self.ctx = ctx
+        H, dk, dv, n = self.H, self.dk, self.dv, self.names
+        # one float32 product, silu in its epilogue on the columns of q, k and v
+        self.w_in = _stack([fetch(n["q"]), fetch(n["k"]), fetch(n["v"]), fetch(n["g"])])
+        self.cols = {"q": 0, "k": H * dk, "v": 2 * H * dk}
+        self.gate_col = 2 * H * dk + H * dv
+        self.norm = fetch(n["norm"]).float().contiguous()
+        self.w_out = fetch(n["o"])
+        self.powers = _decay_powers(self.decay, ctx.device)
+
+    def cache_spec(self):
+        return StateCacheSpec((self.H, self.dk, self.dv))
+
+    def forward(self, h, batch, cache):
+        ctx, T = self.ctx, h.shape[0]
+        proj = linear(ctx, h, self.w_in, torch.float32, act=("silu_first", self.gate_col))
+        raw = torch.empty((T, self.H, self.dv), dtype=torch.float32, device=h.device)
+        ops.decayed_memory(proj, self.cols, batch, cache.state, self.H, self.dk, self.dv, raw, powers=self.powers,
+                           fast=ctx.fast_kernels and ctx.act_dtype == torch.bfloat16)
+        y = torch.empty((T, self.H * self.dv), dtype=ctx.act_dtype, device=h.device)
+        ops.gated_norm(raw, proj, self.gate_col, self.norm, self.eps, y, self.H, self.dv)
+        return linear(ctx, y, self.w_out, torch.float32)
+
+
+class StateSpaceDual(Mixer):
+    """The state-space dual form of Mamba-2: ``heads`` heads of ``vdim`` channels over states of ``state`` numbers per
+    channel, with ``groups`` shared pairs of input and output maps (head h uses number ``h // (heads / groups)``).
+
+    ``W_in h = [z | x | b | c | dt]`` (heads * vdim, the same, groups * state, the same, heads).  x, b and c pass a causal
+    convolution over time per channel (``taps`` taps, the last one the current token's, a bias, zeros before the start)
+    and silu; ``dt = softplus(dt + dt_bias)``.  Per head:
+
+        S = exp(-exp(A_log) dt) S + dt b x^T;   y = S^T c + D x
+
+    The heads side by side times ``silu(z)`` are divided by the root mean square (``eps``) of each of ``norm_groups`` equal
+    parts of the row, multiplied by the weight ``norm``, and ``Wo`` projects back.  State per request: S and the last
+    ``taps - 1`` inputs of the convolution, in float32.  ``names`` renames the tensors (keys: in, conv, conv_bias, dt_bias,
+    A_log, D, norm, o)."""
+
+    _NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D",
+              "norm": "norm", "o": "o"}
+
+    def __init__(self, hidden_size: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_groups: int, eps: float,
+                 names: dict | None = None):
+        if min(heads, vdim, state, groups, conv, norm_groups) < 1 or heads % groups or (heads * vdim) % norm_groups:
+            raise ValueError("state-space mixer: positive sizes, heads a multiple of groups, norm_groups equal parts of a row")
+        if state > 1400:
+            raise ValueError(f"states of {state} numbers per channel are not supported: the scan kernel takes up to 1400")
+        self.hidden, self.H, self.dv, self.N, self.G = hidden_size, heads, vdim, state, groups
+        self.taps, self.parts, self.eps = conv, norm_groups, float(eps)
+        self.inner = heads * vdim
+        self.channels = self.inner + 2 * groups * state           # what passes the convolution: x | b | c
+        self.names = dict(self._NAMES, **(names or {}))
+
+    def tensor_specs(self, available=None):
+        W, H, n = self.hidden, self.H, self.names
+        return {n["in"]: TensorSpec((self.inner + self.channels + H, W)),
+                n["conv"]: TensorSpec((self.channels, self.taps), kind="vector"),
+                n["conv_bias"]: TensorSpec((self.channels,), kind="vector"),
+                n["dt_bias"]: TensorSpec((H,), init="zeros", kind="vector"), n["A_log"]: TensorSpec((H,), init="zeros", kind="vector"),
+                n["D"]: TensorSpec((H,), init="ones", kind="vector"),
+                n["norm"]: TensorSpec((self.inner,), init="ones", kind="vector"), n["o"]: TensorSpec((W, self.inner))}
+
+    def load(self, fetch, ctx):
+        self.ctx = ctx
+        n = self.names
+        w = fetch(n["in"])
+        extra = -w.shape[0] % 8                   # rows of the product start on 16-byte boundaries
+        self.w_in = torch.cat([w, w.new_zeros((extra, w.shape[1]))], dim=0).contiguous() if extra else w
+        self.w_conv = fetch(n["conv"]).float().t().contiguous()                   # [taps, channels]
+        self.b_conv = fetch(n["conv_bias"]).float().contiguous()
+        self.dt_bias, self.A_log, self.D = (fetch(n[k]).float().contiguous() for k in ("dt_bias", "A_log", "D"))
+        self.norm = fetch(n["norm"]).float().contiguous()
+        self.w_out = fetch(n["o"])
+        self.cols = {"v": 0, "k": self.inner, "q": self.inner + self.G * self.N}  # of the convolution's result
+
+    def cache_spec(self):
+        parts = [StateCacheSpec((self.H, self.N, self.dv))]
+        if self.taps > 1:
+            parts.append(StateCacheSpec((self.taps - 1, self.channels)))
+        return CompositeCacheSpec(tuple(parts))
+
+    def forward(self, h, batch, cache):
+        ctx, T, dev = self.ctx, h.shape[0], h.device
+        proj = linear(ctx, h, self.w_in, torch.float32)           # z | x b c | dt
+        xbc = torch.empty((T, self.channels), dtype=torch.float32, device=dev)
+        ops.causal_conv_silu(proj, self.inner, self.w_conv, self.b_conv, batch, cache.parts[1].state if self.taps > 1 else None, xbc)
+        raw = torch.empty((T, self.H, self.dv), dtype=torch.float32, device=dev)
+        ops.decayed_memory(xbc, self.cols, batch, cache.parts[0].state, self.H, self.N, self.dv, raw, q_heads=self.G,
+                           steps=(proj, self.inner + self.channels, self.A_log, self.dt_bias),
+                           fast=ctx.fast_kernels and ctx.act_dtype == torch.bfloat16)
+        y = torch.empty((T, self.inner), dtype=ctx.act_dtype, device=dev)
+        ops.gated_norm(raw, proj, 0, self.norm, self.eps, y, self.H, self.dv, parts=self.parts, gate_first=True, skip=self.D, x=xbc)
+        return linear(ctx, y, self.w_out, torch.float32)
+
+
+def _decay_powers(decay: list, device):
+    """d^0 .. d^64 per head, worked out in float64."""
+    d = torch.tensor(decay, dtype=torch.float64)[:, None]
+    e = torch.arange(ops.retention_chunk_rows() + 1, dtype=torch.float64)[None, :]
+    return torch.pow(d, e).float().to(device).contiguous()
+
+
 def ops_scan_size_ok(dk: int, dv: int, parts: int = 1) -> bool:
     """What ``ops.scan_usable`` checks, without the library: a head's matrix and its helpers fit in 227 KB of
     shared memory and a value is at most 256 wide."""
@@ -295,3 +425,5 @@ def ops_scan_size_ok(dk: int, dv: int, parts: int = 1) -> bool:
 register_part("mixer", "matrix_lstm", MatrixLSTM)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
 register_part("mixer", "retention", Retention)
+register_part("mixer", "lightning_attention", LightningAttention)
+register_part("mixer", "state_space_dual", StateSpaceDual)

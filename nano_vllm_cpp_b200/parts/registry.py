@@ -11,14 +11,15 @@ ARRANGEMENTS: dict = {}
 TOKEN_INPUTS: dict = {}
 CONNECTIONS: dict = {}
 INPUT_FILTERS: dict = {}
+PASS_INPUTS: dict = {}
 
 _TABLES = {"norm": NORMS, "position": POSITION_ENCODINGS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS,
            "arrangement": ARRANGEMENTS, "token_input": TOKEN_INPUTS, "connection": CONNECTIONS,
-           "input_filter": INPUT_FILTERS}
+           "input_filter": INPUT_FILTERS, "pass_input": PASS_INPUTS}
 
 
 def register_part(family: str, kind: str, cls) -> None:
-    """``family``: norm, position, mixer, feed_forward, token_input, connection, input_filter or arrangement."""
+    """``family``: norm, position, mixer, feed_forward, token_input, connection, input_filter, pass_input or arrangement."""
     _TABLES[family][kind] = cls
 
 

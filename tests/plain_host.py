@@ -125,11 +125,14 @@ class CacheManager:
     def __init__(self, windows: list, num_pages, page_size: int, max_requests: int,
                  prefix_caching: bool = False, has_state: bool = False):
         """``windows``: one entry per group (0 = reads every key; ``(window, keep_first)``: the first ``keep_first``
-        positions stay readable behind the window; none for a model without paged layers).
+        positions stay readable behind the window; ``("chunk", n)``: a row reads its own chunk of n positions; none for a
+        model without paged layers).
         ``num_pages``: an int for all groups or a list.  ``has_state``: some layer keeps a per-request state, which
         rules prefix sharing out."""
         if isinstance(num_pages, int):
             num_pages = [num_pages] * len(windows)
+        self.chunks = [int(w[1]) if isinstance(w, (tuple, list)) and w[0] == "chunk" else 0 for w in windows]
+        windows = [0 if c else w for w, c in zip(windows, self.chunks)]
         self.keeps = [int(w[1]) if isinstance(w, (tuple, list)) else 0 for w in windows]
         self.windows = [int(w[0]) if isinstance(w, (tuple, list)) else int(w) for w in windows]
         self.page_size = page_size
@@ -137,7 +140,8 @@ class CacheManager:
         self.max_requests = max_requests
         self._free_slots = list(range(max_requests - 1, -1, -1))
         self.requests: dict = {}
-        self.prefix_caching = (bool(prefix_caching) and not has_state and len(windows) == 1 and self.windows[0] == 0)
+        self.prefix_caching = (bool(prefix_caching) and not has_state and len(windows) == 1 and self.windows[0] == 0
+                               and self.chunks[0] == 0)
 
     # ------------------------------------------------------------------ requests
     def has(self, rid) -> bool:
@@ -170,6 +174,8 @@ class CacheManager:
     def _first_needed_page(self, g: int, start: int) -> int:
         """Lowest page that rows from position ``start`` on still read in group g."""
         w = self.windows[g]
+        if self.chunks[g] > 0:
+            return start // self.chunks[g] * self.chunks[g] // self.page_size
         if w <= 0:
             return 0
         return max(0, start + 1 - w) // self.page_size

@@ -49,7 +49,8 @@ def _call(lib, name, qkv, kc, vc, bt, ent, pos, out, Hq, Hkv, D, page, splits, s
         args += [c_void_p(0), c_int(0)]     # ... and counters for adding the splits up in the kernel itself; none
         args += [c_int(0), c_float(0.0), c_int(0)]      # ... no sink in the softmax, weights as the kernel likes them
         args.append(c_float(0.0))                       # ... scores that are not capped
-        args += [c_void_p(0), ctypes.c_longlong(0)]     # ... and no gates on the heads' outputs
+        args += [c_void_p(0), ctypes.c_longlong(0)]     # ... no gates on the heads' outputs
+        args += [c_int(0), c_void_p(0), c_void_p(0), c_int(0)]      # ... no chunks, and no bias by distance
     args.append(stream)
     return fn(*args)
 
