@@ -343,13 +343,41 @@ def sevelorn_config(z):
             "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": layers}
 
 
+# --design dubarax: the same measurement for the Dubarax decoder beside the two existing models that have its parts, at equal
+# size: a Qwen2-MoE decoder (window attention and a mixture with a shared expert) and the Sevelorn decoder (matrix memories
+# with a fixed decay beside attention around a mixture; one copy of the stream here), with the same width, depth, heads, head
+# size, experts, expert width and vocabulary.  ``layers`` counts layer runs: the first third of Dubarax's layers runs twice.
+# Its layers go parallel (chunked attention beside lightning attention with half as many heads), window attention, state-space
+# (twice the width in channels, heads of 64, states of 128).
+DUBARAX_SIZES = {k: dict(z, streams=1) for k, z in KIFUNEX_SIZES.items()}
+
+
+def dubarax_config(z):
+    W, H, G, D = z["width"], z["heads"], z["kv_heads"], z["dim"]
+    heads = {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": z["window"]}}
+    half = max(1, H // 2)
+    both = {"left": heads, "left_scale": 0.7, "right_scale": 0.7,
+            "right": {"heads": half, "dim": D, "vdim": D, "decay": [1.0 - 2.0 ** (-5 - 7 * h / max(1, half - 1)) for h in range(half)]}}
+    window = dict(heads, softcap=30.0, bias_max=512)
+    memory = {"heads": 2 * W // 64, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}
+    mlp = {"kind": "moe", "expert": {"ff": z["ff"]}, "shared": {"ff": z["shared_ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 4, "keep": 2}}}
+    n = z["layers"] * 3 // 4
+    kinds = [("parallel", both), ("attention", window), ("mamba2", memory)]
+    return {"architecture": "Dubarax", "vocab": z["vocab"], "width": W, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "loop": {"start": 0, "stop": n // 3, "times": 2},
+            "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(n)]}
+
+
 # sizes, the design, and the existing models it is measured beside
 DESIGNS = {"bizodra": (DESIGN_SIZES, [("bizodra", bizodra_config), ("qwen2_dense", dense_qwen_config)]),
            "kifunex": (KIFUNEX_SIZES, [("kifunex", kifunex_config), ("qwen2_moe", sparse_qwen_config)]),
            "sanesun": (DESIGN_SIZES, [("sanesun", sanesun_config), ("bizodra", bizodra_config)]),
            "gekitar": (KIFUNEX_SIZES, [("gekitar", gekitar_config), ("qwen2_moe", sparse_qwen_config)]),
            "sevelorn": (SEVELORN_SIZES, [("sevelorn", sevelorn_config), ("kifunex", kifunex_config),
-                                         ("bizodra", lambda z: bizodra_config(dict(z, ff=z["top"] * z["ff"])))])}
+                                         ("bizodra", lambda z: bizodra_config(dict(z, ff=z["top"] * z["ff"])))]),
+           "dubarax": (DUBARAX_SIZES, [("dubarax", dubarax_config), ("qwen2_moe", sparse_qwen_config),
+                                       ("sevelorn", sevelorn_config)])}
 
 
 def design_bench(args) -> int:
@@ -419,7 +447,7 @@ def design_bench(args) -> int:
             with ops.KernelTimes() as kt:
                 prefill_many()
             row["prefill_together"]["kernels"] = [{"name": r["name"], "calls": r["calls"], "ms": round(r["ms"], 3)}
-                                                  for r in kt.summary()[:12]]
+                                                  for r in kt.summary()[:20]]
             runner.cuda_graphs = graphs
             # the prompt's kernels one by one (outside graphs, an event between any two)
             graphs, runner.cuda_graphs = runner.cuda_graphs, False
@@ -428,7 +456,7 @@ def design_bench(args) -> int:
             runner.close("kt")
             row["prefill_kernels"] = [{"name": r["name"], "calls": r["calls"], "ms": round(r["ms"], 3),
                                        **({"frac_bf16": round(r["flops"] / (r["ms"] * 1e-3) / (P["bf16_tflops"] * 1e12), 3)} if r["flops"] else {})}
-                                      for r in kt.summary()[:12]]
+                                      for r in kt.summary()[:20]]
             runner.cuda_graphs = graphs
             for B in batches:
                 rids = [f"d{B}_{i}" for i in range(B)]
@@ -461,7 +489,7 @@ def design_bench(args) -> int:
                             ops.delay(20000)
                             runner.step(entries, check=False)
                     row["decode_kernels"] = [{"name": r["name"], "calls": r["calls"] // 4, "ms": round(r["ms"] / 4, 4)}
-                                             for r in kt.summary()[:12]]
+                                             for r in kt.summary()[:20]]
                     runner.cuda_graphs = graphs
                 for rid in rids:
                     runner.close(rid)

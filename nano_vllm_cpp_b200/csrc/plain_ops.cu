@@ -747,7 +747,7 @@ NV_API int nv_gather_rows(const void* src, int dt, const int* rows, void* dst, i
 
 // Zeroes the per-request state of every entry that starts its request (first position 0): a request's state must
 // not begin with what the slot's previous holder, or the request itself before a preemption, left there.
-// state: [slots][slot_bytes] bytes, slot_bytes a multiple of 4.  One block per entry.
+// state: [slots][slot_bytes] bytes, slot_bytes a multiple of 4.  Blocks along y share out an entry's state.
 __global__ void reset_fresh_state_kernel(uint32_t* __restrict__ state, long long slot_words,
                                          const int* __restrict__ entry_slot, const int* __restrict__ entry_pos0,
                                          int num_slots) {
@@ -756,14 +756,21 @@ __global__ void reset_fresh_state_kernel(uint32_t* __restrict__ state, long long
   const int slot = entry_slot[e];
   if (slot < 0 || slot >= num_slots) return;
   uint32_t* p = state + (size_t)slot * slot_words;
-  for (long long i = threadIdx.x; i < slot_words; i += blockDim.x) p[i] = 0u;
+  const long long at = (long long)blockIdx.y * blockDim.x + threadIdx.x, step = (long long)gridDim.y * blockDim.x;
+  if (slot_words % 4 == 0 && ((uintptr_t)state & 15) == 0) {
+    for (long long i = at; i < slot_words / 4; i += step) ((uint4*)p)[i] = make_uint4(0, 0, 0, 0);
+  } else {
+    for (long long i = at; i < slot_words; i += step) p[i] = 0u;
+  }
 }
 
 NV_API int nv_reset_fresh_state(void* state, long long slot_bytes, int num_slots, const int* entry_slot,
                                 const int* entry_pos0, int S, cudaStream_t s) {
   if (slot_bytes % 4 || ((uintptr_t)state & 3)) return NV_ERR_BAD_SIZE;
   if (S == 0 || slot_bytes == 0) return NV_OK;
-  reset_fresh_state_kernel<<<S, 256, 0, s>>>((uint32_t*)state, slot_bytes / 4, entry_slot, entry_pos0, num_slots);
+  const long long words = slot_bytes / 4;
+  const unsigned share = (unsigned)(words < 16384 ? 1 : words / 16384 < 64 ? words / 16384 : 64);
+  reset_fresh_state_kernel<<<dim3((unsigned)S, share), 256, 0, s>>>((uint32_t*)state, slot_bytes / 4, entry_slot, entry_pos0, num_slots);
   NV_RETURN_LAST();
 }
 

@@ -191,6 +191,7 @@ struct RetArgs {
   float* raw;               // scan: [T, H, dv]
   uint32_t* chunks;         // chunked form: per chunk and head dk * dv words (float32 sums, then the states' two terms)
   int G;                    // heads of q and k: head h reads q/k head h / (H / G)
+  int hb;                   // chunked form: heads of a block, all with the same q and k
   int raw_out;              // the outputs go to `raw` [T, H, dv] in float32, without norm and gate
   // Row decays (dsrc != nullptr): step size dt = softplus(dsrc[t, d0 + h] + dt_bias[h]), decay exp(-exp(A_log[h]) dt), and
   // the row's k times dt instead of k_scale.
@@ -392,6 +393,7 @@ __global__ void __launch_bounds__(256) retention_finish_kernel(RetArgs a, int T)
 // ------------------------------------------------------------------ the chunked form
 constexpr int CK_THREADS = 256, CK_WARPS = CK_THREADS / 32;
 constexpr int VLD = 64 + 8;            // row of a 64-column slab in shared memory (sixteen bytes of padding)
+constexpr int CK_HEADS = 4;            // most heads that a block takes one after the other (they share q and k)
 
 __device__ __forceinline__ uint32_t s_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
@@ -461,13 +463,14 @@ __device__ __forceinline__ void find_chunk(const int* cu_rows, int S, int min_ro
   if (lane == 0) info[0] = -1;
 }
 
-// Row decays of a chunk, worked out by warp 0: dt[i] the rows' step sizes, cl[i] the base-2 logarithm of the product of the
-// decays of rows 0 .. i.  Rows beyond n neither decay nor count.
-__device__ __forceinline__ void chunk_row_decays(const RetArgs& a, int h, int row0, int n, float* cl, float* dt) {
+// Row decays of a chunk, worked out by a warp: lane l has rows i = 2 l and i + 1, d[] their step sizes, c[] the base-2 logarithm
+// of the product of the decays of rows 0 .. i (and i + 1).  Rows beyond n neither decay nor count.
+__device__ __forceinline__ void chunk_row_decays(const RetArgs& a, int h, int row0, int n, float (&c)[2], float (&d)[2]) {
   const int lane = threadIdx.x & 31, i = 2 * lane;
   const float rate2 = expf(a.A_log[h]) * 1.4426950408889634f;
-  const float d0 = i < n ? step_size_of(a, row0 + i, h) : 0.f, d1 = i + 1 < n ? step_size_of(a, row0 + i + 1, h) : 0.f;
-  const float l0 = -rate2 * d0, l1 = -rate2 * d1;
+  d[0] = i < n ? step_size_of(a, row0 + i, h) : 0.f;
+  d[1] = i + 1 < n ? step_size_of(a, row0 + i + 1, h) : 0.f;
+  const float l0 = -rate2 * d[0], l1 = -rate2 * d[1];
   float inc = l0 + l1;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -475,17 +478,14 @@ __device__ __forceinline__ void chunk_row_decays(const RetArgs& a, int h, int ro
     if (lane >= o) inc += up;
   }
   const float before = __shfl_up_sync(0xffffffffu, inc, 1);
-  const float first = (lane ? before : 0.f) + l0;
-  dt[i] = d0;
-  dt[i + 1] = d1;
-  cl[i] = first;
-  cl[i + 1] = first + l1;
+  c[0] = (lane ? before : 0.f) + l0;
+  c[1] = c[0] + l1;
 }
 
-// Rows row0 .. row0 + n - 1 of one q or k head, turned, times factor(row), as two bfloat16 terms in shared memory
+// Rows row0 .. row0 + n - 1 of one q or k head, turned, as two bfloat16 terms in shared memory
 // [RC][LDS]; rows beyond n and elements beyond dk are zero.
-template <int DKP, typename F>
-__device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, int row0, int n, F factor, bf16* hi, bf16* lo) {
+template <int DKP>
+__device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, int row0, int n, bf16* hi, bf16* lo) {
   constexpr int LDS = DKP + 8;
   const int half = a.half, dk = a.dk, tid = threadIdx.x;
   if (a.v2) {
@@ -516,13 +516,12 @@ __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, 
 #pragma unroll
         for (int b = 0; b < B; ++b) {
           const int r = r0 + CK_WARPS * b;
-          const float f = r < n ? factor(r) : 0.f;
           uint32_t wh, wl;
-          split2((u[b].x * cs[b].x - w[b].x * cs[b].y) * f, (u[b].y * cs[b].z - w[b].y * cs[b].w) * f, wh, wl);
+          split2(u[b].x * cs[b].x - w[b].x * cs[b].y, u[b].y * cs[b].z - w[b].y * cs[b].w, wh, wl);
           *reinterpret_cast<uint32_t*>(hi + r * LDS + d) = wh;
           *reinterpret_cast<uint32_t*>(lo + r * LDS + d) = wl;
           if (turned) {
-            split2((w[b].x * cs[b].x + u[b].x * cs[b].y) * f, (w[b].y * cs[b].z + u[b].y * cs[b].w) * f, wh, wl);
+            split2(w[b].x * cs[b].x + u[b].x * cs[b].y, w[b].y * cs[b].z + u[b].y * cs[b].w, wh, wl);
             *reinterpret_cast<uint32_t*>(hi + r * LDS + d + half) = wh;
             *reinterpret_cast<uint32_t*>(lo + r * LDS + d + half) = wl;
           }
@@ -534,15 +533,14 @@ __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, 
     for (int x = tid; x < RC * items; x += CK_THREADS) {
       const int r = x / items, i = x - r * items;
       const bool live = r < n;
-      const float f = live ? factor(r) : 0.f;
       const float* p = src + (size_t)(row0 + (live ? r : 0)) * a.ld;
       if (i < half) {
         const float2 cs = a.table[(size_t)(row0 + (live ? r : 0)) * half + i];
         const float u = p[i], w = p[i + half];
-        split1(live ? (u * cs.x - w * cs.y) * f : 0.f, hi + r * LDS + i, lo + r * LDS + i);
-        split1(live ? (w * cs.x + u * cs.y) * f : 0.f, hi + r * LDS + i + half, lo + r * LDS + i + half);
+        split1(live ? u * cs.x - w * cs.y : 0.f, hi + r * LDS + i, lo + r * LDS + i);
+        split1(live ? w * cs.x + u * cs.y : 0.f, hi + r * LDS + i + half, lo + r * LDS + i + half);
       } else {
-        split1(live ? p[i + half] * f : 0.f, hi + r * LDS + i + half, lo + r * LDS + i + half);
+        split1(live ? p[i + half] : 0.f, hi + r * LDS + i + half, lo + r * LDS + i + half);
       }
     }
   }
@@ -553,40 +551,46 @@ __device__ __forceinline__ void load_turned(const RetArgs& a, const float* src, 
   }
 }
 
-// Columns c0 .. c0 + 63 of the value head of the chunk's rows, as two terms [RC][VLD]; what does not exist is zero.
-__device__ __forceinline__ void load_values(const RetArgs& a, const float* src, int row0, int n, int c0, bf16* hi, bf16* lo) {
+// Columns c0 .. c0 + 63 of a value head of the chunk's rows, every row times weight[row] (nullptr: as it is), as two terms
+// [RC][VLD]; what does not exist is zero.  Where pairs can be read (v2) a thread fetches its values into registers first,
+// which may happen while the block still works on the slab before.
+constexpr int VREGS = RC / CK_WARPS;
+struct ValueRegs { float2 v[VREGS]; };
+__device__ __forceinline__ void fetch_values(const RetArgs& a, const float* src, int row0, int n, int c0, ValueRegs& x) {
+  if (!a.v2) return;
+  const int c = 2 * (threadIdx.x & 31);
+  const bool col = c0 + c < a.dv;
+#pragma unroll
+  for (int b = 0; b < VREGS; ++b) {
+    const int r = (threadIdx.x >> 5) + CK_WARPS * b;
+    x.v[b] = make_float2(0.f, 0.f);
+    if (r < n && col) x.v[b] = *reinterpret_cast<const float2*>(src + (size_t)(row0 + r) * a.ld + c0 + c);
+  }
+}
+__device__ __forceinline__ void store_values(const RetArgs& a, const float* src, int row0, int n, int c0, const ValueRegs& x,
+                                             const float* weight, bf16* hi, bf16* lo) {
   if (a.v2) {
-    constexpr int B = 8;
     const int c = 2 * (threadIdx.x & 31);
-    const bool col = c0 + c < a.dv;
 #pragma unroll
-    for (int r0 = threadIdx.x >> 5; r0 < RC; r0 += CK_WARPS * B) {
-      float2 v[B];
-#pragma unroll
-      for (int b = 0; b < B; ++b) {
-        const int r = r0 + CK_WARPS * b;
-        v[b] = make_float2(0.f, 0.f);
-        if (r < n && col) v[b] = *reinterpret_cast<const float2*>(src + (size_t)(row0 + r) * a.ld + c0 + c);
-      }
-#pragma unroll
-      for (int b = 0; b < B; ++b) {
-        const int r = r0 + CK_WARPS * b;
-        uint32_t wh, wl;
-        split2(v[b].x, v[b].y, wh, wl);
-        *reinterpret_cast<uint32_t*>(hi + r * VLD + c) = wh;
-        *reinterpret_cast<uint32_t*>(lo + r * VLD + c) = wl;
-      }
+    for (int b = 0; b < VREGS; ++b) {
+      const int r = (threadIdx.x >> 5) + CK_WARPS * b;
+      const float f = weight ? weight[r] : 1.f;
+      uint32_t wh, wl;
+      split2(x.v[b].x * f, x.v[b].y * f, wh, wl);
+      *reinterpret_cast<uint32_t*>(hi + r * VLD + c) = wh;
+      *reinterpret_cast<uint32_t*>(lo + r * VLD + c) = wl;
     }
   } else {
-    for (int x = threadIdx.x; x < RC * 64; x += CK_THREADS) {
-      const int r = x / 64, c = x % 64;
+    for (int x2 = threadIdx.x; x2 < RC * 64; x2 += CK_THREADS) {
+      const int r = x2 / 64, c = x2 % 64;
       const float v = r < n && c0 + c < a.dv ? src[(size_t)(row0 + r) * a.ld + c0 + c] : 0.f;
-      split1(v, hi + r * VLD + c, lo + r * VLD + c);
+      split1(weight ? v * weight[r] : v, hi + r * VLD + c, lo + r * VLD + c);
     }
   }
 }
 
-// Every chunk's own sum: U = sum_j d^(n-1-j) k_j v_j^T, float32 [dk][dv].  grid (chunks, heads).
+// Every chunk's own sum: U = sum_j d^(n-1-j) k_j v_j^T, float32 [dk][dv].  grid (chunks, heads / hb): a block takes hb heads
+// with the same k, whose terms are made once; what a row counts for multiplies its value.
 template <int DKP, bool VAR>
 __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 ? 3 : 1) retention_chunk_sum_kernel(RetArgs a) {
   constexpr int LDS = DKP + 8;
@@ -596,31 +600,44 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 ? 3 : 1) retention_chun
   bf16* vh = kl + RC * LDS;
   bf16* vl = vh + RC * VLD;
   __shared__ int info[3];
-  __shared__ float pw[RC + 1], dts[VAR ? RC : 1];      // powers of the decay; with row decays their running logarithms
-  const int h = blockIdx.y, gh = h / (a.H / a.G), tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+  __shared__ float counts[CK_HEADS][RC];
+  const int h0 = blockIdx.y * a.hb, gh = h0 / (a.H / a.G), tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
   grid_dep_wait();
   grid_dep_launch();
-  if (warp == 0) {
-    find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
-    __syncwarp();
-    if (VAR && info[0] >= 0) chunk_row_decays(a, h, info[1], info[2], pw, dts);
-  }
-  if (!VAR)
-    for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
+  if (warp == 0) find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
   __syncthreads();
   if (info[0] < 0) return;
   const int row0 = info[1], n = info[2];
-  const float ks = a.k_scale;
-  if (VAR && tid == 0) a.chunk_decay[(size_t)blockIdx.x * a.H + h] = exp2f(pw[n - 1]);
-  load_turned<DKP>(a, a.proj + a.k0 + (size_t)gh * a.dk, row0, n,
-                   [&](int r) { return VAR ? exp2f(pw[n - 1] - pw[r]) * dts[VAR ? r : 0] : pw[n - 1 - r] * ks; }, kh, kl);
-  float* U = reinterpret_cast<float*>(a.chunks) + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
+  ValueRegs next;
+  fetch_values(a, a.proj + a.v0 + (size_t)h0 * a.dv, row0, n, 0, next);
+  if (VAR) {
+    if (warp < a.hb) {
+      float c[2], d[2];
+      chunk_row_decays(a, h0 + warp, row0, n, c, d);
+      const float total = __shfl_sync(0xffffffffu, c[1], 31);        // (rows beyond n add nothing)
+      counts[warp][2 * lane] = exp2f(total - c[0]) * d[0];
+      counts[warp][2 * lane + 1] = exp2f(total - c[1]) * d[1];
+      if (lane == 0) a.chunk_decay[(size_t)blockIdx.x * a.H + h0 + warp] = exp2f(total);
+    }
+  } else {
+    for (int i = tid; i < a.hb * RC; i += CK_THREADS) {
+      const int r = i % RC;
+      counts[i / RC][r] = r < n ? a.powers[(size_t)(h0 + i / RC) * (RC + 1) + n - 1 - r] * a.k_scale : 0.f;
+    }
+  }
+  load_turned<DKP>(a, a.proj + a.k0 + (size_t)gh * a.dk, row0, n, kh, kl);
+  __syncthreads();
   const int g = lane / 4, tq = lane % 4;
   const bool even = (a.dv & 1) == 0;
-  for (int c0 = 0; c0 < a.dv; c0 += 64) {
-    if (c0) __syncthreads();
-    load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
+  const int slabs = (a.dv + 63) / 64;
+  for (int step = 0; step < a.hb * slabs; ++step) {
+    const int hh = step / slabs, c0 = (step % slabs) * 64;
+    float* U = reinterpret_cast<float*>(a.chunks) + ((size_t)blockIdx.x * a.H + h0 + hh) * a.dk * a.dv;
+    if (step) __syncthreads();
+    store_values(a, a.proj + a.v0 + (size_t)(h0 + hh) * a.dv, row0, n, c0, next, counts[hh], vh, vl);
     __syncthreads();
+    if (step + 1 < a.hb * slabs)
+      fetch_values(a, a.proj + a.v0 + (size_t)(h0 + (step + 1) / slabs) * a.dv, row0, n, ((step + 1) % slabs) * 64, next);
     // an item of work is sixteen rows and 32 columns of U
     for (int item = warp; item < DKP / 8; item += CK_WARPS) {
       const int d0 = (item >> 1) * 16, n0 = (item & 1) * 32;
@@ -681,18 +698,20 @@ __device__ __forceinline__ void count_chunks_before(const int* cu_rows, int e, i
 
 // Turns an entry's chunk sums into the states its chunks start from, in place, and leaves the last state in the request's
 // slot.  Here every row of a state becomes the row's leading terms [dv bfloat16] and behind them its rest terms
-// [dv bfloat16], which the next kernel copies as they are.  A warp owns a row (its lanes four columns each, NJ times):
-// all of a row's sums are read before its terms are written over them.  grid (entries, heads, dk / 8).
-template <int NJ>
+// [dv bfloat16], which the next kernel copies as they are.  A row is LPR lanes' (four columns each, NJ times): 32, or 16
+// where a row has no more than 64 columns; all of a row's sums are read before its terms are written over them.  grid
+// (entries, heads, rows / (256 / LPR)).
+template <int NJ, int LPR>
 __global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs a) {
   __shared__ int first_s;
-  const int e = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
+  const int e = blockIdx.x, h = blockIdx.y, lane = threadIdx.x % LPR;
   grid_dep_wait();
   grid_dep_launch();
   const int n = a.cu_rows[e + 1] - a.cu_rows[e];
   if (n < a.min_rows) return;
   count_chunks_before(a.cu_rows, e, a.min_rows, &first_s);
-  const int d = blockIdx.z * 8 + (threadIdx.x >> 5);
+  const int d = blockIdx.z * (256 / LPR) + threadIdx.x / LPR;
+  const unsigned lanes = __ballot_sync(0xffffffffu, d < a.dk);
   if (d >= a.dk) return;
   const int count = (n + RC - 1) / RC, dv = a.dv;
   const size_t size = (size_t)a.dk * dv, step = (size_t)a.H * size;
@@ -705,7 +724,7 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs 
   Vals<4> S[NJ];
 #pragma unroll
   for (int j = 0; j < NJ; ++j)
-    if (4 * (lane + 32 * j) < dv) S[j] = ldv<4>(Sg + 4 * (lane + 32 * j));
+    if (4 * (lane + LPR * j) < dv) S[j] = ldv<4>(Sg + 4 * (lane + LPR * j));
   constexpr int U = 8 / NJ;            // chunk sums in flight
   for (int c0 = 0; c0 < count; c0 += U) {
     Vals<4> u[U][NJ];
@@ -713,16 +732,16 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs 
     for (int i = 0; i < U; ++i)
 #pragma unroll
       for (int j = 0; j < NJ; ++j)
-        if (c0 + i < count && 4 * (lane + 32 * j) < dv)
-          u[i][j] = ldv<4>(reinterpret_cast<const float*>(p) + (size_t)(c0 + i) * step + 4 * (lane + 32 * j));
-    __syncwarp();                      // the row's sums have been read by all lanes
+        if (c0 + i < count && 4 * (lane + LPR * j) < dv)
+          u[i][j] = ldv<4>(reinterpret_cast<const float*>(p) + (size_t)(c0 + i) * step + 4 * (lane + LPR * j));
+    __syncwarp(lanes);                 // the row's sums have been read by all lanes
 #pragma unroll
     for (int i = 0; i < U; ++i)
       if (c0 + i < count) {
         const float f = var ? dec[(size_t)(c0 + i) * a.H] : (c0 + i + 1 < count ? full : last);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
-          const int c = 4 * (lane + 32 * j);
+          const int c = 4 * (lane + LPR * j);
           if (c >= dv) continue;
           uint2 hi, lo;
           split2(S[j].v[0], S[j].v[1], hi.x, lo.x);
@@ -737,7 +756,7 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_rows_kernel(RetArgs 
   }
 #pragma unroll
   for (int j = 0; j < NJ; ++j)
-    if (4 * (lane + 32 * j) < dv) stv<4>(Sg + 4 * (lane + 32 * j), S[j]);
+    if (4 * (lane + LPR * j) < dv) stv<4>(Sg + 4 * (lane + LPR * j), S[j]);
 }
 
 // The same for other sizes: an element's two terms are packed in one word (the same thread reads and writes an element).
@@ -780,9 +799,10 @@ __global__ void __launch_bounds__(256) retention_chunk_pass_kernel(RetArgs a) {
 
 __device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
-// Every chunk's outputs, its heads normed and gated.  grid (chunks, heads).  Two warps share sixteen rows: each takes half
-// of the keys for the weights, which both then read from shared memory, and half of every slab's columns.  NS: slabs of
-// 64 value columns.
+// Every chunk's outputs, its heads normed and gated (or as they are, raw_out).  grid (chunks, heads / hb): a block takes hb
+// heads with the same q and k one after the other; their products q . k are made once.  Two warps share sixteen rows: each
+// takes half of the keys for the weights, which both then read from shared memory, and half of every slab's columns.  NS:
+// slabs of 64 value columns.
 template <int DKP, int NS, bool VAR>
 __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) retention_chunk_out_kernel(RetArgs a) {
   constexpr int LDS = DKP + 8;
@@ -798,23 +818,31 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
   bf16* pl = ph + RC * VLD;
   __shared__ float squares[2][RC];
   __shared__ int info[3];
-  __shared__ float pw[RC + 1], dts[VAR ? RC : 1];      // powers of the decay; with row decays their running logarithms
-  const int h = blockIdx.y, gh = h / (a.H / a.G), tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+  // per head: the powers of the decay; with row decays their running logarithms, and the rows' step sizes
+  __shared__ float pws[CK_HEADS][RC + 1], dts[VAR ? CK_HEADS : 1][RC];
+  const int h0 = blockIdx.y * a.hb, gh = h0 / (a.H / a.G), tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
   grid_dep_wait();
   grid_dep_launch();
-  if (warp == 0) {
-    find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
-    __syncwarp();
-    if (VAR && info[0] >= 0) chunk_row_decays(a, h, info[1], info[2], pw, dts);
-  }
-  if (!VAR)
-    for (int i = tid; i <= RC; i += CK_THREADS) pw[i] = a.powers[(size_t)h * (RC + 1) + i];
+  if (warp == 0) find_chunk(a.cu_rows, a.num_entries, a.min_rows, blockIdx.x, info);
   __syncthreads();
   if (info[0] < 0) return;
   const int row0 = info[1], n = info[2];
-  const float ks = a.k_scale;
-  load_turned<DKP>(a, a.proj + a.q0 + (size_t)gh * a.dk, row0, n, [](int) { return 1.f; }, qh, ql);
-  load_turned<DKP>(a, a.proj + a.k0 + (size_t)gh * a.dk, row0, n, [&](int r) { return VAR ? dts[VAR ? r : 0] : ks; }, kh, kl);
+  if (VAR) {
+    if (warp < a.hb) {
+      float c[2], d[2];
+      chunk_row_decays(a, h0 + warp, row0, n, c, d);
+      pws[warp][2 * lane] = c[0];
+      pws[warp][2 * lane + 1] = c[1];
+      dts[VAR ? warp : 0][2 * lane] = d[0];
+      dts[VAR ? warp : 0][2 * lane + 1] = d[1];
+    }
+  } else {
+    for (int i = tid; i < a.hb * (RC + 1); i += CK_THREADS) pws[i / (RC + 1)][i % (RC + 1)] = a.powers[(size_t)h0 * (RC + 1) + i];
+  }
+  load_turned<DKP>(a, a.proj + a.q0 + (size_t)gh * a.dk, row0, n, qh, ql);
+  load_turned<DKP>(a, a.proj + a.k0 + (size_t)gh * a.dk, row0, n, kh, kl);
+  ValueRegs next;
+  fetch_values(a, a.proj + a.v0 + (size_t)h0 * a.dv, row0, n, 0, next);
   __syncthreads();
   const int g = lane / 4, tq = lane % 4;
   const int rb = warp >> 1, side = warp & 1;         // rows 16 rb .. 16 rb + 15; which half of the keys and columns
@@ -822,42 +850,32 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
   const int q_at = (rb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * LDS + 8 * (lane / 16);
   const bool busy = rb * 16 < n;
 
-  // the weights d^(i-j) (q_i . k_j) of these rows and this warp's 32 keys, as two terms
-  {
-    float s[4][4];
+  // q_i . k_j of these rows and this warp's 32 keys
+  float s[4][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-    if (busy && 2 * side <= rb) {
+  for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+  if (busy && 2 * side <= rb) {
 #pragma unroll
-      for (int kk = 0; kk < DKP / 16; ++kk) {
-        uint32_t ah[4], al[4];
-        ldsm4(qh + q_at + kk * 16, ah);
-        ldsm4(ql + q_at + kk * 16, al);
+    for (int kk = 0; kk < DKP / 16; ++kk) {
+      uint32_t ah[4], al[4];
+      ldsm4(qh + q_at + kk * 16, ah);
+      ldsm4(ql + q_at + kk * 16, al);
 #pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          if (2 * side + np > rb) continue;        // keys after these rows
-          uint32_t bh[4], bl[4];
-          const int at = ((2 * side + np) * 16 + (lane % 8) + 8 * (lane / 16)) * LDS + kk * 16 + 8 * ((lane / 8) % 2);
-          ldsm4(kh + at, bh);
-          ldsm4(kl + at, bl);
-          mma_terms(s[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
-          mma_terms(s[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-        }
+      for (int np = 0; np < 2; ++np) {
+        if (2 * side + np > rb) continue;          // keys after these rows
+        uint32_t bh[4], bl[4];
+        const int at = ((2 * side + np) * 16 + (lane % 8) + 8 * (lane / 16)) * LDS + kk * 16 + 8 * ((lane / 8) % 2);
+        ldsm4(kh + at, bh);
+        ldsm4(kl + at, bl);
+        mma_terms(s[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+        mma_terms(s[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
       }
     }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int j = side * 32 + i * 8 + 2 * tq;
-      uint32_t wh, wl;
-      auto since = [&](int r, int from) { return VAR ? exp2f(pw[r] - pw[from]) : pw[r - from]; };   // decay from row `from` to r
-      split2(j <= r_lo ? s[i][0] * since(r_lo, j) : 0.f, j + 1 <= r_lo ? s[i][1] * since(r_lo, j + 1) : 0.f, wh, wl);
-      *reinterpret_cast<uint32_t*>(ph + r_lo * VLD + j) = wh;
-      *reinterpret_cast<uint32_t*>(pl + r_lo * VLD + j) = wl;
-      split2(j <= r_hi ? s[i][2] * since(r_hi, j) : 0.f, j + 1 <= r_hi ? s[i][3] * since(r_hi, j + 1) : 0.f, wh, wl);
-      *reinterpret_cast<uint32_t*>(ph + r_hi * VLD + j) = wh;
-      *reinterpret_cast<uint32_t*>(pl + r_hi * VLD + j) = wl;
-    }
   }
+  for (int hh = 0; hh < a.hb; ++hh) {
+  const int h = h0 + hh;
+  const float* pw = pws[hh];
+  const float* dt = dts[VAR ? hh : 0];
   const uint32_t* St = a.chunks + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
   const float f_lo = VAR ? exp2f(pw[r_lo]) : pw[r_lo + 1], f_hi = VAR ? exp2f(pw[r_hi]) : pw[r_hi + 1];
   float o[NS][4][4];
@@ -865,7 +883,24 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
 #pragma unroll
   for (int sl = 0; sl < NS; ++sl) {
     const int c0 = sl * 64;
-    __syncthreads();                               // the keys (or the last slab) have been read by everyone
+    __syncthreads();                               // the keys (or the last slab, the last weights) have been read by everyone
+    if (sl == 0) {                                 // the weights d^(i-j) (q_i . k_j), as two terms
+      auto weight = [&](float qk, int r, int from) {
+        if (from > r) return 0.f;
+        return VAR ? qk * exp2f(pw[r] - pw[from]) * dt[VAR ? from : 0] : qk * pw[r - from] * a.k_scale;
+      };
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int j = side * 32 + i * 8 + 2 * tq;
+        uint32_t wh, wl;
+        split2(weight(s[i][0], r_lo, j), weight(s[i][1], r_lo, j + 1), wh, wl);
+        *reinterpret_cast<uint32_t*>(ph + r_lo * VLD + j) = wh;
+        *reinterpret_cast<uint32_t*>(pl + r_lo * VLD + j) = wl;
+        split2(weight(s[i][2], r_hi, j), weight(s[i][3], r_hi, j + 1), wh, wl);
+        *reinterpret_cast<uint32_t*>(ph + r_hi * VLD + j) = wh;
+        *reinterpret_cast<uint32_t*>(pl + r_hi * VLD + j) = wl;
+      }
+    }
     if (a.planes) {                                // the state's terms as they are, sixteen bytes at a time
 #pragma unroll 4
       for (int x = tid; x < DKP * 16; x += CK_THREADS) {
@@ -877,7 +912,11 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
       }
       asm volatile("cp.async.commit_group;" ::: "memory");
     }
-    load_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, vh, vl);
+    store_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, next, nullptr, vh, vl);
+    {
+      const int more = hh * NS + sl + 1;           // the next slab's values are on their way while this one is worked on
+      if (more < a.hb * NS) fetch_values(a, a.proj + a.v0 + (size_t)(h0 + more / NS) * a.dv, row0, n, (more % NS) * 64, next);
+    }
     if (a.planes) {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     } else {
@@ -954,7 +993,7 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
           }
         }
       }
-    return;
+    continue;
   }
   ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 1);
   ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
@@ -990,6 +1029,7 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
         }
       }
     }
+  }
 }
 
 // ------------------------------------------------------------------ the row of all heads: skip, gate, norm
@@ -1002,7 +1042,7 @@ struct GatedNormArgs {
   long long gate_ld;
   const float* w;           // [n]
   void* out;                // [T, n]
-  int out_dt, n, dv, parts, gate_first;
+  int out_dt, n, dv, parts, gate_first, head_chunks;   // head_chunks: a chunk's elements are all one head's
   float eps;
 };
 
@@ -1017,6 +1057,7 @@ __global__ void __launch_bounds__(GN_THREADS) gated_norm_kernel(GatedNormArgs a)
   const int m = a.n / a.parts, base = blockIdx.y * m, chunks = m / VEC;
   grid_dep_wait();
   grid_dep_launch();
+  const bool fast = a.out_dt == NV_DT_BF16;        // (the result is rounded to bfloat16)
   const float* raw = a.raw + (size_t)t * a.n + base;
   const float* gate = a.gate + (size_t)t * a.gate_ld + base;
   const float* x = a.x + (size_t)t * a.x_ld + base;
@@ -1025,12 +1066,12 @@ __global__ void __launch_bounds__(GN_THREADS) gated_norm_kernel(GatedNormArgs a)
     if (a.skip) {
       const Vals<VEC> xv = ldv<VEC>(x + c * VEC);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.skip[(base + c * VEC + i) / a.dv], xv.v[i], v.v[i]);
+      for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.skip[(base + c * VEC + (a.head_chunks ? 0 : i)) / a.dv], xv.v[i], v.v[i]);
     }
     if (a.gate_first) {
       const Vals<VEC> g = ldv<VEC>(gate + c * VEC);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v.v[i] *= silu_of(g.v[i]);
+      for (int i = 0; i < VEC; ++i) v.v[i] *= fast ? silu_fast(g.v[i]) : silu_of(g.v[i]);
     }
     return v;
   };
@@ -1063,7 +1104,7 @@ __global__ void __launch_bounds__(GN_THREADS) gated_norm_kernel(GatedNormArgs a)
     if (!a.gate_first) {
       const Vals<VEC> g = ldv<VEC>(gate + c * VEC);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v.v[i] *= 1.f / (1.f + expf(-g.v[i]));
+      for (int i = 0; i < VEC; ++i) v.v[i] *= fast ? __fdividef(1.f, 1.f + __expf(-g.v[i])) : 1.f / (1.f + expf(-g.v[i]));
     }
     st_out<VEC>(a.out, a.out_dt, (size_t)t * a.n + base + (size_t)c * VEC, v);
   };
@@ -1099,11 +1140,12 @@ int launch_chunks(const RetArgs& a, int max_chunks, cudaStream_t s) {
   if (rc) return rc;
   rc = allow(retention_chunk_out_kernel<DKP, NS, VAR>, chunk_out_smem<DKP>());
   if (rc) return rc;
-  const dim3 grid(max_chunks, a.H);
+  const dim3 grid(max_chunks, a.H / a.hb);
   NV_RETURN_IF(launch_dep(retention_chunk_sum_kernel<DKP, VAR>, grid, dim3(CK_THREADS), chunk_sum_smem<DKP>(), s, a));
-  const dim3 rows(a.num_entries, a.H, (a.dk + 7) / 8);
-  if (a.planes && a.dv <= 128) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<1>, rows, dim3(256), 0, s, a));
-  else if (a.planes) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<2>, rows, dim3(256), 0, s, a));
+  const dim3 rows(a.num_entries, a.H, (a.dk + 7) / 8), rows2(a.num_entries, a.H, (a.dk + 15) / 16);
+  if (a.planes && a.dv <= 64) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<1, 16>, rows2, dim3(256), 0, s, a));
+  else if (a.planes && a.dv <= 128) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<1, 32>, rows, dim3(256), 0, s, a));
+  else if (a.planes) NV_RETURN_IF(launch_dep(retention_chunk_pass_rows_kernel<2, 32>, rows, dim3(256), 0, s, a));
   else NV_RETURN_IF(launch_dep(retention_chunk_pass_kernel, dim3(a.num_entries, a.H, (a.dk * a.dv + 255) / 256), dim3(256), 0, s, a));
   NV_RETURN_IF(launch_dep(retention_chunk_out_kernel<DKP, NS, VAR>, grid, dim3(CK_THREADS), chunk_out_smem<DKP>(), s, a));
   NV_RETURN_LAST();
@@ -1221,6 +1263,9 @@ NV_API int nv_retention(int what, const float* proj, long long ld, int q0, int k
             g0 % 2 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)table & 15) && !((uintptr_t)chunks & 15) &&
             !((uintptr_t)out & 15) && !((uintptr_t)raw & 7)) ? 1 : 0;
     a.planes = (dv % 8 == 0 && S_stride % 4 == 0 && !((uintptr_t)S & 15) && !((uintptr_t)chunks & 15)) ? 1 : 0;
+    // heads that share q and k, several to a block, as long as the step has blocks enough for the multiprocessors
+    a.hb = 1;
+    while (a.hb < CK_HEADS && (H / G) % (2 * a.hb) == 0 && (long long)max_chunks * (H / (2 * a.hb)) >= 288) a.hb *= 2;
     if (dk <= 64) return launch_chunks_dk<64>(a, max_chunks, s);
     if (dk <= 128) return launch_chunks_dk<128>(a, max_chunks, s);
     return launch_chunks_dk<256>(a, max_chunks, s);
@@ -1248,13 +1293,15 @@ NV_API int nv_gated_norm(const float* raw, const float* skip, const float* x, lo
   if (!dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;
   if (H < 1 || dv < 1 || parts < 1 || parts > 65535 || (H * dv) % parts || (skip && !x)) return NV_ERR_BAD_SIZE;
   if (T == 0) return NV_OK;
-  GatedNormArgs a = {raw, skip, x, x_ld, gate, gate_ld, w, out, out_dt, H * dv, dv, parts, gate_first, eps};
+  GatedNormArgs a = {raw, skip, x, x_ld, gate, gate_ld, w, out, out_dt, H * dv, dv, parts, gate_first, 0, eps};
   if (!x) a.x = raw;                     // (never read)
   const int m = a.n / parts;
   const bool vec = m % 4 == 0 && gate_ld % 4 == 0 && (!skip || (x_ld % 4 == 0 && !((uintptr_t)x & 15))) &&
                    !((uintptr_t)raw & 15) && !((uintptr_t)gate & 15) && !((uintptr_t)w & 15) && !((uintptr_t)out & 15);
+  a.head_chunks = dv % (vec ? 4 : 1) == 0;
   const int chunks = vec ? m / 4 : m;
-  const int threads = chunks < GN_THREADS ? (chunks + 31) / 32 * 32 : GN_THREADS;
+  const int half = (chunks + 1) / 2;     // two chunks a thread: their loads are in flight together
+  const int threads = half < GN_THREADS ? (half + 31) / 32 * 32 : GN_THREADS;
   if (vec) NV_RETURN_IF(launch_dep(gated_norm_kernel<4>, dim3(T, parts), dim3(threads), 0, s, a));
   else NV_RETURN_IF(launch_dep(gated_norm_kernel<1>, dim3(T, parts), dim3(threads), 0, s, a));
   NV_RETURN_LAST();

@@ -1,6 +1,7 @@
 """Generation through the Python entry point and the command line: greedy tokens equal the plain
 implementation's, sampled tokens equal the plain sampler's on the engine's logits, a preempted
 request resumes with the same tokens, and batch composition does not change a request's tokens."""
+import gc
 import os
 import subprocess
 import sys
@@ -367,6 +368,7 @@ def test_the_start_up_step_sizes_the_workspace(folders):
     sp = [SamplingParams(temperature=0.8 if i % 2 else 0.0, max_tokens=12, ignore_eos=True, seed=i) for i in range(6)]
     grew = {}
     for warm in (True, False):
+        gc.collect()                # engines of earlier tests that wait for the collector hold memory the steps could use
         torch.cuda.synchronize()
         torch.cuda.empty_cache()
         eng = engine(folders[case], dtype="bfloat16", max_model_len=160, num_kv_blocks=48, max_num_batched_tokens=256,
