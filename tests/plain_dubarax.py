@@ -74,9 +74,10 @@ def bucket_of(n, rows, far):
     return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
 
 
-def attention(h, W, p, m, mask, cap=0.0, slopes=None, table=None, far=0):
+def attention(h, W, p, m, mask, cap=0.0, slopes=None, table=None, far=0, only=None):
     """Grouped-query softmax attention with biased projections: a score is ``scale q.k``, then capped, then changed by what
-    the distance gives (``slopes`` per head, or a learned ``table`` [rows, heads] read through ``bucket_of``)."""
+    the distance gives (``slopes`` per head, or a learned ``table`` [rows, heads] read through ``bucket_of``).  ``only``: just
+    these rows are worked out and returned."""
     T, H, G, D = h.shape[0], int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
     V = int(m.get("vdim", D))
     q = (h @ W[p + "q"].T + W[p + "q.b"]).view(T, H, D)
@@ -84,7 +85,7 @@ def attention(h, W, p, m, mask, cap=0.0, slopes=None, table=None, far=0):
     v = (h @ W[p + "v"].T + W[p + "v.b"]).view(T, G, V)
     out = torch.zeros(T, H, V, dtype=F64)
     rows = [bucket_of(n, table.shape[0], far) for n in range(T)] if table is not None else None
-    for i in range(T):
+    for i in range(T) if only is None else only:
         lo = first_visible(i, mask)
         dist = [i - j for j in range(lo, i + 1)]
         for hd in range(H):
@@ -97,16 +98,17 @@ def attention(h, W, p, m, mask, cap=0.0, slopes=None, table=None, far=0):
             if table is not None:
                 s = s + table[[rows[n] for n in dist], hd]
             out[i, hd] = torch.softmax(s, dim=0) @ v[lo:i + 1, g]
-    return out.reshape(T, H * V) @ W[p + "o"].T + W[p + "o.b"]
+    out = out.reshape(T, H * V) if only is None else out.reshape(T, H * V)[only]
+    return out @ W[p + "o"].T + W[p + "o.b"]
 
 
-def chunk_attention(h, W, p, m):
-    return attention(h, W, p, m, ("chunk", int(m["mask"]["size"])), slopes=linear_bias(int(m["heads"])))
+def chunk_attention(h, W, p, m, only=None):
+    return attention(h, W, p, m, ("chunk", int(m["mask"]["size"])), slopes=linear_bias(int(m["heads"])), only=only)
 
 
-def window_attention(h, W, p, m):
+def window_attention(h, W, p, m, only=None):
     return attention(h, W, p, m, ("window", int(m["mask"]["size"])), cap=float(m["softcap"]), table=W[p + "rel"],
-                     far=int(m["bias_max"]))
+                     far=int(m["bias_max"]), only=only)
 
 
 # ------------------------------------------------------------------------------ matrix memories
