@@ -476,8 +476,8 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __gri
     const int h_lo = kvh * G + g0 + min(g, ng - 1), h_hi = kvh * G + g0 + min(g + 8, ng - 1);
     const float slope_lo = MOD && a.bias.slope ? a.bias.slope[h_lo] * 1.4426950408889634f : 0.f;
     const float slope_hi = MOD && a.bias.slope ? a.bias.slope[h_hi] * 1.4426950408889634f : 0.f;
-    const float* tab_lo = MOD && a.bias.table ? a.bias.table + (size_t)h_lo * (a.bias.last + 1) : nullptr;
-    const float* tab_hi = MOD && a.bias.table ? a.bias.table + (size_t)h_hi * (a.bias.last + 1) : nullptr;
+    const float* tab_lo = MOD ? bias_row(a.bias, h_lo) : nullptr;
+    const float* tab_hi = MOD ? bias_row(a.bias, h_hi) : nullptr;
     for (int i = warp; i < n_pages; i += WARPS) {
       mbar_wait(&full_bar[s], ph, a.err, 0x7112);
       const uint32_t kbase = smem0 + (uint32_t)s * stage_bytes;
@@ -792,7 +792,7 @@ NV_API int nv_attention_decode(const void* qkv, int q_dt, int q_stride, const vo
   // gates must have been written before the kernel that precedes this one on the stream.
   // softcap > 0: scaled scores are capped, s -> softcap * tanh(s / softcap).  chunk > 0: a row at position p sees the
   // positions from p / chunk * chunk on (and there is no window).  slopes [Hq]: head h's score with a key at distance n loses
-  // slopes[h] * n; bias_table [Hq, bias_len]: it gains bias_table[h][min(n, bias_len - 1)]; both after the cap.
+  // slopes[h] * n; bias_table [Hq, 64 + bias_len + 64] (see ScoreBias): it gains bias_table[h][min(n, bias_len - 1)]; both after the cap.
   // has_sink: a further key with the score sink_score and no value in every softmax; it keeps the tensor-core form
   // out.  float_weights: the weights keep all their bits in their product with the values (the lane-per-chunk
   // kernel multiplies in float32; the tensor-core form takes them as three bfloat16 terms instead of one).

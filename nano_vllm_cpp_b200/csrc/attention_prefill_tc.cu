@@ -249,7 +249,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       const bool live = r < nrows;
       const int w_lo = first_visible(p_row, a.window, a.chunk);
       const float slope = a.bias.slope ? a.bias.slope[h] * 1.4426950408889634f : 0.f;
-      const float* tab = a.bias.table ? a.bias.table + (size_t)h * (a.bias.last + 1) : nullptr;
+      const float* tab = bias_row(a.bias, h);
       const uint32_t lane_off = (uint32_t)(q * 32) << 16;
       float m = -INFINITY, l = 0.f;
       for (int i = 0; i < n_blocks; ++i) {
@@ -266,24 +266,25 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           if (a.map.cap1 > 0.f) {
 #pragma unroll
             for (int c = 0; c < TKB; ++c) s[c] = capped_log2(a.map, s[c]);
-          } else {
+            if (slope != 0.f) {
+              const float b0 = -slope * d0;
 #pragma unroll
-            for (int c = 0; c < TKB; ++c) s[c] *= a.map.in;
-          }
-          if (slope != 0.f) {
+              for (int c = 0; c < TKB; ++c) s[c] += fmaf(slope, (float)c, b0);
+            }
+          } else {
             const float b0 = -slope * d0;
 #pragma unroll
-            for (int c = 0; c < TKB; ++c) s[c] += fmaf(slope, (float)c, b0);
+            for (int c = 0; c < TKB; ++c) s[c] = fmaf(s[c], a.map.in, fmaf(slope, (float)c, b0));
           }
           if (tab) {
             if (p_row - j0 - (TKB - 1) >= a.bias.last) {   // every key of the block is as far as the table goes, or farther
               const float b = __ldg(tab + a.bias.last) * 1.4426950408889634f;
 #pragma unroll
               for (int c = 0; c < TKB; ++c) s[c] += b;
-            } else {
+            } else {                                       // distances from d - 63 on, within the row and its pads
+              const float* at = tab + max(p_row - j0, 0);  // (a block of keys after the row is masked whole)
 #pragma unroll
-              for (int c = 0; c < TKB; ++c)
-                s[c] = fmaf(__ldg(tab + min(max(p_row - j0 - c, 0), a.bias.last)), 1.4426950408889634f, s[c]);
+              for (int c = 0; c < TKB; ++c) s[c] = fmaf(__ldg(at - c), 1.4426950408889634f, s[c]);
             }
           }
         }
@@ -441,7 +442,7 @@ NV_API int nv_attention_prefill_tc(const void* qkv, int q_stride, int T, const v
   // has_sink: a further key with the score sink_score and no value in every softmax.  softcap > 0: a scaled score s
   // becomes softcap * tanh(s / softcap) before mask and softmax.  gate: head h's output of row t is multiplied by
   // sigmoid(gate[t * gate_ld + h]).  chunk > 0: a row at position p sees the positions from p / chunk * chunk on (and there is
-  // no window).  slopes [Hq], bias_table [Hq, bias_len]: head h's score with a key at distance n loses slopes[h] * n and
+  // no window).  slopes [Hq], bias_table [Hq, 64 + bias_len + 64] (see ScoreBias): head h's score with a key at distance n loses slopes[h] * n and
   // gains bias_table[h][min(n, bias_len - 1)], after the cap.
   if (chunk < 0 || (chunk > 0 && window > 0) || (bias_table && bias_len < 1)) return NV_ERR_BAD_SIZE;
   if (!nv_attention_prefill_tc_usable(D, page) || Hkv <= 0 || Hq % Hkv) return NV_ERR_UNSUPPORTED;

@@ -123,15 +123,21 @@ __device__ __forceinline__ float head_gate_of(const HeadGate& g, long long t, in
 }
 
 // What the distance between a row and a key gives to their score, after the cap and before the softmax: -slope[h] * n, and
-// table[h * (last + 1) + min(n, last)], for query head h and distance n (either array may be nullptr).
+// entry min(n, last) of the head's row of a table, for query head h and distance n (either array may be nullptr).  A table's
+// row has NV_BIAS_PAD further entries on both sides (copies of its ends), so that a run of neighbouring keys around either end
+// can be read without clamping every index.
+#define NV_BIAS_PAD 64
 struct ScoreBias {
   const float* slope;
   const float* table;
   int last;
 };
+__device__ __forceinline__ const float* bias_row(const ScoreBias& b, int h) {      // the row's entry 0
+  return b.table ? b.table + (size_t)h * (b.last + 1 + 2 * NV_BIAS_PAD) + NV_BIAS_PAD : nullptr;
+}
 __device__ __forceinline__ float score_bias_of(const ScoreBias& b, int h, int n) {
   float v = b.slope ? -b.slope[h] * (float)n : 0.f;
-  if (b.table) v += b.table[(size_t)h * (b.last + 1) + min(n, b.last)];
+  if (b.table) v += bias_row(b, h)[min(n, b.last)];
   return v;
 }
 // The first position that a row at position p sees: a sliding window (0: none), or the start of its chunk (0: no chunks).

@@ -441,13 +441,24 @@ def attention_decode(qkv, k_cache, v_cache, block_table, row_entry, positions, s
 
 def _score_bias(chunk: int, slopes, table, Hq: int):
     """``chunk`` > 0: a row at position p sees the positions from ``p // chunk * chunk`` on (and there is no window).
-    ``slopes`` (float32 [Hq]) and ``table`` (float32 [Hq, n]): the score of query head h with a key at distance d loses
-    ``slopes[h] * d`` and gains ``table[h, min(d, n - 1)]``, behind the cap.  What the attention launchers take for them."""
+    ``slopes`` (float32 [Hq]) and ``table`` (from ``bias_table_of`` a float32 [Hq, n]): the score of query head h with a key
+    at distance d loses ``slopes[h] * d`` and gains ``table[h, min(d, n - 1)]``, behind the cap.  What the attention
+    launchers take for them."""
     _cuda_contig(slopes, table)
     _f32(slopes, table)
     _need(slopes is None or slopes.numel() == Hq, "attention: one slope per query head")
-    _need(table is None or (table.dim() == 2 and table.shape[0] == Hq and table.shape[1] >= 1), "attention: a row of biases per query head")
-    return chunk, _p(slopes), _p(table), (table.shape[1] if table is not None else 0)
+    _need(table is None or (table.dim() == 2 and table.shape[0] == Hq and table.shape[1] > 2 * BIAS_PAD), "attention: a padded row of biases per query head")
+    return chunk, _p(slopes), _p(table), (table.shape[1] - 2 * BIAS_PAD if table is not None else 0)
+
+
+BIAS_PAD = 64
+
+
+def bias_table_of(table):
+    """A float32 [Hq, n] of biases by distance as the attention kernels take it: the ends of every row repeated on both sides,
+    so that they read runs of neighbouring distances without clamping every index."""
+    t = table.float()
+    return torch.cat([t[:, :1].expand(-1, BIAS_PAD), t, t[:, -1:].expand(-1, BIAS_PAD)], dim=1).contiguous()
 
 
 def _head_gates(gate, T: int, Hq: int):

@@ -1404,7 +1404,7 @@ NV_API int nv_paged_attention_general(const void* q, int q_dt, const void* kc, c
                                       int Hkv, int Hv, int D, int Dv, int key_span, int page, float softcap,
                                       const float* gate, long long gate_ld, int chunk, const float* slopes,
                                       const float* bias_table, int bias_len, cudaStream_t s) {
-  // chunk > 0: a row at position p sees the positions from p / chunk * chunk on; slopes [Hq], bias_table [Hq, bias_len]: what
+  // chunk > 0: a row at position p sees the positions from p / chunk * chunk on; slopes [Hq], bias_table [Hq, 64 + bias_len + 64]: what
   // the distance n takes off a head's score, slopes[h] * n, and gives to it, bias_table[h][min(n, bias_len - 1)], after the cap
   if (chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0)) || (bias_table && bias_len < 1)) return NV_ERR_BAD_SIZE;
   if (!dt_ok(q_dt) || !dt_ok(cache_dt) || !dt_ok(out_dt)) return NV_ERR_BAD_DTYPE;

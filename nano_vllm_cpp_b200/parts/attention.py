@@ -194,7 +194,7 @@ class PagedAttention(Mixer):
         if self.distance_far is not None:       # spread out: one number per head and distance
             rel = fetch(n["rel"]).float()
             rows = torch.tensor(distance_buckets(rel.shape[0], self.distance_far), device=rel.device)
-            self.bias_table = rel[rows].t().contiguous()
+            self.bias_table = ops.bias_table_of(rel[rows].t())
         # q, k and v rows are stacked so that one product makes all three (src/model.cpp:508-513)
         rows = [fetch(n["q"])]
         if self.own_kv:

@@ -602,6 +602,7 @@ def test_score_options_in_every_kernel(D, H, G, page):
     bt = batch.block_tables[0]
     scale = 1.5 / math.sqrt(D)
     slopes, table = dev32(0.05 + 0.2 * rnd(4, H).abs()), dev32(2.0 * rnd(5, H, 41))
+    padded = ops.bias_table_of(table)
     rows = [(e, p + t, r) for r, (e, p, t) in enumerate((e, p, t) for e, (n, p) in enumerate(zip(lengths, pos0)) for t in range(n))]
     picked = [x for x in rows if x[2] % 17 == 0 or x[0] == 2 or x[1] in (20, 21, 39, 40)]
 
@@ -627,7 +628,7 @@ def test_score_options_in_every_kernel(D, H, G, page):
     for case, (cap, sl, tb, window, chunk, sink) in enumerate([(4.0, 0, 1, 33, 0, 0), (0, 1, 0, 0, 40, 0), (6.0, 1, 1, 0, 21, 0), (0, 0, 1, 0, 0, 0),
                                                               (3.0, 0, 0, 0, 500, 0), (0, 0, 0, 0, 64, 0), (5.0, 1, 0, 77, 0, 1)]):
         want = plain(cap, sl, tb, window, chunk, sink)
-        opts = dict(softcap=cap, chunk=chunk, slopes=slopes if sl else None, bias_table=table if tb else None, sink_score=0.0 if sink else None)
+        opts = dict(softcap=cap, chunk=chunk, slopes=slopes if sl else None, bias_table=padded if tb else None, sink_score=0.0 if sink else None)
         err = ops.ErrorFlag(DEV)
         qd = q.to(DEV)
         for kernel, terms in (("auto", 1), ("auto", 3), ("mma", 1), ("mma", 3)):
