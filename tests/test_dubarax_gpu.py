@@ -357,7 +357,7 @@ def test_routing_limited_to_groups(E, K, count, keep):
 @pytest.mark.parametrize("fast", [True, False])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("width,mlp", [(64, pd.moe(8, 2, 24, 4, 2, 40)), (64, pd.moe(6, 3, 40, 2, 1, 80)), (50, pd.moe(3, 2, 20, 3, 2, 0)),
-                                       (256, pd.moe(16, 4, 128, 4, 2, 256)), (128, pd.moe(12, 3, 64, 4, 3, 96)), (64, pd.moe(1, 1, 16, 1, 1, 16))])
+                                       (256, pd.moe(16, 4, 128, 4, 2, 256)), (128, pd.moe(10, 3, 128, 5, 3, 192)), (64, pd.moe(1, 1, 16, 1, 1, 16))])
 def test_mixture_alone(width, mlp, dtype, fast):
     """One row, a handful, and more rows than the one-launch routing takes; shared experts of a whole number of expert widths
     and of another width, and none."""
@@ -555,7 +555,7 @@ def attention_weights(m, width, seed):
 
 
 SIZES = [(4, 2, 32, 48, 0.2), (3, 3, 40, 24, 0.11), (8, 2, 64, 64, 0.125), (2, 2, 128, 128, 0.09), (6, 1, 96, 96, 0.1), (20, 1, 64, 32, 0.12),
-         (2, 1, 256, 256, 0.06), (2, 1, 192, 80, 0.07), (1, 1, 8, 16, 0.5), (8, 1, 48, 48, 0.14), (17, 1, 144, 136, 0.08)]
+         (2, 1, 256, 256, 0.06), (2, 1, 192, 80, 0.07), (1, 1, 8, 16, 0.5), (12, 2, 48, 40, 0.13), (17, 1, 144, 136, 0.08)]
 MASKS = [("chunk", 20), ("chunk", 64), ("chunk", 1000), ("window", 19), ("window", 1), ("window", 400)]
 
 
@@ -856,7 +856,7 @@ def drawn_config(seed):
         heads = kv * rng.choice([1, 2, 4])
         if kind == "parallel":
             n = rng.choice([1, 2, 3])
-            layers.append(pd.parallel_layer(pd.chunk_part(heads, kv, dim, rng.choice([dim, 32]), rng.choice([5, 16, 31, 48, 200]), rng.uniform(0.1, 0.3)),
+            layers.append(pd.parallel_layer(pd.chunk_part(heads, kv, dim, rng.choice([dim, 32]), rng.choice([5, 16, 31, 48, 180]), rng.uniform(0.1, 0.3)),
                                             pd.lightning_part(n, rng.choice([16, 24, 64, 80]), rng.choice([16, 40, 64, 96]), [rng.uniform(0.5, 1.0) for _ in range(n)]),
                                             rng.uniform(0.3, 1.2), rng.uniform(0.3, 1.2), mlp=ff, type=kind + suffix))
         elif kind == "attention":
