@@ -371,11 +371,12 @@ __global__ void __launch_bounds__(256) rope_store_kernel(void* __restrict__ qkv,
       const size_t cbase = (((size_t)blk * Hkv + (h - Hq)) * page + slot) * D;
       *((uint4*)((bf16*)kc + cbase) + c) = *((const uint4*)((const bf16*)qkv + row + (size_t)h * D) + c);
     }
-  } else
-  for (int i = threadIdx.x; i < (k_hi - k_lo) * tail; i += blockDim.x) {
-    const int h = k_lo + i / tail, d = rotary_dim + i % tail;
-    const size_t cbase = (((size_t)blk * Hkv + (h - Hq)) * page + slot) * D;
-    st_dt(kc, cache_dt, cbase + d, ld_dt(qkv, dt, row + (size_t)h * D + d));
+  } else {
+    for (int i = threadIdx.x; i < (k_hi - k_lo) * tail; i += blockDim.x) {
+      const int h = k_lo + i / tail, d = rotary_dim + i % tail;
+      const size_t cbase = (((size_t)blk * Hkv + (h - Hq)) * page + slot) * D;
+      st_dt(kc, cache_dt, cbase + d, ld_dt(qkv, dt, row + (size_t)h * D + d));
+    }
   }
   const int v_lo = max(h_begin, Hq + Hkv);
   if (packed) {                                    // 16-byte copies of v

@@ -873,162 +873,162 @@ __global__ void __launch_bounds__(CK_THREADS, DKP <= 128 && NS <= 2 ? 2 : 1) ret
     }
   }
   for (int hh = 0; hh < a.hb; ++hh) {
-  const int h = h0 + hh;
-  const float* pw = pws[hh];
-  const float* dt = dts[VAR ? hh : 0];
-  const uint32_t* St = a.chunks + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
-  const float f_lo = VAR ? exp2f(pw[r_lo]) : pw[r_lo + 1], f_hi = VAR ? exp2f(pw[r_hi]) : pw[r_hi + 1];
-  float o[NS][4][4];
-  float ss_lo = 0.f, ss_hi = 0.f;
+    const int h = h0 + hh;
+    const float* pw = pws[hh];
+    const float* dt = dts[VAR ? hh : 0];
+    const uint32_t* St = a.chunks + ((size_t)blockIdx.x * a.H + h) * a.dk * a.dv;
+    const float f_lo = VAR ? exp2f(pw[r_lo]) : pw[r_lo + 1], f_hi = VAR ? exp2f(pw[r_hi]) : pw[r_hi + 1];
+    float o[NS][4][4];
+    float ss_lo = 0.f, ss_hi = 0.f;
 #pragma unroll
-  for (int sl = 0; sl < NS; ++sl) {
-    const int c0 = sl * 64;
-    __syncthreads();                               // the keys (or the last slab, the last weights) have been read by everyone
-    if (sl == 0) {                                 // the weights d^(i-j) (q_i . k_j), as two terms
-      auto weight = [&](float qk, int r, int from) {
-        if (from > r) return 0.f;
-        return VAR ? qk * exp2f(pw[r] - pw[from]) * dt[VAR ? from : 0] : qk * pw[r - from] * a.k_scale;
-      };
+    for (int sl = 0; sl < NS; ++sl) {
+      const int c0 = sl * 64;
+      __syncthreads();                               // the keys (or the last slab, the last weights) have been read by everyone
+      if (sl == 0) {                                 // the weights d^(i-j) (q_i . k_j), as two terms
+        auto weight = [&](float qk, int r, int from) {
+          if (from > r) return 0.f;
+          return VAR ? qk * exp2f(pw[r] - pw[from]) * dt[VAR ? from : 0] : qk * pw[r - from] * a.k_scale;
+        };
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int j = side * 32 + i * 8 + 2 * tq;
-        uint32_t wh, wl;
-        split2(weight(s[i][0], r_lo, j), weight(s[i][1], r_lo, j + 1), wh, wl);
-        *reinterpret_cast<uint32_t*>(ph + r_lo * VLD + j) = wh;
-        *reinterpret_cast<uint32_t*>(pl + r_lo * VLD + j) = wl;
-        split2(weight(s[i][2], r_hi, j), weight(s[i][3], r_hi, j + 1), wh, wl);
-        *reinterpret_cast<uint32_t*>(ph + r_hi * VLD + j) = wh;
-        *reinterpret_cast<uint32_t*>(pl + r_hi * VLD + j) = wl;
+        for (int i = 0; i < 4; ++i) {
+          const int j = side * 32 + i * 8 + 2 * tq;
+          uint32_t wh, wl;
+          split2(weight(s[i][0], r_lo, j), weight(s[i][1], r_lo, j + 1), wh, wl);
+          *reinterpret_cast<uint32_t*>(ph + r_lo * VLD + j) = wh;
+          *reinterpret_cast<uint32_t*>(pl + r_lo * VLD + j) = wl;
+          split2(weight(s[i][2], r_hi, j), weight(s[i][3], r_hi, j + 1), wh, wl);
+          *reinterpret_cast<uint32_t*>(ph + r_hi * VLD + j) = wh;
+          *reinterpret_cast<uint32_t*>(pl + r_hi * VLD + j) = wl;
+        }
       }
-    }
-    if (a.planes) {                                // the state's terms as they are, sixteen bytes at a time
+      if (a.planes) {                                // the state's terms as they are, sixteen bytes at a time
 #pragma unroll 4
-      for (int x = tid; x < DKP * 16; x += CK_THREADS) {
-        const int d = x >> 4, c = 8 * (x & 7), term = (x >> 3) & 1;
-        bf16* dst = (term ? kl : kh) + d * VLD + c;
-        if (d < a.dk && c0 + c < a.dv)
-          cp_async16(dst, reinterpret_cast<const bf16*>(St + (size_t)d * a.dv) + term * a.dv + c0 + c);
-        else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        for (int x = tid; x < DKP * 16; x += CK_THREADS) {
+          const int d = x >> 4, c = 8 * (x & 7), term = (x >> 3) & 1;
+          bf16* dst = (term ? kl : kh) + d * VLD + c;
+          if (d < a.dk && c0 + c < a.dv)
+            cp_async16(dst, reinterpret_cast<const bf16*>(St + (size_t)d * a.dv) + term * a.dv + c0 + c);
+          else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
       }
-      asm volatile("cp.async.commit_group;" ::: "memory");
-    }
-    store_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, next, nullptr, vh, vl);
-    {
-      const int more = hh * NS + sl + 1;           // the next slab's values are on their way while this one is worked on
-      if (more < a.hb * NS) fetch_values(a, a.proj + a.v0 + (size_t)(h0 + more / NS) * a.dv, row0, n, (more % NS) * 64, next);
-    }
-    if (a.planes) {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    } else {
-      for (int x = tid; x < DKP * 64; x += CK_THREADS) {
-        const int d = x / 64, c = x % 64;
-        const uint32_t w = d < a.dk && c0 + c < a.dv ? St[(size_t)d * a.dv + c0 + c] : 0u;
-        const __nv_bfloat162 pk = *reinterpret_cast<const __nv_bfloat162*>(&w);
-        kh[d * VLD + c] = pk.x;
-        kl[d * VLD + c] = pk.y;
+      store_values(a, a.proj + a.v0 + (size_t)h * a.dv, row0, n, c0, next, nullptr, vh, vl);
+      {
+        const int more = hh * NS + sl + 1;           // the next slab's values are on their way while this one is worked on
+        if (more < a.hb * NS) fetch_values(a, a.proj + a.v0 + (size_t)(h0 + more / NS) * a.dv, row0, n, (more % NS) * 64, next);
       }
+      if (a.planes) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+      } else {
+        for (int x = tid; x < DKP * 64; x += CK_THREADS) {
+          const int d = x / 64, c = x % 64;
+          const uint32_t w = d < a.dk && c0 + c < a.dv ? St[(size_t)d * a.dv + c0 + c] : 0u;
+          const __nv_bfloat162 pk = *reinterpret_cast<const __nv_bfloat162*>(&w);
+          kh[d * VLD + c] = pk.x;
+          kl[d * VLD + c] = pk.y;
+        }
+      }
+      __syncthreads();
+      float (&oc)[4][4] = o[sl];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) oc[i][0] = oc[i][1] = oc[i][2] = oc[i][3] = 0.f;
+      if (!busy || c0 + side * 32 >= a.dv) continue;
+#pragma unroll
+      for (int kk = 0; kk < DKP / 16; ++kk) {
+        if (kk * 16 >= a.dk) continue;
+        uint32_t ah[4], al[4];
+        ldsm4(qh + q_at + kk * 16, ah);
+        ldsm4(ql + q_at + kk * 16, al);
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t bh[4], bl[4];
+          const int at = (kk * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + side * 32 + np * 16 + 8 * (lane / 16);
+          ldsm4_t(kh + at, bh);
+          ldsm4_t(kl + at, bl);
+          mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+          mma_terms(oc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { oc[i][0] *= f_lo; oc[i][1] *= f_lo; oc[i][2] *= f_hi; oc[i][3] *= f_hi; }
+#pragma unroll
+      for (int kb = 0; kb < 4; ++kb) {
+        if (kb > rb) continue;
+        uint32_t ah[4], al[4];
+        const int pat = (rb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + kb * 16 + 8 * (lane / 16);
+        ldsm4(ph + pat, ah);
+        ldsm4(pl + pat, al);
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t bh[4], bl[4];
+          const int at = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + side * 32 + np * 16 + 8 * (lane / 16);
+          ldsm4_t(vh + at, bh);
+          ldsm4_t(vl + at, bl);
+          mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
+          mma_terms(oc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {                  // (columns beyond dv are zero)
+        ss_lo = fmaf(oc[i][0], oc[i][0], fmaf(oc[i][1], oc[i][1], ss_lo));
+        ss_hi = fmaf(oc[i][2], oc[i][2], fmaf(oc[i][3], oc[i][3], ss_hi));
+      }
+    }
+    if (a.raw_out) {
+#pragma unroll
+      for (int sl = 0; sl < NS; ++sl)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int r = half ? r_hi : r_lo;
+          if (r >= n) continue;
+          float* to = a.raw + ((size_t)(row0 + r) * a.H + h) * a.dv;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int col = sl * 64 + side * 32 + i * 8 + 2 * tq;
+            if (col >= a.dv) continue;
+            if (a.v2) *reinterpret_cast<float2*>(to + col) = make_float2(o[sl][i][2 * half], o[sl][i][2 * half + 1]);
+            else {
+              to[col] = o[sl][i][2 * half];
+              if (col + 1 < a.dv) to[col + 1] = o[sl][i][2 * half + 1];
+            }
+          }
+        }
+      continue;
+    }
+    ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 1);
+    ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
+    ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 1);
+    ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 2);
+    if (tq == 0) {
+      squares[side][r_lo] = ss_lo;
+      squares[side][r_hi] = ss_hi;
     }
     __syncthreads();
-    float (&oc)[4][4] = o[sl];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) oc[i][0] = oc[i][1] = oc[i][2] = oc[i][3] = 0.f;
-    if (!busy || c0 + side * 32 >= a.dv) continue;
-#pragma unroll
-    for (int kk = 0; kk < DKP / 16; ++kk) {
-      if (kk * 16 >= a.dk) continue;
-      uint32_t ah[4], al[4];
-      ldsm4(qh + q_at + kk * 16, ah);
-      ldsm4(ql + q_at + kk * 16, al);
-#pragma unroll
-      for (int np = 0; np < 2; ++np) {
-        uint32_t bh[4], bl[4];
-        const int at = (kk * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + side * 32 + np * 16 + 8 * (lane / 16);
-        ldsm4_t(kh + at, bh);
-        ldsm4_t(kl + at, bl);
-        mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
-        mma_terms(oc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) { oc[i][0] *= f_lo; oc[i][1] *= f_lo; oc[i][2] *= f_hi; oc[i][3] *= f_hi; }
-#pragma unroll
-    for (int kb = 0; kb < 4; ++kb) {
-      if (kb > rb) continue;
-      uint32_t ah[4], al[4];
-      const int pat = (rb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + kb * 16 + 8 * (lane / 16);
-      ldsm4(ph + pat, ah);
-      ldsm4(pl + pat, al);
-#pragma unroll
-      for (int np = 0; np < 2; ++np) {
-        uint32_t bh[4], bl[4];
-        const int at = (kb * 16 + (lane % 8) + 8 * ((lane / 8) % 2)) * VLD + side * 32 + np * 16 + 8 * (lane / 16);
-        ldsm4_t(vh + at, bh);
-        ldsm4_t(vl + at, bl);
-        mma_terms(oc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
-        mma_terms(oc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {                  // (columns beyond dv are zero)
-      ss_lo = fmaf(oc[i][0], oc[i][0], fmaf(oc[i][1], oc[i][1], ss_lo));
-      ss_hi = fmaf(oc[i][2], oc[i][2], fmaf(oc[i][3], oc[i][3], ss_hi));
-    }
-  }
-  if (a.raw_out) {
+    const float n_lo = rsqrtf((squares[0][r_lo] + squares[1][r_lo]) / (float)a.dv + a.eps);
+    const float n_hi = rsqrtf((squares[0][r_hi] + squares[1][r_hi]) / (float)a.dv + a.eps);
 #pragma unroll
     for (int sl = 0; sl < NS; ++sl)
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int r = half ? r_hi : r_lo;
         if (r >= n) continue;
-        float* to = a.raw + ((size_t)(row0 + r) * a.H + h) * a.dv;
+        const float rn = half ? n_hi : n_lo;
+        const float* gp = a.proj + (size_t)(row0 + r) * a.ld + a.g0 + (size_t)h * a.dv;
+        const size_t at = ((size_t)(row0 + r) * a.H + h) * a.dv;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int col = sl * 64 + side * 32 + i * 8 + 2 * tq;
           if (col >= a.dv) continue;
-          if (a.v2) *reinterpret_cast<float2*>(to + col) = make_float2(o[sl][i][2 * half], o[sl][i][2 * half + 1]);
-          else {
-            to[col] = o[sl][i][2 * half];
-            if (col + 1 < a.dv) to[col + 1] = o[sl][i][2 * half + 1];
+          const float x = o[sl][i][2 * half] * rn, y = o[sl][i][2 * half + 1] * rn;
+          if (a.v2 && a.out_dt == NV_DT_BF16) {
+            const float2 gg = *reinterpret_cast<const float2*>(gp + col);
+            *reinterpret_cast<__nv_bfloat162*>((bf16*)a.out + at + col) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
+          } else {
+            st_dt(a.out, a.out_dt, at + col, x * silu_fast(gp[col]));
+            if (col + 1 < a.dv) st_dt(a.out, a.out_dt, at + col + 1, y * silu_fast(gp[col + 1]));
           }
         }
       }
-    continue;
-  }
-  ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 1);
-  ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
-  ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 1);
-  ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 2);
-  if (tq == 0) {
-    squares[side][r_lo] = ss_lo;
-    squares[side][r_hi] = ss_hi;
-  }
-  __syncthreads();
-  const float n_lo = rsqrtf((squares[0][r_lo] + squares[1][r_lo]) / (float)a.dv + a.eps);
-  const float n_hi = rsqrtf((squares[0][r_hi] + squares[1][r_hi]) / (float)a.dv + a.eps);
-#pragma unroll
-  for (int sl = 0; sl < NS; ++sl)
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = half ? r_hi : r_lo;
-      if (r >= n) continue;
-      const float rn = half ? n_hi : n_lo;
-      const float* gp = a.proj + (size_t)(row0 + r) * a.ld + a.g0 + (size_t)h * a.dv;
-      const size_t at = ((size_t)(row0 + r) * a.H + h) * a.dv;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int col = sl * 64 + side * 32 + i * 8 + 2 * tq;
-        if (col >= a.dv) continue;
-        const float x = o[sl][i][2 * half] * rn, y = o[sl][i][2 * half + 1] * rn;
-        if (a.v2 && a.out_dt == NV_DT_BF16) {
-          const float2 gg = *reinterpret_cast<const float2*>(gp + col);
-          *reinterpret_cast<__nv_bfloat162*>((bf16*)a.out + at + col) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
-        } else {
-          st_dt(a.out, a.out_dt, at + col, x * silu_fast(gp[col]));
-          if (col + 1 < a.dv) st_dt(a.out, a.out_dt, at + col + 1, y * silu_fast(gp[col + 1]));
-        }
-      }
-    }
   }
 }
 

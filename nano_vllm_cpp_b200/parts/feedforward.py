@@ -118,7 +118,8 @@ class SparseMoeSwiGLU(FeedForward):
     float32; the ``top_k`` largest ``s + correction`` are chosen (``choice_bias``: a learned vector ``correction``
     [experts] that steers the choice only), and the weights are the chosen experts' ``s`` without it.  ``route_scale``
     multiplies the weights.  ``groups`` = (count, keep): the experts form ``count`` equal groups of neighbours, a group
-    counts as its largest score, and only experts of the ``keep`` best groups can be chosen.  ``router_bias`` (softmax scores): a learned vector ``router_bias`` [experts] is added to the
+    counts as its largest score, and only experts of the ``keep`` best groups can be chosen.  ``router_bias`` (softmax
+    scores): a learned vector ``router_bias`` [experts] is added to the
     logits before the softmax; with ``renormalize`` the weights are then the softmax over the chosen biased logits.
     ``shared_gate=False``: the shared expert has no gate and is added as it is.  ``names``
     gives the tensors' names where they are not the usual ones (keys: router, router_bias, correction, shared_gate, and the
@@ -295,9 +296,10 @@ class SparseMoeSwiGLU(FeedForward):
         fast = (ctx.fast_kernels and h.dtype == torch.bfloat16 and self.w_gate_up.dtype == torch.bfloat16
                 and self.w_down.dtype == torch.bfloat16 and self.hidden % 8 == 0 and self.inter % 8 == 0)
         al = self._alignment(T * KT, self.E + C, dev, fast)
+        groups = self.groups[0] if self.groups else 0
         x_sorted = None
         if (fast and C and T <= SIDE_MAX_ROWS and al.secondary is None
-                and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden, self.groups[0] if self.groups else 0)):
+                and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden, groups)):
             return self._forward_beside(h, logits, gate_logit, idx, score, al)
         if fast and C and T >= 256 and al.secondary is None:
             return self._forward_beside(h, logits, gate_logit, idx, score, al, many=True)
@@ -307,7 +309,7 @@ class SparseMoeSwiGLU(FeedForward):
             if self._counters is None:
                 self._counters = torch.zeros(2, dtype=torch.int32, device=dev)
             zero, c0, c1 = self._counters, self._counters[0:1], self._counters[1:2]
-        if fast and al.secondary is None and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden, self.groups[0] if self.groups else 0):
+        if fast and al.secondary is None and ops.moe_route_small_usable(T, self.E, self.K, C, self.hidden, groups):
             x_sorted = ops.moe_route_small(logits, self.K, self.renorm, C, gate_logit, idx, score, al, ctx.err,
                                            x=None, zero=zero, rule=self.rule)   # one block copies rows slower than the copy kernel does
         else:
